@@ -13,14 +13,18 @@
 //                           split-K slabs): q and k turned by the rotary angle of the token's position (optional),
 //                           scaled, v copied, and the decay of every key channel worked out from a low-rank map:
 //                               z = W2 (x W1^T) + b,   a = sigmoid(z)^(1/tau) = exp(log_sigmoid(z) / tau)
+//                           or (decay form 1)  z = W2 tanh(x W1^T) + b,   a = exp(-exp(z)); the decay alone where q, k and v are
+//                           read from the projections as they are
 //   wllm_linattn_scan       the recurrence.  Grid (tiles of 64 value columns, heads, requests); a lane owns two
 //                           columns of S, a warp a run of at most 16 key channels of them, in registers.  Tokens
 //                           arrive in tiles of 8 through a two-stage cp.async ring; the warps' partial dot products of a
 //                           tile's tokens meet in shared memory once a tile and are added in warp order.  Long portions of prompts are cut
 //                           into segments that are walked side by side: from zero for their local end states, which a
 //                           small kernel chains into start states, and once more from those for the outputs.
-//   wllm_head_gate_norm     per head: o / sqrt(mean(o^2) + eps) [* w] * silu(g), rounded once to the matrix type
-//                           (the operand of the output projection).
+//                           With a bonus u per key channel the output is taken in front of the update, with the token's own
+//                           key and value counted u times: o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t (time mixing).
+//   wllm_head_gate_norm     per head: o / sqrt(mean(o^2) + eps) [* w] * silu(g) [* factor], rounded once to the matrix type
+//                           (the operand of the output projection).  w is shared by the heads or a gain of the whole row.
 #include "common.cuh"
 
 __device__ __forceinline__ float la_any(const void* p, int dtype, size_t i) {
@@ -59,7 +63,7 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
                        const int* __restrict__ positions, const float* __restrict__ inv_freq, int rot_dim,
                        float q_scale, float k_scale, const void* __restrict__ w2, const void* __restrict__ b2,
                        int w_dtype, float inv_tau, float* __restrict__ q, float* __restrict__ k,
-                       float* __restrict__ v, float* __restrict__ decay) {
+                       float* __restrict__ v, float* __restrict__ decay, int form) {
     __shared__ __align__(16) float low_s[PREP_RK][TT];      // the tokens' low-rank vectors, a run of PREP_RK columns at a time
     pdl_begin();
     const int t_lo = blockIdx.x * TT, h = blockIdx.y;
@@ -67,7 +71,7 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
     const int half = rot_dim >> 1, rest = D - rot_dim;
     // q and k: the rotated pairs, then the channels behind them; v: a copy.  One flat loop each over (token, element),
     // so that a thread's loads do not wait for one another.
-    for (int which = 0; which < 2; ++which) {
+    for (int which = 0; which < (q ? 2 : 0); ++which) {
         const int off = (which ? k_off : q_off) + h * D;
         float* base = which ? k : q;
         const float scale = which ? k_scale : q_scale;
@@ -87,7 +91,7 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
             base[((size_t)t * H + h) * D + c] = la_in<MULTI>(fused, in_dtype, parts, part_stride, (size_t)t * row_stride + off + c) * scale;
         }
     }
-    for (int idx = threadIdx.x; idx < count * V; idx += blockDim.x) {
+    for (int idx = threadIdx.x; idx < (q ? count * V : 0); idx += blockDim.x) {
         const int tt = idx / V, c = idx - tt * V, t = t_lo + tt;
         v[((size_t)t * H + h) * V + c] = la_in<MULTI>(fused, in_dtype, parts, part_stride, (size_t)t * row_stride + v_off + h * V + c);
     }
@@ -108,8 +112,10 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
             __syncthreads();
             for (int idx = threadIdx.x; idx < TT * PREP_RK; idx += blockDim.x) {
                 const int r = idx / TT, tt = idx % TT;
-                low_s[r][tt] = (tt < count && r < rk)
+                float low = (tt < count && r < rk)
                     ? la_in<MULTI>(fused, in_dtype, parts, part_stride, (size_t)(t_lo + tt) * row_stride + a_off + r0 + r) : 0.f;
+                if (form == 1) low = tanhf(low);
+                low_s[r][tt] = low;
             }
             float wr[PREP_RK];
             if (vec && rk == PREP_RK) {
@@ -153,10 +159,32 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
                 if (tt >= count) break;
                 // log(sigmoid(z)) = min(z, 0) - log(1 + e^-|z|), exact at both ends
                 const float log_sig = fminf(z[tt], 0.f) - log1pf(expf(-fabsf(z[tt])));
-                decay[((size_t)(t_lo + tt) * H + h) * D + c] = expf(log_sig * inv_tau);
+                decay[((size_t)(t_lo + tt) * H + h) * D + c] = form == 1 ? expf(-expf(z[tt])) : expf(log_sig * inv_tau);
             }
         }
     }
+}
+
+// q null: q, k and v stay where they are and only the decay is worked out.  form 0: sigmoid(z)^(1/tau); 1: exp(-exp(z)) over tanh of
+// the low-rank columns (tau is not used).
+WLLM_API int wllm_linattn_prepare_form(const void* fused, int in_dtype, int row_stride, int parts, long long part_stride, int q_off,
+                                       int k_off, int v_off, int a_off, int n, int H, int D, int V, int rank, const int* positions,
+                                       const float* inv_freq, int rot_dim, float q_scale, float k_scale, const void* w2,
+                                       const void* b2, int w_dtype, float tau, float* q, float* k, float* v, float* decay, int form,
+                                       cudaStream_t stream) {
+    if (n <= 0) return WLLM_OK;
+    if (H <= 0 || H > 65535 || D <= 0 || V <= 0 || parts < 1 || rot_dim < 0 || rot_dim > D || (rot_dim & 1) || form < 0 || form > 1) return WLLM_BAD_SIZE;
+    if (a_off >= 0 && (rank <= 0 || !(tau > 0.f) || !w2 || !b2 || !decay)) return WLLM_BAD_SIZE;
+    if ((in_dtype != WLLM_BF16 && in_dtype != WLLM_F32) || (a_off >= 0 && w_dtype != WLLM_BF16 && w_dtype != WLLM_F32))
+        return WLLM_BAD_DTYPE;
+#define PREP2(TT, M) wllm_launch(linattn_prepare_kernel<TT, M>, dim3((n + TT - 1) / TT, H), 128, 0, stream, fused, \
+        in_dtype, row_stride, parts, (size_t)part_stride, q_off, k_off, v_off, a_off, n, H, D, V, rank, positions, \
+        inv_freq, rot_dim, q_scale, k_scale, w2, b2, w_dtype, a_off >= 0 ? 1.0f / tau : 0.f, q, k, v, decay, form)
+#define PREP(TT) (parts > 1 ? PREP2(TT, true) : PREP2(TT, false))
+    if ((long long)n * H >= 2048) return PREP(8);
+    return PREP(1);
+#undef PREP
+#undef PREP2
 }
 
 WLLM_API int wllm_linattn_prepare(const void* fused, int in_dtype, int row_stride, int parts, long long part_stride, int q_off,
@@ -164,19 +192,9 @@ WLLM_API int wllm_linattn_prepare(const void* fused, int in_dtype, int row_strid
                                   const float* inv_freq, int rot_dim, float q_scale, float k_scale, const void* w2,
                                   const void* b2, int w_dtype, float tau, float* q, float* k, float* v, float* decay,
                                   cudaStream_t stream) {
-    if (n <= 0) return WLLM_OK;
-    if (H <= 0 || H > 65535 || D <= 0 || V <= 0 || parts < 1 || rot_dim < 0 || rot_dim > D || (rot_dim & 1)) return WLLM_BAD_SIZE;
-    if (a_off >= 0 && (rank <= 0 || !(tau > 0.f) || !w2 || !b2 || !decay)) return WLLM_BAD_SIZE;
-    if ((in_dtype != WLLM_BF16 && in_dtype != WLLM_F32) || (a_off >= 0 && w_dtype != WLLM_BF16 && w_dtype != WLLM_F32))
-        return WLLM_BAD_DTYPE;
-#define PREP2(TT, M) wllm_launch(linattn_prepare_kernel<TT, M>, dim3((n + TT - 1) / TT, H), 128, 0, stream, fused, \
-        in_dtype, row_stride, parts, (size_t)part_stride, q_off, k_off, v_off, a_off, n, H, D, V, rank, positions, \
-        inv_freq, rot_dim, q_scale, k_scale, w2, b2, w_dtype, a_off >= 0 ? 1.0f / tau : 0.f, q, k, v, decay)
-#define PREP(TT) (parts > 1 ? PREP2(TT, true) : PREP2(TT, false))
-    if ((long long)n * H >= 2048) return PREP(8);
-    return PREP(1);
-#undef PREP
-#undef PREP2
+    if (q == nullptr) return WLLM_BAD_SIZE;
+    return wllm_linattn_prepare_form(fused, in_dtype, row_stride, parts, part_stride, q_off, k_off, v_off, a_off, n, H, D, V, rank, positions,
+                                     inv_freq, rot_dim, q_scale, k_scale, w2, b2, w_dtype, tau, q, k, v, decay, 0, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -209,13 +227,16 @@ __device__ __forceinline__ void la_cp16(float* smem_dst, const float* src) {    
 // a time, and with two columns a lane every such read feeds eight multiply-adds; one column a lane and one channel
 // a read left the kernel waiting for shared memory (a read a multiply-add).
 // FULL: every warp holds LA_CPT channels (the head's key size is a multiple of 16): the loops carry no guards.
-template <bool PER_CHANNEL, int MODE, bool FULL>
+// BONUS: the output is S_(t-1)^T q + (q . (u k)) v, taken channel by channel in front of the update.
+// q, k and v are rows `q_stride`, `k_stride`, `v_stride` elements apart.
+template <bool PER_CHANNEL, int MODE, bool FULL, bool BONUS>
 __global__ void __launch_bounds__(512)
 linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v,
                     const float* __restrict__ decay, const float* __restrict__ head_decay, float* __restrict__ state,
                     float* __restrict__ out, const int* __restrict__ req_q_start, const int* __restrict__ req_q_len,
                     const int* __restrict__ req_slot, int H, int D, int V, int cpt, int seg_len, int max_seg,
-                    float* __restrict__ seg_state, float* __restrict__ seg_decay) {
+                    float* __restrict__ seg_state, float* __restrict__ seg_decay, size_t q_stride, size_t k_stride, size_t v_stride,
+                    const float* __restrict__ bonus) {
     extern __shared__ __align__(16) float la_smem[];
     pdl_begin();
     const int r = MODE == 0 ? blockIdx.z : blockIdx.z / max_seg, seg = MODE == 0 ? 0 : blockIdx.z % max_seg, h = blockIdx.y;
@@ -237,7 +258,7 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
     float* stage0 = la_smem;
     float* red = la_smem + 2 * LA_TT * per_token;             // [2][warps][LA_TT][64]
 
-    float S0[LA_CPT], S1[LA_CPT], P[LA_CPT];
+    float S0[LA_CPT], S1[LA_CPT], P[LA_CPT], U[LA_CPT];
     float* Sg = state + (((size_t)slot * H + h) * D) * V;
     // (a request of several segments reads every start from the scratch, the first one too: its last segment
     // may write the slot before its first one has started)
@@ -248,28 +269,32 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
         S0[i] = (ch && col0) ? St[(size_t)(c_lo + i) * V + j0] : 0.f;
         S1[i] = (ch && col1) ? St[(size_t)(c_lo + i) * V + j1] : 0.f;
         P[i] = 1.f;
+        U[i] = BONUS && (FULL || c_lo + i < c_hi) ? bonus[h * D + c_lo + i] : 0.f;
     }
     const float fixed = PER_CHANNEL ? 0.f : head_decay[h];
 
     // rows of whole 16-byte pieces (key sizes in steps of 16, value sizes in steps of 4, aligned buffers): a warp a token,
     // a lane a piece of q, k and the decay, sixteen lanes a piece of v; no division, a quarter of the copies
     const bool pieces = FULL && (V & 3) == 0 &&
-        ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (PER_CHANNEL ? (uintptr_t)decay : 0)) & 15) == 0);
+        ((((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (PER_CHANNEL ? (uintptr_t)decay : 0)) & 15) == 0) &&
+        ((q_stride | k_stride | v_stride) & 3) == 0;
     auto load_tile = [&](int tile, int stage) {
         float* dst = stage0 + (size_t)stage * LA_TT * per_token;
         const int first = t0 + tile * LA_TT, count = min(LA_TT, q_len - tile * LA_TT);
         if (pieces) {
             for (int tt = warp; tt < count; tt += warps) {
                 const size_t at = ((size_t)(first + tt) * H + h) * D;
+                const float* qrow = q + (size_t)(first + tt) * q_stride + (size_t)h * D;
+                const float* krow = k + (size_t)(first + tt) * k_stride + (size_t)h * D;
                 float* d = dst + tt * per_token;
                 for (int c = 4 * lane; c < D; c += 128) {
-                    la_cp16(d + c, q + at + c);
-                    la_cp16(d + Dp + c, k + at + c);
+                    la_cp16(d + c, qrow + c);
+                    la_cp16(d + Dp + c, krow + c);
                     if (PER_CHANNEL) la_cp16(d + 2 * Dp + c, decay + at + c);
                 }
                 if (lane < LA_COLS / 4) {
                     const int cc = blockIdx.x * LA_COLS + 4 * lane;
-                    const float* vrow = v + ((size_t)(first + tt) * H + h) * V;
+                    const float* vrow = v + (size_t)(first + tt) * v_stride + (size_t)h * V;
                     if (cc + 3 < V) la_cp16(d + NA * Dp + 4 * lane, vrow + cc);
                     else
                         for (int e = 0; e < 4; ++e) la_cp4(d + NA * Dp + 4 * lane + e, vrow + min(cc + e, V - 1));
@@ -282,14 +307,14 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
             const int tt = idx / D, c = idx - tt * D;
             const size_t at = ((size_t)(first + tt) * H + h) * D + c;
             float* d = dst + tt * per_token + c;
-            la_cp4(d, q + at);
-            la_cp4(d + Dp, k + at);
+            la_cp4(d, q + (size_t)(first + tt) * q_stride + (size_t)h * D + c);
+            la_cp4(d + Dp, k + (size_t)(first + tt) * k_stride + (size_t)h * D + c);
             if (PER_CHANNEL) la_cp4(d + 2 * Dp, decay + at);
         }
         for (int idx = threadIdx.x; idx < count * LA_COLS; idx += blockDim.x) {
             const int tt = idx / LA_COLS, cc = idx % LA_COLS;
             la_cp4(dst + tt * per_token + NA * Dp + cc,
-                   v + ((size_t)(first + tt) * H + h) * V + min(blockIdx.x * LA_COLS + cc, V - 1));
+                   v + (size_t)(first + tt) * v_stride + (size_t)h * V + min(blockIdx.x * LA_COLS + cc, V - 1));
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -326,10 +351,15 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
 #pragma unroll
                         for (int e = 0; e < 4; ++e) {
                             if (FULL || c_lo + i4 + e < c_hi) {   // (the last channels of a head whose size is no multiple of 4)
+                                if (BONUS && MODE != 1) {
+                                    const float uk = U[i4 + e] * ke[e];
+                                    p0[tt] = fmaf(fmaf(uk, v0, S0[i4 + e]), qe[e], p0[tt]);
+                                    p1[tt] = fmaf(fmaf(uk, v1, S1[i4 + e]), qe[e], p1[tt]);
+                                }
                                 S0[i4 + e] = fmaf(ae[e], S0[i4 + e], ke[e] * v0);
                                 S1[i4 + e] = fmaf(ae[e], S1[i4 + e], ke[e] * v1);
                                 if (MODE == 1) P[i4 + e] *= ae[e];
-                                else {
+                                else if (!BONUS) {
                                     p0[tt] = fmaf(S0[i4 + e], qe[e], p0[tt]);
                                     p1[tt] = fmaf(S1[i4 + e], qe[e], p1[tt]);
                                 }
@@ -412,13 +442,17 @@ __global__ void linattn_combine_kernel(const float* __restrict__ state, const in
 // state: [slots, H, D, V].  Requests by start, length and state slot; a length of 0 or a slot of -1 is passed by.
 // seg_len > 0: portions longer than that are cut into segments that run side by side (at most max_seg a request, which
 // must cover the longest portion); seg_state holds requests * max_seg * H * D * V floats, seg_decay requests * max_seg * H * D.
-WLLM_API int wllm_linattn_scan(const float* q, const float* k, const float* v, const float* decay, const float* head_decay,
-                               float* state, float* out, const int* req_q_start, const int* req_q_len, const int* req_slot,
-                               int requests, int H, int D, int V, int seg_len, int max_seg, float* seg_state, float* seg_decay,
-                               cudaStream_t stream) {
+// q_stride, k_stride, v_stride: elements between two tokens' rows (H * D, H * D and H * V where the rows lie one behind the other).
+// bonus [H, D] (null: none): time mixing, see above; with a decay per key channel.
+WLLM_API int wllm_linattn_scan_rows(const float* q, const float* k, const float* v, long long q_stride, long long k_stride,
+                                    long long v_stride, const float* decay, const float* head_decay, const float* bonus, float* state,
+                                    float* out, const int* req_q_start, const int* req_q_len, const int* req_slot, int requests, int H,
+                                    int D, int V, int seg_len, int max_seg, float* seg_state, float* seg_decay, cudaStream_t stream) {
     if (requests <= 0) return WLLM_OK;
     if (H <= 0 || H > 65535 || requests > 65535 || D <= 0 || D > 16 * LA_CPT || V <= 0) return WLLM_BAD_SIZE;
     if (!decay && !head_decay) return WLLM_BAD_SIZE;
+    if (bonus && !decay) return WLLM_BAD_SIZE;
+    if (q_stride < (long long)H * D || k_stride < (long long)H * D || v_stride < (long long)H * V) return WLLM_BAD_SIZE;
     const bool cut = seg_len > 0 && max_seg > 1;
     if (cut && (!seg_state || !seg_decay || (long long)requests * max_seg > 65535)) return WLLM_BAD_SIZE;
     const int most = (D + LA_CPT - 1) / LA_CPT;
@@ -430,29 +464,41 @@ WLLM_API int wllm_linattn_scan(const float* q, const float* k, const float* v, c
     static bool raised = false;
     if (!raised) {
         cudaError_t e = cudaSuccess;
-#define RAISE(PC, M) if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_scan_kernel<PC, M, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); \
-        if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_scan_kernel<PC, M, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)
-        RAISE(true, 0); RAISE(true, 1); RAISE(true, 2); RAISE(false, 0); RAISE(false, 1); RAISE(false, 2);
+#define RAISE(PC, M, B) if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_scan_kernel<PC, M, true, B>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); \
+        if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_scan_kernel<PC, M, false, B>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)
+        RAISE(true, 0, false); RAISE(true, 1, false); RAISE(true, 2, false); RAISE(false, 0, false); RAISE(false, 1, false); RAISE(false, 2, false);
+        RAISE(true, 0, true); RAISE(true, 2, true);
 #undef RAISE
         if (e != cudaSuccess) return 1000 + (int)e;
         raised = true;
     }
-#define SCAN2(PC, MODE, F, GRID) wllm_launch(linattn_scan_kernel<PC, MODE, F>, GRID, warps * 32, smem, stream, q, k, v, decay, head_decay, \
-        state, out, req_q_start, req_q_len, req_slot, H, D, V, cpt, seg_len, max_seg, seg_state, seg_decay)
-#define SCAN(PC, MODE, GRID) (full ? SCAN2(PC, MODE, true, GRID) : SCAN2(PC, MODE, false, GRID))
+#define SCAN2(PC, MODE, F, B, GRID) wllm_launch(linattn_scan_kernel<PC, MODE, F, B>, GRID, warps * 32, smem, stream, q, k, v, decay, head_decay, \
+        state, out, req_q_start, req_q_len, req_slot, H, D, V, cpt, seg_len, max_seg, seg_state, seg_decay, (size_t)q_stride, (size_t)k_stride, \
+        (size_t)v_stride, bonus)
+#define SCAN1(PC, MODE, B, GRID) (full ? SCAN2(PC, MODE, true, B, GRID) : SCAN2(PC, MODE, false, B, GRID))
+#define SCAN(MODE, GRID) (bonus ? SCAN1(true, MODE, true, GRID) : decay ? SCAN1(true, MODE, false, GRID) : SCAN1(false, MODE, false, GRID))
     if (!cut) {
         const dim3 grid(vtiles, H, requests);
-        return decay ? SCAN(true, 0, grid) : SCAN(false, 0, grid);
+        return SCAN(0, grid);
     }
     const dim3 grid(vtiles, H, requests * max_seg);
-    int st = decay ? SCAN(true, 1, grid) : SCAN(false, 1, grid);
+    int st = decay ? SCAN1(true, 1, false, grid) : SCAN1(false, 1, false, grid);      // (no outputs yet: the bonus does not matter)
     if (st != WLLM_OK) return st;
     st = wllm_launch(linattn_combine_kernel, dim3((D * V + 255) / 256, H, requests), 256, 0, stream, (const float*)state,
                      req_q_len, req_slot, H, D, V, seg_len, max_seg, seg_state, (const float*)seg_decay);
     if (st != WLLM_OK) return st;
-    return decay ? SCAN(true, 2, grid) : SCAN(false, 2, grid);
+    return SCAN(2, grid);
 #undef SCAN
+#undef SCAN1
 #undef SCAN2
+}
+
+WLLM_API int wllm_linattn_scan(const float* q, const float* k, const float* v, const float* decay, const float* head_decay,
+                               float* state, float* out, const int* req_q_start, const int* req_q_len, const int* req_slot,
+                               int requests, int H, int D, int V, int seg_len, int max_seg, float* seg_state, float* seg_decay,
+                               cudaStream_t stream) {
+    return wllm_linattn_scan_rows(q, k, v, (long long)H * D, (long long)H * D, (long long)H * V, decay, head_decay, nullptr, state, out,
+                                  req_q_start, req_q_len, req_slot, requests, H, D, V, seg_len, max_seg, seg_state, seg_decay, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -461,7 +507,7 @@ WLLM_API int wllm_linattn_scan(const float* q, const float* k, const float* v, c
 template <typename TO, bool MULTI>
 __global__ void head_gate_norm_kernel(const float* __restrict__ o, const void* __restrict__ fused, int in_dtype, int row_stride,
                                       int parts, size_t part_stride, int g_off, const void* __restrict__ w, int w_dtype,
-                                      float eps, TO* __restrict__ out, int H, int V) {
+                                      float eps, TO* __restrict__ out, int H, int V, int w_head_stride, size_t out_stride, float factor) {
     pdl_begin();
     const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x;
     const float* orow = o + ((size_t)t * H + h) * V;
@@ -473,22 +519,30 @@ __global__ void head_gate_norm_kernel(const float* __restrict__ o, const void* _
     for (int c = lane; c < V; c += 32) {
         const float g = la_in<MULTI>(fused, in_dtype, parts, part_stride, grow + c);
         float y = orow[c] * inv;
-        if (w) y *= la_any(w, w_dtype, c);
-        out[((size_t)t * H + h) * V + c] = from_f32<TO>(y * (g / (1.0f + expf(-g))));
+        if (w) y *= la_any(w, w_dtype, (size_t)h * w_head_stride + c);
+        out[(size_t)t * out_stride + (size_t)h * V + c] = from_f32<TO>(y * (g / (1.0f + expf(-g))) * factor);
     }
 }
 
-// out[n, H*V] = o / sqrt(mean_V(o^2) + eps) * w[V] (w may be null) * silu(g), g = fused[:, g_off + h*V + c]
-WLLM_API int wllm_head_gate_norm(const float* o, const void* fused, int in_dtype, int row_stride, int parts,
-                                 long long part_stride, int g_off, const void* w, int w_dtype, float eps, void* out,
-                                 int out_dtype, int n, int H, int V, cudaStream_t stream) {
+// out[n, H*V] = o / sqrt(mean_V(o^2) + eps) * w[V] (w may be null) * silu(g) * factor, g = fused[:, g_off + h*V + c]; per_head: w is
+// [H*V], a gain of the whole row; out's rows are out_stride elements apart
+WLLM_API int wllm_head_gate_norm_rows(const float* o, const void* fused, int in_dtype, int row_stride, int parts,
+                                      long long part_stride, int g_off, const void* w, int w_dtype, int per_head, float eps, void* out,
+                                      int out_dtype, int out_stride, float factor, int n, int H, int V, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
-    if (H <= 0 || H > 65535 || V <= 0 || parts < 1) return WLLM_BAD_SIZE;
+    if (H <= 0 || H > 65535 || V <= 0 || parts < 1 || out_stride < H * V) return WLLM_BAD_SIZE;
     if ((in_dtype != WLLM_BF16 && in_dtype != WLLM_F32) || (w && w_dtype != WLLM_BF16 && w_dtype != WLLM_F32)) return WLLM_BAD_DTYPE;
 #define GATE(TO, M) wllm_launch(head_gate_norm_kernel<TO, M>, dim3(n, H), 32, 0, stream, o, fused, in_dtype, row_stride, parts, \
-        (size_t)part_stride, g_off, w, w_dtype, eps, (TO*)out, H, V)
+        (size_t)part_stride, g_off, w, w_dtype, eps, (TO*)out, H, V, per_head ? V : 0, (size_t)out_stride, factor)
     if (out_dtype == WLLM_BF16) return parts > 1 ? GATE(bf16, true) : GATE(bf16, false);
     if (out_dtype == WLLM_F32) return parts > 1 ? GATE(float, true) : GATE(float, false);
 #undef GATE
     return WLLM_BAD_DTYPE;
+}
+
+WLLM_API int wllm_head_gate_norm(const float* o, const void* fused, int in_dtype, int row_stride, int parts,
+                                 long long part_stride, int g_off, const void* w, int w_dtype, float eps, void* out,
+                                 int out_dtype, int n, int H, int V, cudaStream_t stream) {
+    return wllm_head_gate_norm_rows(o, fused, in_dtype, row_stride, parts, part_stride, g_off, w, w_dtype, 0, eps, out, out_dtype, H * V, 1.0f,
+                                    n, H, V, stream);
 }

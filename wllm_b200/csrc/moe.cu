@@ -17,6 +17,10 @@
 //            tokens' rows copied into sorted order (moe_gather) and the table of row tiles that the plan writes.
 //   combine  out[token] = sum over the token's ranks, in rank order, of weight * y[place] (+ gate * shared unit).
 //
+// A router may add a correction per expert to the scores for the choice alone, divide the chosen scores by their sum
+// (plus a small number), and end with identity experts: the last ones of its list, without matrices, whose output is the
+// token's row itself.  Their pairs are sorted behind all others, no product touches them, and the combine reads the row.
+//
 // Two more forms.  Scores: softmax over all experts, or (score_mode 1) sigmoid(z) expert by expert, not normalised (without
 // groups the experts are then chosen by z itself: the same order, and no ties where large logits all round to a score of 1).  Unit
 // (MODE 2): an expert without a gate, down(relu(up (s a))^2), whose input is multiplied by the pair's score s: the up product
@@ -33,11 +37,12 @@ template <typename T>
 __global__ void __launch_bounds__(1024)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ w_gate,
                  int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate_out, int n, int H, int E, int top,
-                 int groups, int groups_kept, int tpb, int score_mode) {
-    extern __shared__ float route_smem[];          // [tpb][H] the tokens' rows, [tpb][E] scores, [tpb][groups] group scores
+                 int groups, int groups_kept, int tpb, int score_mode, const float* __restrict__ correction, float renorm_eps) {
+    extern __shared__ float route_smem[];          // [tpb][H] the tokens' rows, [tpb][E] scores, [tpb][groups] group scores, [tpb][E] corrected scores
     float* hs_all = route_smem;
     float* sc_all = hs_all + (size_t)tpb * H;
     float* gs_all = sc_all + (size_t)tpb * E;
+    float* ch_all = gs_all + (size_t)tpb * groups;
     pdl_begin();
     const int t0 = blockIdx.x * tpb, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
     const int here = min(tpb, n - t0);
@@ -85,7 +90,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
         const int t = t0 + j;
         float* sc = sc_all + (size_t)j * E;
         float* gs = gs_all + (size_t)j * groups;
-        if (score_mode == 1 && groups == 1) {
+        if (score_mode == 1 && groups == 1 && correction == nullptr && renorm_eps < 0.f) {
             // sigmoid scores without groups: the choice is made on the logits themselves (the sigmoid keeps their order, but
             // large logits all round to a score of 1 and would tie); the weights are the chosen logits' sigmoids
             for (int k = 0; k < top; ++k) {
@@ -117,15 +122,21 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
             for (int e = lane; e < E; e += 32) sc[e] *= inv;
         }
         __syncwarp();
-        const int per = E / groups;
-        for (int g = lane; g < groups; g += 32) {
-            float best = -INFINITY;
-            for (int i = 0; i < per; ++i) best = fmaxf(best, sc[g * per + i]);
-            gs[g] = best;
+        float* ch = sc;                             // what the choice is made on
+        if (correction != nullptr) {
+            ch = ch_all + (size_t)j * E;
+            for (int e = lane; e < E; e += 32) ch[e] = sc[e] + correction[e];
+            __syncwarp();
         }
-        __syncwarp();
+        const int per = E / groups;
         // the groups that stay: groups_kept times the best one left (ties: the lower index); the others' experts leave
         if (groups_kept < groups) {
+            for (int g = lane; g < groups; g += 32) {
+                float best = -INFINITY;
+                for (int i = 0; i < per; ++i) best = fmaxf(best, ch[g * per + i]);
+                gs[g] = best;
+            }
+            __syncwarp();
             for (int pick = 0; pick < groups_kept; ++pick) {
                 float best = -INFINITY; int at = 0x7fffffff;
                 for (int g = lane; g < groups; g += 32) { const float v = gs[g]; if (v > best) { best = v; at = g; } }
@@ -133,22 +144,30 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
                     const float ob = __shfl_xor_sync(0xffffffffu, best, o); const int oa = __shfl_xor_sync(0xffffffffu, at, o);
                     if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
                 }
-                if (lane == 0) gs[at] = -2.0f;              // marked as kept (scores lie in [0, 1])
+                if (lane == 0) gs[min(at, groups - 1)] = -INFINITY;              // marked as kept
                 __syncwarp();
             }
-            for (int e = lane; e < E; e += 32) if (gs[e / per] != -2.0f) sc[e] = -1.0f;
+            for (int e = lane; e < E; e += 32) if (gs[e / per] != -INFINITY) ch[e] = -INFINITY;
             __syncwarp();
         }
+        float total = 0.f;
         for (int k = 0; k < top; ++k) {
             float best = -INFINITY; int at = 0x7fffffff;
-            for (int e = lane; e < E; e += 32) { const float v = sc[e]; if (v > best) { best = v; at = e; } }
+            for (int e = lane; e < E; e += 32) { const float v = ch[e]; if (v > best) { best = v; at = e; } }
             for (int o = 16; o > 0; o >>= 1) {
                 const float ob = __shfl_xor_sync(0xffffffffu, best, o); const int oa = __shfl_xor_sync(0xffffffffu, at, o);
                 if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
             }
-            if (lane == 0) { chosen[(size_t)t * top + k] = at; weights[(size_t)t * top + k] = best; sc[at] = -3.0f; }
+            at = min(at, E - 1);                        // (scores that are no numbers choose nothing; the index stays inside)
+            if (lane == 0) {
+                const float weight = sc[at];
+                total += weight;
+                chosen[(size_t)t * top + k] = at; weights[(size_t)t * top + k] = weight; ch[at] = -INFINITY;
+            }
             __syncwarp();
         }
+        if (renorm_eps >= 0.f && lane == 0)
+            for (int k = 0; k < top; ++k) weights[(size_t)t * top + k] = weights[(size_t)t * top + k] / (total + renorm_eps);
     }
 }
 
@@ -176,11 +195,12 @@ __global__ void __launch_bounds__(128) moe_count_kernel(const int* __restrict__ 
 // order fill the sorted rows from offset[e]: sorted[r] = pair, place[pair] = r.  The warp of (expert, segment) places its
 // segment's pairs behind those of the segments before it.
 // With `tiles` (null: none): the table of row tiles of `tile_rows` rows of one expert each, for the products that walk it:
-// tiles[0] = their number, then (expert, first sorted row, rows) a tile, expert by expert.
+// tiles[0] = their number, then (expert, first sorted row, rows) a tile, expert by expert, for the first `tile_experts` experts (the
+// others have no matrices).
 __global__ void __launch_bounds__(128) moe_place_kernel(const int* __restrict__ chosen, int pairs, int E, int segs, int seg_len,
                                                         const int* __restrict__ partial, int* __restrict__ count,
                                                         int* __restrict__ offset, int* __restrict__ sorted, int* __restrict__ place,
-                                                        int* __restrict__ tiles, int tile_rows) {
+                                                        int* __restrict__ tiles, int tile_rows, int tile_experts) {
     pdl_begin();
     const int w = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (w >= E * segs) return;
@@ -208,13 +228,13 @@ __global__ void __launch_bounds__(128) moe_place_kernel(const int* __restrict__ 
             offset[e] = before;
             if (e == E - 1) offset[E] = before + mine_total;
         }
-        if (tiles) {
+        if (tiles && e < tile_experts) {
             const int n_tiles = (mine_total + tile_rows - 1) / tile_rows;
             for (int t = lane; t < n_tiles; t += 32) {
                 int* entry = tiles + 1 + 3 * (tiles_before + t);
                 entry[0] = e; entry[1] = before + t * tile_rows; entry[2] = min(tile_rows, mine_total - t * tile_rows);
             }
-            if (e == E - 1 && lane == 0) tiles[0] = tiles_before + n_tiles;
+            if (e == tile_experts - 1 && lane == 0) tiles[0] = tiles_before + n_tiles;
         }
     }
     int at = before + mine_before;
@@ -490,6 +510,11 @@ moe_grouped_mma_kernel(const bf16* __restrict__ a, int a_stride, const bf16* __r
         }
 }
 
+__device__ __forceinline__ float moe_row_at(const void* p, int dtype, size_t i) {
+    return dtype == WLLM_BF16 ? __bfloat162float(reinterpret_cast<const bf16*>(p)[i]) : reinterpret_cast<const float*>(p)[i];
+}
+
+// chosen (null: no identity experts): ranks whose expert is real_experts or above take the token's own row of x instead of y.
 // out[t][c] = sum_k weights[t][k] * y[place[t top + k]][c]  (+ gate[t] * shared[t][c], shared a tensor of TS or `parts`
 // 32-bit partial sums added in order first)
 // Many rows: a CTA of a few warps a token, one load after the other a thread (other CTAs hide the wait).
@@ -497,14 +522,17 @@ template <typename TS>
 __global__ void __launch_bounds__(256)
 moe_combine_rows_kernel(const float* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weights, int top,
                         const TS* __restrict__ shared, int parts, size_t part_stride, const float* __restrict__ gate,
-                        float* __restrict__ out, int H) {
+                        float* __restrict__ out, int H, const int* __restrict__ chosen, int real_experts,
+                        const void* __restrict__ x, int x_dtype) {
     pdl_begin();
     const int t = blockIdx.x;
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
         float v = 0.f;
         for (int k = 0; k < top; ++k) {
             // every product and sum rounded on its own, in both kernels: one result whichever serves the row
-            const float term = __fmul_rn(weights ? weights[(size_t)t * top + k] : 1.0f, y[(size_t)place[(size_t)t * top + k] * H + c]);
+            const bool own = chosen != nullptr && chosen[(size_t)t * top + k] >= real_experts;       // an identity expert: the token's row
+            const float term = __fmul_rn(weights ? weights[(size_t)t * top + k] : 1.0f,
+                                         own ? moe_row_at(x, x_dtype, (size_t)t * H + c) : y[(size_t)place[(size_t)t * top + k] * H + c]);
             v = k == 0 ? term : __fadd_rn(v, term);
         }
         if (shared != nullptr) {
@@ -513,7 +541,7 @@ moe_combine_rows_kernel(const float* __restrict__ y, const int* __restrict__ pla
                 const float part = to_f32(shared[(size_t)p * part_stride + (size_t)t * H + c]);
                 s = p == 0 ? part : __fadd_rn(s, part);
             }
-            v = fmaf(gate[t], s, v);
+            v = fmaf(gate ? gate[t] : 1.0f, s, v);
         }
         out[(size_t)t * H + c] = v;
     }
@@ -525,12 +553,17 @@ template <typename TS>
 __global__ void __launch_bounds__(1024)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place, const float* __restrict__ weights, int top,
                    const TS* __restrict__ shared, int parts, size_t part_stride, const float* __restrict__ gate,
-                   float* __restrict__ out, int H) {
+                   float* __restrict__ out, int H, const int* __restrict__ chosen, int real_experts,
+                        const void* __restrict__ x, int x_dtype) {
     __shared__ int s_place[64];
     __shared__ float s_weight[64];
     pdl_begin();
     const int t = blockIdx.x;
-    for (int k = threadIdx.x; k < min(top, 64); k += blockDim.x) { s_place[k] = place[(size_t)t * top + k]; s_weight[k] = weights ? weights[(size_t)t * top + k] : 1.0f; }
+    for (int k = threadIdx.x; k < min(top, 64); k += blockDim.x) {
+        const bool own = chosen != nullptr && chosen[(size_t)t * top + k] >= real_experts;           // an identity expert: the token's row
+        s_place[k] = own ? -1 : place[(size_t)t * top + k];
+        s_weight[k] = weights ? weights[(size_t)t * top + k] : 1.0f;
+    }
     __syncthreads();
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
         float v = 0.f;
@@ -541,9 +574,9 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place, c
                 const int k = k0 + u;
                 term[u] = 0.f;
                 if (k < top) {
-                    const int row = k < 64 ? s_place[k] : place[(size_t)t * top + k];
+                    const int row = k < 64 ? s_place[k] : (chosen != nullptr && chosen[(size_t)t * top + k] >= real_experts ? -1 : place[(size_t)t * top + k]);
                     const float wk = k < 64 ? s_weight[k] : (weights ? weights[(size_t)t * top + k] : 1.0f);
-                    term[u] = __fmul_rn(wk, y[(size_t)row * H + c]);
+                    term[u] = __fmul_rn(wk, row < 0 ? moe_row_at(x, x_dtype, (size_t)t * H + c) : y[(size_t)row * H + c]);
                 }
             }
 #pragma unroll
@@ -560,15 +593,16 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place, c
                 for (int u = 0; u < 16; ++u)
                     if (p0 + u < parts) s = (p0 + u == 0) ? part[u] : __fadd_rn(s, part[u]);
             }
-            v = fmaf(gate[t], s, v);
+            v = fmaf(gate ? gate[t] : 1.0f, s, v);
         }
         out[(size_t)t * H + c] = v;
     }
 }
 
-WLLM_API int wllm_moe_route(const void* h, int dtype, const float* w_router, const float* w_gate, int* chosen, float* weights,
-                            float* gate_out, int n, int H, int E, int top, int groups, int groups_kept, int score_mode,
-                            cudaStream_t stream) {
+// correction [E] (null: none): added to the scores for the choice; renorm_eps >= 0: the chosen scores over (their sum + renorm_eps)
+WLLM_API int wllm_moe_route_corrected(const void* h, int dtype, const float* w_router, const float* w_gate, int* chosen, float* weights,
+                                      float* gate_out, int n, int H, int E, int top, int groups, int groups_kept, int score_mode,
+                                      const float* correction, float renorm_eps, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
     if (score_mode != 0 && score_mode != 1) return WLLM_BAD_SIZE;
     if (H <= 0 || E <= 0 || E > MOE_MAX_EXPERTS || top < 1 || groups < 1 || E % groups != 0 || groups_kept < 1 ||
@@ -577,8 +611,9 @@ WLLM_API int wllm_moe_route(const void* h, int dtype, const float* w_router, con
     // tokens a CTA: eight once the tokens alone fill the device (each row of the router is then read once for eight), as
     // long as their rows fit in shared memory
     int tpb = n >= 1024 ? 8 : (n >= 296 ? 2 : 1);
-    while (tpb > 1 && (size_t)tpb * (H + E + groups) * sizeof(float) > 160 * 1024) tpb >>= 1;
-    const size_t smem = (size_t)tpb * (H + E + groups) * sizeof(float);
+    const size_t per_token = ((size_t)H + E + groups + (correction ? E : 0)) * sizeof(float);
+    while (tpb > 1 && tpb * per_token > 160 * 1024) tpb >>= 1;
+    const size_t smem = tpb * per_token;
     if (smem > 200 * 1024) return WLLM_BAD_SIZE;
     const int threads = 32 * (E + 1 < 4 ? 4 : (E + 1 > 32 ? 32 : E + 1));      // a warp an expert (and the shared gate), up to 32
 #define GO(T) do { \
@@ -587,7 +622,7 @@ WLLM_API int wllm_moe_route(const void* h, int dtype, const float* w_router, con
             if (er != cudaSuccess) return 1000 + (int)er; \
         } \
         return wllm_launch(moe_route_kernel<T>, (n + tpb - 1) / tpb, threads, smem, stream, (const T*)h, w_router, w_gate, chosen, weights, \
-                           gate_out, n, H, E, top, groups, groups_kept, tpb, score_mode); \
+                           gate_out, n, H, E, top, groups, groups_kept, tpb, score_mode, correction, renorm_eps); \
     } while (0)
     if (dtype == WLLM_BF16) GO(bf16);
     if (dtype == WLLM_F32) GO(float);
@@ -595,22 +630,35 @@ WLLM_API int wllm_moe_route(const void* h, int dtype, const float* w_router, con
     return WLLM_BAD_DTYPE;
 }
 
+WLLM_API int wllm_moe_route(const void* h, int dtype, const float* w_router, const float* w_gate, int* chosen, float* weights,
+                            float* gate_out, int n, int H, int E, int top, int groups, int groups_kept, int score_mode,
+                            cudaStream_t stream) {
+    return wllm_moe_route_corrected(h, dtype, w_router, w_gate, chosen, weights, gate_out, n, H, E, top, groups, groups_kept, score_mode,
+                                    nullptr, -1.0f, stream);
+}
+
 // count [E], offset [E + 1], sorted [pairs], place [pairs]
 constexpr int MOE_PLAN_SEGMENTS = 8;
 
 // tiles (null: none): 1 + 3 * (ceil(pairs / tile_rows) + E) ints, the table of row tiles (see moe_place_kernel).
 // scratch (null: none): MOE_PLAN_SEGMENTS * E ints; with it, long pair lists are scanned by that many warps an expert.
-WLLM_API int wllm_moe_plan_tiles(const int* chosen, int pairs, int E, int* count, int* offset, int* sorted, int* place, int* tiles,
-                                 int tile_rows, int* scratch, cudaStream_t stream) {
+// tile_experts: the experts that have matrices (the first of the E); the table lists their tiles.
+WLLM_API int wllm_moe_plan_real(const int* chosen, int pairs, int E, int* count, int* offset, int* sorted, int* place, int* tiles,
+                                int tile_rows, int* scratch, int tile_experts, cudaStream_t stream) {
     if (pairs <= 0) return WLLM_OK;
-    if (E <= 0 || E > MOE_MAX_EXPERTS || (tiles != nullptr && tile_rows < 1)) return WLLM_BAD_SIZE;
+    if (E <= 0 || E > MOE_MAX_EXPERTS || (tiles != nullptr && tile_rows < 1) || tile_experts < 1 || tile_experts > E) return WLLM_BAD_SIZE;
     const int segs = (scratch != nullptr && pairs >= 2048) ? MOE_PLAN_SEGMENTS : 1;
     const int seg_len = ((pairs + segs - 1) / segs + 127) / 128 * 128;
     int* partial = segs > 1 ? scratch : count;           // one segment: the partial counts are the counts
     const int st = wllm_launch(moe_count_kernel, (E * segs + 3) / 4, 128, 0, stream, chosen, pairs, E, segs, seg_len, partial);
     if (st != WLLM_OK) return st;
     return wllm_launch(moe_place_kernel, (E * segs + 3) / 4, 128, 0, stream, chosen, pairs, E, segs, seg_len, (const int*)partial, count,
-                       offset, sorted, place, tiles, tile_rows);
+                       offset, sorted, place, tiles, tile_rows, tile_experts);
+}
+
+WLLM_API int wllm_moe_plan_tiles(const int* chosen, int pairs, int E, int* count, int* offset, int* sorted, int* place, int* tiles,
+                                 int tile_rows, int* scratch, cudaStream_t stream) {
+    return wllm_moe_plan_real(chosen, pairs, E, count, offset, sorted, place, tiles, tile_rows, scratch, E, stream);
 }
 
 WLLM_API int wllm_moe_plan(const int* chosen, int pairs, int E, int* count, int* offset, int* sorted, int* place, cudaStream_t stream) {
@@ -694,18 +742,27 @@ WLLM_API int wllm_moe_grouped(const void* a, int a_stride, const void* w, void* 
     return wllm_moe_grouped_unit(a, a_stride, w, out, dtype, gated ? 1 : 0, pairs, N, K, offset, sorted, E, top, limit, slope, nullptr, stream);
 }
 
-WLLM_API int wllm_moe_combine(const float* y, const int* place, const float* weights, int top, const void* shared, int shared_dtype,
-                              int parts, long long part_stride, const float* gate, float* out, int n, int H, cudaStream_t stream) {
+// gate null: the shared unit joins as it is.  chosen (null: no identity experts) [n, top], real_experts, x [n, H]: see above.
+WLLM_API int wllm_moe_combine_own(const float* y, const int* place, const float* weights, int top, const void* shared, int shared_dtype,
+                                  int parts, long long part_stride, const float* gate, float* out, int n, int H, const int* chosen,
+                                  int real_experts, const void* x, int x_dtype, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
-    if (H <= 0 || top < 1 || parts < 1 || (shared != nullptr && gate == nullptr)) return WLLM_BAD_SIZE;
+    if (H <= 0 || top < 1 || parts < 1 || (chosen != nullptr && x == nullptr)) return WLLM_BAD_SIZE;
+    if (chosen != nullptr && x_dtype != WLLM_BF16 && x_dtype != WLLM_F32) return WLLM_BAD_DTYPE;
     int threads = H >= 1024 ? 256 : 128;
     if (n <= 64) threads = H >= 2048 ? 1024 : (H >= 1024 ? 512 : threads);      // few rows: a thread a column or two, every load in flight
     const bool few = n <= 64;
     if (shared == nullptr || shared_dtype == WLLM_F32)
         return wllm_launch(few ? moe_combine_kernel<float> : moe_combine_rows_kernel<float>, n, threads, 0, stream, y, place, weights, top,
-                           (const float*)shared, parts, (size_t)part_stride, gate, out, H);
+                           (const float*)shared, parts, (size_t)part_stride, gate, out, H, chosen, real_experts, x, x_dtype);
     if (shared_dtype == WLLM_BF16 && parts == 1)
         return wllm_launch(few ? moe_combine_kernel<bf16> : moe_combine_rows_kernel<bf16>, n, threads, 0, stream, y, place, weights, top,
-                           (const bf16*)shared, parts, (size_t)part_stride, gate, out, H);
+                           (const bf16*)shared, parts, (size_t)part_stride, gate, out, H, chosen, real_experts, x, x_dtype);
     return WLLM_BAD_DTYPE;
+}
+
+WLLM_API int wllm_moe_combine(const float* y, const int* place, const float* weights, int top, const void* shared, int shared_dtype,
+                              int parts, long long part_stride, const float* gate, float* out, int n, int H, cudaStream_t stream) {
+    if (shared != nullptr && gate == nullptr) return WLLM_BAD_SIZE;
+    return wllm_moe_combine_own(y, place, weights, top, shared, shared_dtype, parts, part_stride, gate, out, n, H, nullptr, 0, nullptr, WLLM_F32, stream);
 }

@@ -441,3 +441,147 @@ WLLM_API int wllm_sandwich_norm(float* resid, const void* a, int a_dtype, int a_
     return wllm_sandwich_norm_offset(resid, a, a_dtype, a_parts, a_stride, wa, b, b_dtype, b_parts, b_stride, wb, inner_eps, factor,
                                      wp, 0.f, center_p, eps_p, w, offset, center, eps, w_dtype, out, out_dtype, rows, n, H, stream);
 }
+
+// ---------------------------------------------------------------------------------------------------
+// Several branches join the residual at once, and one or two norms of the sum go out, in one kernel a row:
+//     r  += s_0 a_0 + s_1 a_1 + s_2 a_2                   (each a tensor or 32-bit slabs; the factors are plain numbers)
+//     out_j = r_g / sqrt(mean(r_g^2) + eps) * (offset + w_j)   for every of `groups` equal parts r_g of the row
+// (two outputs: a block whose two sublayers read norms of the same residual; groups = 1: the plain norm).  The row lies in
+// shared memory between the passes; a part's sum of squares is made of pieces of fixed places, a warp each, added in order.
+// With `rows` the residual is read at rows[i] and left as it is.  Without outputs the branches are added and that is all.
+// ---------------------------------------------------------------------------------------------------
+struct FoldTerm {
+    const void* p;
+    int dtype, parts;
+    size_t stride;
+    float factor;
+};
+struct FoldTerms {
+    FoldTerm t[3];
+    int count;
+};
+constexpr int FOLD_MAX_GROUPS = 1024;
+
+// elements c .. c + VEC - 1 of one term's row: part 0 + part 1 + ... in that order
+template <int VEC, bool MULTI>
+__device__ __forceinline__ void fold_load(const FoldTerm& f, size_t i, float (&v)[4]) {
+    v[0] = v[1] = v[2] = v[3] = 0.f;
+    if (VEC == 1) { v[0] = parts_at<MULTI>(f.p, f.dtype, f.parts, f.stride, i); return; }
+    if (f.dtype == WLLM_BF16) { load4(reinterpret_cast<const bf16*>(f.p) + i, v); return; }
+    const float* p = reinterpret_cast<const float*>(f.p) + i;
+    if (!MULTI || f.parts == 1) { load4(p, v); return; }
+    add_parts<float, 4>(v, p, f.parts, f.stride);
+}
+
+template <typename TO, int VEC, bool MULTI>
+__global__ void __launch_bounds__(512)
+fold_norm_kernel(float* __restrict__ resid, FoldTerms terms, const void* __restrict__ w1, const void* __restrict__ w2, int w_dtype,
+                 float offset, float eps, int groups, int pieces, TO* __restrict__ out1, TO* __restrict__ out2,
+                 const int* __restrict__ rows, int H) {
+    extern __shared__ __align__(16) float fold_s[];       // [H] the row, [groups * pieces] partial sums, [groups] scales
+    float* part_s = fold_s + ((H + 3) & ~3);
+    float* inv_s = part_s + groups * pieces;
+    pdl_begin();
+    const int i = blockIdx.x;
+    const size_t row0 = (size_t)(rows ? rows[i] : i) * H;
+    const bool write_back = terms.count > 0 && rows == nullptr;
+    for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+        float v[4] = {0.f, 0.f, 0.f, 0.f}, a[3][4];
+        if (VEC == 4) load4(resid + row0 + c, v); else v[0] = resid[row0 + c];
+#pragma unroll
+        for (int k = 0; k < 3; ++k)
+            if (k < terms.count) fold_load<VEC, MULTI>(terms.t[k], row0 + c, a[k]);
+#pragma unroll
+        for (int k = 0; k < 3; ++k)
+            if (k < terms.count) {
+#pragma unroll
+                for (int e = 0; e < VEC; ++e) v[e] = fmaf(terms.t[k].factor, a[k][e], v[e]);
+            }
+        if (write_back) {
+            if (VEC == 4) store4(resid + row0 + c, v); else resid[row0 + c] = v[0];
+        }
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) fold_s[c + e] = v[e];
+    }
+    if (out1 == nullptr) return;
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int size = H / groups, per = (size + pieces - 1) / pieces;
+    for (int p = warp; p < groups * pieces; p += warps) {
+        const int g = p / pieces, lo = (p % pieces) * per, hi = min(size, lo + per);
+        float ss = 0.f;
+        for (int c = lo + lane; c < hi; c += 32) { const float x = fold_s[g * size + c]; ss = fmaf(x, x, ss); }
+        ss = warp_sum(ss);
+        if (lane == 0) part_s[p] = ss;
+    }
+    __syncthreads();
+    for (int g = threadIdx.x; g < groups; g += blockDim.x) {
+        float ss = part_s[g * pieces];
+        for (int k = 1; k < pieces; ++k) ss += part_s[g * pieces + k];
+        inv_s[g] = 1.0f / sqrtf(ss / (float)size + eps);
+    }
+    __syncthreads();
+    for (int c = threadIdx.x * VEC; c < H; c += blockDim.x * VEC) {
+        float y[4], o[4];
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y[e] = fold_s[c + e] * inv_s[(c + e) / size];
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            TO* out = k ? out2 : out1;
+            if (out == nullptr) break;
+            const void* w = k ? w2 : w1;
+            float wv[4] = {0.f, 0.f, 0.f, 0.f};
+            if (VEC == 4) {
+                if (w_dtype == WLLM_BF16) load4(reinterpret_cast<const bf16*>(w) + c, wv);
+                else load4(reinterpret_cast<const float*>(w) + c, wv);
+            } else wv[0] = any_at(w, w_dtype, c);
+#pragma unroll
+            for (int e = 0; e < VEC; ++e) o[e] = y[e] * (offset + wv[e]);
+            if (VEC == 4) store4(out + (size_t)i * H + c, o); else out[(size_t)i * H + c] = from_f32<TO>(o[0]);
+        }
+    }
+}
+
+// terms: `count` branches (at most 3), given by pointer, element type, slabs, stride between slabs and factor; w1, w2 of one
+// element type; out2 (and w2) may be null, and out1 too (then only the addition happens).
+WLLM_API int wllm_fold_norm(float* resid, int count, const void* a0, int t0, int p0, long long s0, float f0, const void* a1, int t1,
+                            int p1, long long s1, float f1, const void* a2, int t2, int p2, long long s2, float f2, const void* w1,
+                            const void* w2, int w_dtype, float offset, float eps, int groups, void* out1, void* out2, int out_dtype,
+                            const int* rows, int n, int H, cudaStream_t stream) {
+    if (n <= 0) return WLLM_OK;
+    if (H <= 0 || H > 40 * 1024 || count < 0 || count > 3 || groups < 1 || groups > FOLD_MAX_GROUPS || H % groups != 0) return WLLM_BAD_SIZE;
+    if ((out1 != nullptr && w1 == nullptr) || (out2 != nullptr && (out1 == nullptr || w2 == nullptr))) return WLLM_BAD_SIZE;
+    FoldTerms terms = {{{a0, t0, p0, (size_t)s0, f0}, {a1, t1, p1, (size_t)s1, f1}, {a2, t2, p2, (size_t)s2, f2}}, count};
+    bool multi = false, vec = H % 4 == 0 && !(((uintptr_t)resid | (uintptr_t)w1 | (uintptr_t)w2 | (uintptr_t)out1 | (uintptr_t)out2) & 15);
+    for (int k = 0; k < count; ++k) {
+        const FoldTerm& f = terms.t[k];
+        if (f.p == nullptr || f.parts < 1) return WLLM_BAD_SIZE;
+        if ((f.dtype != WLLM_BF16 && f.dtype != WLLM_F32) || (f.parts > 1 && f.dtype != WLLM_F32)) return WLLM_BAD_DTYPE;
+        multi = multi || f.parts > 1;
+        vec = vec && !((uintptr_t)f.p & 15) && f.stride % 4 == 0;
+    }
+    if (out1 != nullptr && w_dtype != WLLM_BF16 && w_dtype != WLLM_F32) return WLLM_BAD_DTYPE;
+    const int per = vec ? 4 : 1;
+    const int threads = H / per >= 512 ? 512 : (H / per >= 256 ? 256 : 128), warps = threads / 32;
+    const int pieces = groups >= warps ? 1 : warps / groups;
+    const size_t smem = ((size_t)((H + 3) & ~3) + (size_t)groups * pieces + groups) * sizeof(float);
+#define FOLD2(TO, V, M) do { \
+        static bool raised = false; \
+        if (!raised && smem > 48 * 1024) { \
+            const cudaError_t e = cudaFuncSetAttribute(fold_norm_kernel<TO, V, M>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024); \
+            if (e != cudaSuccess) return 1000 + (int)e; \
+            raised = true; \
+        } \
+        return wllm_launch(fold_norm_kernel<TO, V, M>, n, threads, smem, stream, resid, terms, w1, w2, w_dtype, offset, eps, groups, pieces, \
+                           (TO*)out1, (TO*)out2, rows, H); \
+    } while (0)
+#define FOLD(TO) do { \
+        if (vec) { if (multi) FOLD2(TO, 4, true); else FOLD2(TO, 4, false); } \
+        else { if (multi) FOLD2(TO, 1, true); else FOLD2(TO, 1, false); } \
+    } while (0)
+    if (out_dtype == WLLM_BF16) FOLD(bf16);
+    if (out_dtype == WLLM_F32) FOLD(float);
+#undef FOLD
+#undef FOLD2
+    return WLLM_BAD_DTYPE;
+}

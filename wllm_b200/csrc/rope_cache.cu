@@ -12,7 +12,10 @@
 // slots the row holds query heads alone.
 // Value heads may have a size of their own (`vd`): the fused row is nq heads of hd, nkv heads of hd, nkv heads
 // of vd.  With `unit_norm` every rotated query and key head is divided by its root mean square,
-// y / sqrt(mean(y^2) + norm_eps), in 32-bit, before it is rounded and stored.
+// y / sqrt(mean(y^2) + norm_eps), in 32-bit, before it is rounded and stored.  Beside that (`wllm_rope_head_norm_kv_write`) query and
+// key heads may carry gains shared by the heads (in front of the turn: x / sqrt(mean(x^2) + eps) * gain, then turned), queries a
+// factor that grows with the position, 1 + coef ln(floor((position + 1) / every) + 1), and value heads may be divided by their
+// root mean square before they are cached.
 //
 // With row gains (`wllm_rope_row_norm_kv_write`) the query row and the key row of a token are normed as wholes, all heads at
 // once, in front of the turn: q <- q / sqrt(mean(q^2) + eps) * wq over the token's nq * hd query elements, the same for k.
@@ -87,6 +90,23 @@ __global__ void rope_kv_write_kernel(const TI* __restrict__ qkv, int row_stride,
     }
 }
 
+// What a head norm does beside the division (all off by default).  `count`, `v_count`: the elements that count for the means
+// (heads that are held in steps of 8 elements carry zeros behind them).
+struct HeadNorm {
+    const void* q_gain;      // [hd] or null; with gains the norm and the gain come in front of the turn
+    const void* k_gain;
+    int gain_dtype, count, v_count;
+    int norm_values;         // value heads are divided by their root mean square
+    float temp_coef;         // queries times 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1); temp_every 0: no factor
+    int temp_every;
+};
+__device__ __forceinline__ float gain_at(const void* p, int dtype, int i) {
+    return dtype == WLLM_BF16 ? __bfloat162float(reinterpret_cast<const bf16*>(p)[i]) : reinterpret_cast<const float*>(p)[i];
+}
+__device__ __forceinline__ float query_factor(const HeadNorm& hn, int position) {
+    return hn.temp_every > 0 ? 1.0f + hn.temp_coef * logf((float)((position + 1) / hn.temp_every + 1)) : 1.0f;
+}
+
 // Heads that are divided by their root mean square after the turn: a warp a head (grid (token, groups of heads)),
 // the head's elements in the lanes' registers between the turn and the scaling, the sum of squares by shuffles: no
 // barrier, no shared memory, and the same arithmetic for a head whatever the step's size.  Value heads are copied.
@@ -97,7 +117,7 @@ rope_unit_norm_kernel(const TI* __restrict__ qkv, int row_stride, int in_splits,
                       TO* __restrict__ q_out, int q_stride, const int* __restrict__ positions,
                       const int* __restrict__ slots, const float* __restrict__ inv_freq,
                       TO* __restrict__ k_pages, TO* __restrict__ v_pages, int nq, int nkv, int hd,
-                      int rot_dim, int page_size, int interleaved, int vd, float norm_eps) {
+                      int rot_dim, int page_size, int interleaved, int vd, float norm_eps, HeadNorm hn) {
     pdl_launch_dependents();
     const int t = blockIdx.x, lane = threadIdx.x & 31;
     const int h = blockIdx.y * 4 + (threadIdx.x >> 5);       // this warp's head
@@ -137,9 +157,25 @@ rope_unit_norm_kernel(const TI* __restrict__ qkv, int row_stride, int in_splits,
             return v;
         };
         if (value) {
-            for (int c = lane; c < vd; c += 32) dst[c] = from_f32<TO>(in(c));
+            if (!hn.norm_values) {
+                for (int c = lane; c < vd; c += 32) dst[c] = from_f32<TO>(in(c));
+                return;
+            }
+            float yv[16], sv = 0.f;
+#pragma unroll
+            for (int u = 0; u < 16; ++u) {
+                const int c = lane + 32 * u;
+                yv[u] = 0.f;
+                if (c < vd) { yv[u] = in(c); sv += yv[u] * yv[u]; }
+            }
+            const float inv_v = 1.0f / sqrtf(warp_sum(sv) / (float)hn.v_count + norm_eps);
+#pragma unroll
+            for (int u = 0; u < 16; ++u)
+                if (lane + 32 * u < vd) dst[lane + 32 * u] = from_f32<TO>(yv[u] * inv_v);
             return;
         }
+        const void* gain = h < nq ? hn.q_gain : hn.k_gain;
+        const float factor = h < nq ? query_factor(hn, positions[t]) : 1.0f;
         float ya[8], yb[8], yr[16];
         float ss = 0.f;
 #pragma unroll
@@ -148,18 +184,28 @@ rope_unit_norm_kernel(const TI* __restrict__ qkv, int row_stride, int in_splits,
             ya[u] = yb[u] = 0.f;
             if (j < half) {
                 const int ia = interleaved ? 2 * j : j, ib = interleaved ? 2 * j + 1 : j + half;
-                rotate_pair(in(ia), in(ib), sn[u], cs[u], ya[u], yb[u]);
-                ss += ya[u] * ya[u] + yb[u] * yb[u];
+                float xa = in(ia), xb = in(ib);
+                if (gain) {          // the turn keeps the norm, so the sum may be taken of the elements in front of it
+                    ss += xa * xa + xb * xb;
+                    xa *= gain_at(gain, hn.gain_dtype, ia);
+                    xb *= gain_at(gain, hn.gain_dtype, ib);
+                }
+                rotate_pair(xa, xb, sn[u], cs[u], ya[u], yb[u]);
+                if (!gain) ss += ya[u] * ya[u] + yb[u] * yb[u];
             }
         }
 #pragma unroll
         for (int u = 0; u < 16; ++u) {
             const int c = rot_dim + lane + 32 * u;
             yr[u] = 0.f;
-            if (c < hd) { yr[u] = in(c); ss += yr[u] * yr[u]; }
+            if (c < hd) {
+                yr[u] = in(c);
+                ss += yr[u] * yr[u];
+                if (gain) yr[u] *= gain_at(gain, hn.gain_dtype, c);
+            }
         }
         ss = warp_sum(ss);
-        const float inv = 1.0f / sqrtf(ss / (float)hd + norm_eps);
+        const float inv = (1.0f / sqrtf(ss / (float)hn.count + norm_eps)) * factor;
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
             const int j = lane + 32 * u;
@@ -185,7 +231,7 @@ __global__ void __launch_bounds__(128)
 rope_unit_norm_rows_kernel(const bf16* __restrict__ qkv, int row_stride, bf16* __restrict__ q_out, int q_stride,
                            const int* __restrict__ positions, const int* __restrict__ slots, const float* __restrict__ inv_freq,
                            bf16* __restrict__ k_pages, bf16* __restrict__ v_pages, int nq, int nkv, int hd, int rot_dim,
-                           int page_size, int vd, float norm_eps) {
+                           int page_size, int vd, float norm_eps, HeadNorm hn) {
     extern __shared__ float sc[];            // [half] sines, [half] cosines
     pdl_launch_dependents();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -198,10 +244,12 @@ rope_unit_norm_rows_kernel(const bf16* __restrict__ qkv, int row_stride, bf16* _
     const bf16* row = qkv + (size_t)t * row_stride;
     const int rotated = slot < 0 ? nq : nq + nkv;
     const int pair_items = half / 8, rest_items = (hd - rot_dim) / 8;       // at most 32 and 64
+    const float q_factor = query_factor(hn, positions[t]);
     for (int h = warp; h < rotated; h += 4) {
         const bf16* x = row + (size_t)h * hd;
         bf16* dst = h < nq ? q_out + (size_t)t * q_stride + (size_t)h * hd
                            : k_pages + (((size_t)(slot / page_size) * nkv + (h - nq)) * page_size + slot % page_size) * hd;
+        const void* gain = h < nq ? hn.q_gain : hn.k_gain;
         float ya[8], yb[8], yr[2][8];
         float ss = 0.f;
         if (lane < pair_items) {
@@ -211,8 +259,14 @@ rope_unit_norm_rows_kernel(const bf16* __restrict__ qkv, int row_stride, bf16* _
             const bf16* xb = reinterpret_cast<const bf16*>(&b);
 #pragma unroll
             for (int e = 0; e < 8; ++e) {
-                rotate_pair(to_f32(xa[e]), to_f32(xb[e]), sc[j + e], sc[half + j + e], ya[e], yb[e]);
-                ss += ya[e] * ya[e] + yb[e] * yb[e];
+                float fa = to_f32(xa[e]), fb = to_f32(xb[e]);
+                if (gain) {
+                    ss += fa * fa + fb * fb;
+                    fa *= gain_at(gain, hn.gain_dtype, j + e);
+                    fb *= gain_at(gain, hn.gain_dtype, j + half + e);
+                }
+                rotate_pair(fa, fb, sc[j + e], sc[half + j + e], ya[e], yb[e]);
+                if (!gain) ss += ya[e] * ya[e] + yb[e] * yb[e];
             }
         }
 #pragma unroll
@@ -222,11 +276,15 @@ rope_unit_norm_rows_kernel(const bf16* __restrict__ qkv, int row_stride, bf16* _
                 const uint4 r = *reinterpret_cast<const uint4*>(x + rot_dim + item * 8);
                 const bf16* xr = reinterpret_cast<const bf16*>(&r);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) { yr[u][e] = to_f32(xr[e]); ss += yr[u][e] * yr[u][e]; }
+                for (int e = 0; e < 8; ++e) {
+                    yr[u][e] = to_f32(xr[e]);
+                    ss += yr[u][e] * yr[u][e];
+                    if (gain) yr[u][e] *= gain_at(gain, hn.gain_dtype, rot_dim + item * 8 + e);
+                }
             }
         }
         ss = warp_sum(ss);
-        const float inv = 1.0f / sqrtf(ss / (float)hd + norm_eps);
+        const float inv = (1.0f / sqrtf(ss / (float)hn.count + norm_eps)) * (h < nq ? q_factor : 1.0f);
         if (lane < pair_items) {
             uint4 oa, ob;
             bf16* pa = reinterpret_cast<bf16*>(&oa);
@@ -250,6 +308,36 @@ rope_unit_norm_rows_kernel(const bf16* __restrict__ qkv, int row_stride, bf16* _
     }
     if (slot < 0) return;
     const int whole = vd / 8;
+    if (hn.norm_values) {          // a warp a value head
+        for (int kvh = warp; kvh < nkv; kvh += 4) {
+            const bf16* x = row + (size_t)(nq + nkv) * hd + (size_t)kvh * vd;
+            bf16* dst = v_pages + (((size_t)(slot / page_size) * nkv + kvh) * page_size + slot % page_size) * vd;
+            float y[2][8], ss = 0.f;
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int item = lane + 32 * u;
+                if (item < whole) {
+                    const uint4 r = *reinterpret_cast<const uint4*>(x + item * 8);
+                    const bf16* xr = reinterpret_cast<const bf16*>(&r);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) { y[u][e] = to_f32(xr[e]); ss += y[u][e] * y[u][e]; }
+                }
+            }
+            const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)hn.v_count + norm_eps);
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int item = lane + 32 * u;
+                if (item < whole) {
+                    uint4 o;
+                    bf16* po = reinterpret_cast<bf16*>(&o);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) po[e] = from_f32<bf16>(y[u][e] * inv);
+                    *reinterpret_cast<uint4*>(dst + item * 8) = o;
+                }
+            }
+        }
+        return;
+    }
     for (int item = threadIdx.x; item < nkv * whole; item += blockDim.x) {
         const int kvh = item / whole, c = (item % whole) * 8;
         bf16* dst = v_pages + (((size_t)(slot / page_size) * nkv + kvh) * page_size + slot % page_size) * vd;
@@ -343,9 +431,6 @@ __global__ void rope_kv_write_rows_kernel(const bf16* __restrict__ qkv, int row_
 // (partial sums added in slab order) go to shared memory with their sums of squares (block sums in a fixed order, so a
 // token's result does not depend on the step), then every thread turns pairs of the normed, gained elements.  The means
 // divide by q_count and k_count (heads that are held in steps of 8 elements carry zeros behind them, which count for nothing).
-__device__ __forceinline__ float gain_at(const void* p, int dtype, int i) {
-    return dtype == WLLM_BF16 ? __bfloat162float(reinterpret_cast<const bf16*>(p)[i]) : reinterpret_cast<const float*>(p)[i];
-}
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256)
 rope_row_norm_kernel(const TI* __restrict__ qkv, int row_stride, int in_splits, size_t in_split_stride,
@@ -572,6 +657,50 @@ WLLM_API int wllm_rope_row_norm_kv_write(const void* qkv, int in_dtype, int row_
     return WLLM_BAD_DTYPE;
 }
 
+// heads divided by their root mean square, with what `hn` asks for beside that
+static int launch_head_norm(const void* qkv, int in_dtype, int row_stride, int in_splits, long long in_split_stride, void* q_out,
+                            int out_dtype, int q_stride, const int* positions, const int* slots, const float* inv_freq, void* k_pages,
+                            void* v_pages, int n, int nq, int nkv, int hd, int rot_dim, int page_size, int interleaved, int vd,
+                            float norm_eps, HeadNorm hn, cudaStream_t stream) {
+    if (hd > 512) return WLLM_BAD_SIZE;
+    if (n >= 256 && !interleaved && in_dtype == WLLM_BF16 && out_dtype == WLLM_BF16 && in_splits == 1 && hd % 8 == 0 && vd % 8 == 0 &&
+        rot_dim % 16 == 0 && row_stride % 8 == 0 && q_stride % 8 == 0 && !((uintptr_t)qkv & 15) && !((uintptr_t)q_out & 15) &&
+        !((uintptr_t)k_pages & 15) && !((uintptr_t)v_pages & 15))
+        return wllm_launch(rope_unit_norm_rows_kernel, n, 128, (size_t)rot_dim * sizeof(float), stream, (const bf16*)qkv, row_stride,
+                           (bf16*)q_out, q_stride, positions, slots, inv_freq, (bf16*)k_pages, (bf16*)v_pages, nq, nkv, hd,
+                           rot_dim, page_size, vd, norm_eps, hn);
+    // four heads a CTA at every size.  A CTA a token whose warps walk every fourth head (angles worked out once a lane)
+    // was measured slower over a prompt: 2,048 tokens, 10 heads of 256: 76 us against 48
+    const dim3 ugrid(n, (nq + 2 * nkv + 3) / 4);
+#define UN(TI, TO) wllm_launch(rope_unit_norm_kernel<TI, TO>, ugrid, 128, 0, stream, (const TI*)qkv, row_stride, in_splits, \
+    (size_t)in_split_stride, (TO*)q_out, q_stride, positions, slots, inv_freq, (TO*)k_pages, (TO*)v_pages, nq, nkv, hd, \
+    rot_dim, page_size, interleaved, vd, norm_eps, hn)
+    if (in_dtype == WLLM_BF16 && out_dtype == WLLM_BF16) return UN(bf16, bf16);
+    if (in_dtype == WLLM_F32 && out_dtype == WLLM_BF16) return UN(float, bf16);
+    if (in_dtype == WLLM_F32 && out_dtype == WLLM_F32) return UN(float, float);
+#undef UN
+    return WLLM_BAD_DTYPE;
+}
+
+// q_gain, k_gain [hd] of one element type (both or neither); count, v_count: the elements of a head that count for the means;
+// norm_values: value heads are divided by their root mean square too; temp_every > 0: the queries' factor by position.
+WLLM_API int wllm_rope_head_norm_kv_write(const void* qkv, int in_dtype, int row_stride, int in_splits, long long in_split_stride,
+                                          void* q_out, int out_dtype, int q_stride, const int* positions, const int* slots,
+                                          const float* inv_freq, void* k_pages, void* v_pages, int n, int nq, int nkv, int hd,
+                                          int rot_dim, int page_size, int interleaved, int vd, float norm_eps, const void* q_gain,
+                                          const void* k_gain, int gain_dtype, int count, int v_count, int norm_values, float temp_coef,
+                                          int temp_every, cudaStream_t stream) {
+    if (n <= 0) return WLLM_OK;
+    if (hd <= 0 || vd <= 0 || vd > 512 || rot_dim < 0 || rot_dim > hd || (rot_dim & 1) || page_size <= 0 || nq <= 0 || nkv < 0 ||
+        (nkv == 0 && slots != nullptr) || in_splits < 1 || count <= 0 || count > hd || v_count <= 0 || v_count > vd || temp_every < 0)
+        return WLLM_BAD_SIZE;
+    if ((q_gain == nullptr) != (k_gain == nullptr)) return WLLM_BAD_SIZE;
+    if (gain_dtype != WLLM_BF16 && gain_dtype != WLLM_F32) return WLLM_BAD_DTYPE;
+    return launch_head_norm(qkv, in_dtype, row_stride, in_splits, in_split_stride, q_out, out_dtype, q_stride, positions, slots, inv_freq,
+                            k_pages, v_pages, n, nq, nkv, hd, rot_dim, page_size, interleaved, vd, norm_eps,
+                            HeadNorm{q_gain, k_gain, gain_dtype, count, v_count, norm_values, temp_coef, temp_every}, stream);
+}
+
 // vd: size of a value head (hd when they are the same); unit_norm: divide rotated q and k heads by their root mean square.
 WLLM_API int wllm_rope_kv_write_general(const void* qkv, int in_dtype, int row_stride, int in_splits, long long in_split_stride,
                                         void* q_out, int out_dtype, int q_stride, const int* positions, const int* slots,
@@ -587,26 +716,10 @@ WLLM_API int wllm_rope_kv_write_general(const void* qkv, int in_dtype, int row_s
         return wllm_launch(rope_kv_write_rows_kernel, n, 128, (size_t)rot_dim * sizeof(float), stream, (const bf16*)qkv, row_stride,
                            (bf16*)q_out, q_stride, positions, slots, inv_freq, (bf16*)k_pages, (bf16*)v_pages, nq, nkv, hd,
                            rot_dim, page_size, interleaved);
-    if (unit_norm) {
-        if (hd > 512) return WLLM_BAD_SIZE;
-        if (n >= 256 && !interleaved && in_dtype == WLLM_BF16 && out_dtype == WLLM_BF16 && in_splits == 1 && hd % 8 == 0 && vd % 8 == 0 &&
-            rot_dim % 16 == 0 && row_stride % 8 == 0 && q_stride % 8 == 0 && !((uintptr_t)qkv & 15) && !((uintptr_t)q_out & 15) &&
-            !((uintptr_t)k_pages & 15) && !((uintptr_t)v_pages & 15))
-            return wllm_launch(rope_unit_norm_rows_kernel, n, 128, (size_t)rot_dim * sizeof(float), stream, (const bf16*)qkv, row_stride,
-                               (bf16*)q_out, q_stride, positions, slots, inv_freq, (bf16*)k_pages, (bf16*)v_pages, nq, nkv, hd,
-                               rot_dim, page_size, vd, norm_eps);
-        // four heads a CTA at every size.  A CTA a token whose warps walk every fourth head (angles worked out once a lane)
-        // was measured slower over a prompt: 2,048 tokens, 10 heads of 256: 76 us against 48
-        const dim3 ugrid(n, (nq + 2 * nkv + 3) / 4);
-#define UN(TI, TO) wllm_launch(rope_unit_norm_kernel<TI, TO>, ugrid, 128, 0, stream, (const TI*)qkv, row_stride, in_splits, \
-        (size_t)in_split_stride, (TO*)q_out, q_stride, positions, slots, inv_freq, (TO*)k_pages, (TO*)v_pages, nq, nkv, hd, \
-        rot_dim, page_size, interleaved, vd, norm_eps)
-        if (in_dtype == WLLM_BF16 && out_dtype == WLLM_BF16) return UN(bf16, bf16);
-        if (in_dtype == WLLM_F32 && out_dtype == WLLM_BF16) return UN(float, bf16);
-        if (in_dtype == WLLM_F32 && out_dtype == WLLM_F32) return UN(float, float);
-#undef UN
-        return WLLM_BAD_DTYPE;
-    }
+    if (unit_norm)
+        return launch_head_norm(qkv, in_dtype, row_stride, in_splits, in_split_stride, q_out, out_dtype, q_stride, positions, slots, inv_freq,
+                                k_pages, v_pages, n, nq, nkv, hd, rot_dim, page_size, interleaved, vd, norm_eps,
+                                HeadNorm{nullptr, nullptr, WLLM_F32, hd, vd, 0, 0.f, 0}, stream);
     const int threads = hd >= 256 ? 128 : (hd >= 128 ? 64 : 32);
     // One CTA a token once the tokens alone fill the SMs several times over; below that a CTA a head, which keeps a
     // token's heads (and the partial sums each has to add) on different SMs: 256 tokens x 10 heads of 4 parts took

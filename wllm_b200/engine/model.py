@@ -112,9 +112,11 @@ class ComposedModel:
             part = todo.pop()
             todo.extend(part.parts() if hasattr(part, "parts") else [])     # a mixer made of mixers
             for t in vars(part).values():
-                if isinstance(t, torch.Tensor) and t.data_ptr() not in seen and t.dim() >= 1 and t.numel() > 1:
-                    seen.add(t.data_ptr())
-                    total += t.numel() * t.element_size()
+                if isinstance(t, torch.Tensor) and t.dim() >= 1 and t.numel() > 1:
+                    memory = t.untyped_storage()          # (several tensors may be views of one matrix)
+                    if memory.data_ptr() not in seen:
+                        seen.add(memory.data_ptr())
+                        total += memory.nbytes()
         return total
 
     # -- one step ------------------------------------------------------------------

@@ -14,6 +14,8 @@ FAMILIES = {
     "activation": [{}],
     "linear_attention": [{}],
     "delta_rule": [{}],
+    "rg_lru": [{}],
+    "token_blend": [{}],
     "latent_attention": [{}],
     "hyper_connections": [{}],
     "moe": [{}],

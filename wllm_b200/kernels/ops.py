@@ -200,6 +200,32 @@ def sandwich_norm(resid: torch.Tensor, a, out: torch.Tensor, post_weight: torch.
                                          _stream()), "sandwich_norm")
     return out
 
+
+def fold_norm(resid: torch.Tensor, terms, weights, eps: float, outs, groups: int = 1, offset: float = 0.0, rows=None) -> None:
+    """resid += sum of factor * branch over `terms` (at most three of (tensor [n, H] | float32 partial sums [S, n, H], S or 0, factor)),
+    then outs[j] = resid / sqrt(mean over each of `groups` equal parts of the row + eps) * (offset + weights[j]) for one or two
+    outputs (csrc/norm.cu); no outputs: the addition alone.  With `rows` the residual is read at those rows and left as it is."""
+    N, H = resid.shape
+    n = rows.shape[0] if rows is not None else N
+    _need_cuda(resid, rows, *[t[0] for t in terms], *weights, *outs)
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and len(terms) <= 3 and len(weights) == len(outs) <= 2
+    for w, o in zip(weights, outs):
+        assert w.shape == (H,) and w.is_contiguous() and w.dtype == weights[0].dtype
+        assert o.shape == (n, H) and o.is_contiguous() and o.dtype == outs[0].dtype
+    args = []
+    for k in range(3):
+        if k < len(terms):
+            t, parts, factor = terms[k]
+            args += [*_branch_args((t, parts), N, H), c_float(factor)]
+        else:
+            args += [_ptr(None), _F32, 1, ctypes.c_longlong(0), c_float(0.0)]
+    lib = load_family("norm")
+    _check(lib.wllm_fold_norm(_ptr(resid), len(terms), *args, _ptr(weights[0] if weights else None), _ptr(weights[1] if len(weights) > 1 else None),
+                              _dt(weights[0]) if weights else _F32, c_float(offset), c_float(eps), groups, _ptr(outs[0] if outs else None),
+                              _ptr(outs[1] if len(outs) > 1 else None), _dt(outs[0]) if outs else _F32,
+                              _ptr(_int32(rows, "rows") if rows is not None else None), n, H, _stream()), "fold_norm")
+
+
 def hyper_norm(src: torch.Tensor, dst: torch.Tensor, S: int, branch, prev_mix, prev_out, in_w, gain: torch.Tensor, eps: float,
                out: torch.Tensor, rows=None) -> torch.Tensor:
     """A residual of S streams and the norm in front of a sublayer (csrc/hyper_connections.cu).  `src`: the streams
@@ -301,6 +327,38 @@ def rope_row_norm_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, positions: to
                                            q_count, k_count, c_float(eps), _ptr(bias), _ptr(v_first if mix is not None else None),
                                            _ptr(blend if mix == "later" else None), {None: 0, "first": 1, "later": 2}[mix],
                                            _stream()), "rope_row_norm_kv_write")
+
+
+def rope_head_norm_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, positions: torch.Tensor, slots, inv_freq: torch.Tensor,
+                            k_pages, v_pages, nq: int, nkv: int, hd: int, rot_dim: int, page_size: int, eps: float,
+                            q_gain: torch.Tensor | None = None, k_gain: torch.Tensor | None = None, count: int | None = None,
+                            v_count: int | None = None, norm_values: bool = False, temp_coef: float = 0.0, temp_every: int = 0,
+                            in_splits: int = 0, pairing: str = "half", vd: int | None = None) -> None:
+    """As rope_kv_write with query and key heads divided by their root mean square (csrc/rope_cache.cu), and beside that: gains
+    [hd] shared by the heads (x / sqrt(mean(x^2) + eps) * gain, then turned); values divided by their root mean square per head
+    (`norm_values`); queries times 1 + temp_coef * ln(floor((position + 1) / temp_every) + 1) (temp_every 0: as they are).
+    `count`, `v_count`: the elements of a head that count for the means (heads held in steps of 8 carry zeros behind them)."""
+    if pairing not in ("half", "interleaved"):
+        raise KernelError(f"rotary pairing {pairing!r} not supported (half, interleaved)")
+    _need_cuda(qkv, q_out, positions, slots, inv_freq, k_pages, v_pages, q_gain, k_gain)
+    vd = hd if vd is None else vd
+    ptr, dt, row_stride, nparts, part_stride, n = _fused_args(qkv, in_splits)
+    assert qkv.shape[-1] >= (nq + nkv) * hd + nkv * vd and q_out.shape == (n, nq * hd) and q_out.stride(1) == 1
+    assert inv_freq.dtype == torch.float32 and inv_freq.numel() == rot_dim // 2 and inv_freq.is_contiguous()
+    assert (q_gain is None) == (k_gain is None)
+    for gain in (q_gain, k_gain):
+        assert gain is None or (gain.shape == (hd,) and gain.is_contiguous() and gain.dtype == q_gain.dtype)
+    if slots is not None:
+        assert k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.dtype == q_out.dtype == v_pages.dtype
+    lib = load_family("rope_cache")
+    _check(lib.wllm_rope_head_norm_kv_write(ptr, dt, row_stride, nparts, part_stride, _ptr(q_out), _dt(q_out), q_out.stride(0),
+                                            _ptr(_int32(positions, "positions")),
+                                            _ptr(_int32(slots, "slots") if slots is not None else None), _ptr(inv_freq),
+                                            _ptr(k_pages), _ptr(v_pages), n, nq, nkv, hd, rot_dim, page_size,
+                                            1 if pairing == "interleaved" else 0, vd, c_float(eps), _ptr(q_gain), _ptr(k_gain),
+                                            _dt(q_gain) if q_gain is not None else _F32, hd if count is None else count,
+                                            vd if v_count is None else v_count, 1 if norm_values else 0, c_float(temp_coef),
+                                            temp_every, _stream()), "rope_head_norm_kv_write")
 
 
 def latent_prepare(fused: torch.Tensor, parts: int, positions: torch.Tensor, slots, inv_freq: torch.Tensor, gain: torch.Tensor,
@@ -1011,6 +1069,23 @@ def linattn_prepare(fused, parts: int, q_off: int, k_off: int, v_off: int, heads
                                     c_float(tau), _ptr(q), _ptr(k), _ptr(v), _ptr(decay), _stream()), "linattn_prepare")
 
 
+def linattn_decay(low: torch.Tensor, parts: int, low_off: int, w2: torch.Tensor, b2: torch.Tensor, heads: int, dim: int,
+                  decay: torch.Tensor) -> torch.Tensor:
+    """The decay per key channel of time mixing, decay [n, heads*dim] = exp(-exp(w2 @ tanh(low) + b2)), where `low` are the
+    rank = w2.shape[1] columns of the projection `low` [n, W] (or partial sums [parts, n, W]) from `low_off`; 32-bit."""
+    _need_cuda(low, w2, b2, decay)
+    ptr, dt, row_stride, nparts, part_stride, n = _fused_args(low, parts)
+    assert w2.shape[0] == heads * dim and w2.is_contiguous() and b2.shape == (heads * dim,) and b2.dtype == w2.dtype and b2.is_contiguous()
+    assert decay.dtype == torch.float32 and decay.is_contiguous() and decay.shape == (n, heads * dim)
+    assert low_off + w2.shape[1] <= low.shape[-1]
+    lib = load_family("linear_attention")
+    null = _ptr(None)
+    _check(lib.wllm_linattn_prepare_form(ptr, dt, row_stride, nparts, part_stride, 0, 0, 0, low_off, n, heads, dim, dim, w2.shape[1], null,
+                                         null, 0, c_float(1.0), c_float(1.0), _ptr(w2), _ptr(b2), _dt(w2), c_float(1.0), null, null, null,
+                                         _ptr(decay), 1, _stream()), "linattn_decay")
+    return decay
+
+
 LINATTN_SEGMENT_FROM = 128     # portions of at least this many tokens may be cut into segments that run side by side
 LINATTN_MIN_SEGMENT = 32
 
@@ -1035,13 +1110,14 @@ def linattn_segment_plan(max_q_len: int, requests_multi: int, heads: int, vdim: 
 def linattn_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay, head_decay, state: torch.Tensor,
                  out: torch.Tensor, req_q_start: torch.Tensor, req_q_len: torch.Tensor, req_slot: torch.Tensor, heads: int,
                  dim: int, vdim: int, seg_len: int = 0, max_seg: int = 1, seg_state: torch.Tensor | None = None,
-                 seg_decay: torch.Tensor | None = None) -> torch.Tensor:
+                 seg_decay: torch.Tensor | None = None, bonus: torch.Tensor | None = None) -> torch.Tensor:
     """S <- diag(a_t) S + k_t v_t^T, o_t = S^T q_t over every request's tokens of the step, from and to the
     request's row of `state` [slots, heads, dim, vdim] (float32).  `decay` [n, heads*dim] per key channel, or None
     with `head_decay` [heads].  With seg_len > 0 and max_seg > 1 (linattn_segment_plan) portions are cut into segments
     of seg_len tokens that run side by side; seg_state (requests * max_seg * heads * dim * vdim floats) and seg_decay
-    (requests * max_seg * heads * dim) are their scratch."""
-    _need_cuda(q, k, v, decay, head_decay, state, out, req_q_start, req_q_len, req_slot, seg_state, seg_decay)
+    (requests * max_seg * heads * dim) are their scratch.  q, k and v may be columns of wider rows.  `bonus` [heads*dim]
+    (time mixing): o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t, the output in front of the update."""
+    _need_cuda(bonus, q, k, v, decay, head_decay, state, out, req_q_start, req_q_len, req_slot, seg_state, seg_decay)
     R = req_q_len.shape[0]
     if seg_len > 0 and max_seg > 1:
         assert seg_state.dtype == seg_decay.dtype == torch.float32 and seg_state.is_contiguous() and seg_decay.is_contiguous()
@@ -1049,15 +1125,20 @@ def linattn_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay, head_
         global launches
         launches += 2         # the segments' first walk and the kernel that chains their states
     n = q.shape[0]
-    assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (q, k, v, state, out))
+    assert all(t.dtype == torch.float32 for t in (q, k, v, state, out)) and all(t.stride(1) == 1 for t in (q, k, v))
+    assert state.is_contiguous() and out.is_contiguous()
     assert q.shape == k.shape == (n, heads * dim) and v.shape == out.shape == (n, heads * vdim)
     assert state.shape[1:] == (heads, dim, vdim)
+    assert bonus is None or (decay is not None and bonus.dtype == torch.float32 and bonus.shape == (heads * dim,) and bonus.is_contiguous())
     if decay is not None:
         assert decay.dtype == torch.float32 and decay.is_contiguous() and decay.shape == q.shape
     else:
         assert head_decay.dtype == torch.float32 and head_decay.shape == (heads,) and head_decay.is_contiguous()
     lib = load_family("linear_attention")
-    _check(lib.wllm_linattn_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(decay), _ptr(head_decay), _ptr(state), _ptr(out),
+    def stride(t, width):
+        return ctypes.c_longlong(t.stride(0) if n > 1 else max(t.stride(0), width))
+    _check(lib.wllm_linattn_scan_rows(_ptr(q), _ptr(k), _ptr(v), stride(q, heads * dim), stride(k, heads * dim), stride(v, heads * vdim),
+                                 _ptr(decay), _ptr(head_decay), _ptr(bonus), _ptr(state), _ptr(out),
                                  _ptr(_int32(req_q_start, "req_q_start")), _ptr(_int32(req_q_len, "req_q_len")),
                                  _ptr(_int32(req_slot, "req_slot")), R, heads, dim, vdim, seg_len, max_seg,
                                  _ptr(seg_state), _ptr(seg_decay), _stream()),
@@ -1066,17 +1147,20 @@ def linattn_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay, head_
 
 
 def head_gate_norm(o: torch.Tensor, fused, parts: int, gate_off: int, weight, eps: float, out: torch.Tensor, heads: int,
-                   vdim: int) -> torch.Tensor:
-    """out[n, heads*vdim] = o / sqrt(mean over a head of o^2 + eps) [* weight[vdim]] * silu(gate), the gate being the
-    columns of the fused projection row from `gate_off`; 32-bit inside, rounded once to out's element type."""
+                   vdim: int, factor: float = 1.0) -> torch.Tensor:
+    """out[n, heads*vdim] = o / sqrt(mean over a head of o^2 + eps) [* weight] * silu(gate) * factor, the gate being the
+    columns of the fused projection row from `gate_off`; 32-bit inside, rounded once to out's element type.  weight [vdim] is
+    shared by the heads, weight [heads*vdim] a gain of the whole row; `out` may be columns of wider rows."""
     _need_cuda(o, fused, weight, out)
     ptr, dt, row_stride, nparts, part_stride, n = _fused_args(fused, parts)
-    assert o.dtype == torch.float32 and o.is_contiguous() and o.shape == (n, heads * vdim) == out.shape and out.is_contiguous()
-    assert weight is None or (weight.shape == (vdim,) and weight.is_contiguous())
+    assert o.dtype == torch.float32 and o.is_contiguous() and o.shape == (n, heads * vdim) == out.shape and out.stride(1) == 1
+    assert weight is None or (weight.shape in ((vdim,), (heads * vdim,)) and weight.is_contiguous())
+    whole_row = weight is not None and weight.shape[0] == heads * vdim
     lib = load_family("linear_attention")
-    _check(lib.wllm_head_gate_norm(_ptr(o), ptr, dt, row_stride, nparts, part_stride, gate_off, _ptr(weight),
-                                   _dt(weight) if weight is not None else _F32, c_float(eps), _ptr(out), _dt(out), n, heads,
-                                   vdim, _stream()), "head_gate_norm")
+    _check(lib.wllm_head_gate_norm_rows(_ptr(o), ptr, dt, row_stride, nparts, part_stride, gate_off, _ptr(weight),
+                                        _dt(weight) if weight is not None else _F32, 1 if whole_row else 0, c_float(eps), _ptr(out),
+                                        _dt(out), max(out.stride(0), heads * vdim), c_float(factor), n, heads, vdim, _stream()),
+           "head_gate_norm")
     return out
 
 
@@ -1140,13 +1224,15 @@ def delta_scan(q, k, v, beta, decay, state, out, req_q_start, req_q_len, req_slo
 
 
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, w_gate, chosen: torch.Tensor, weights: torch.Tensor, gate_out,
-              groups: int = 1, groups_kept: int = 1, scores: str = "softmax") -> None:
+              groups: int = 1, groups_kept: int = 1, scores: str = "softmax", correction: torch.Tensor | None = None,
+              renorm_eps: float | None = None) -> None:
     """The router of routed experts (csrc/moe.cu): scores = softmax(w_router x) in 32-bit over all E experts (`scores`
     'sigmoid': sigmoid(w_router x) expert by expert, not normalised; without groups the choice is made on the logits, whose order
     the sigmoid keeps, so that large logits that all round to a score of 1 do not tie), the choice
     limited to the `groups_kept` best of `groups` groups of neighbouring experts; chosen [n, top] (descending score) and
-    weights [n, top] (the scores as they are).  With `w_gate` [H], gate_out[n] = sigmoid(w_gate . x)."""
-    _need_cuda(x, w_router, w_gate, chosen, weights, gate_out)
+    weights [n, top] (the scores as they are).  With `w_gate` [H], gate_out[n] = sigmoid(w_gate . x).  `correction` [E] (float32) joins
+    the scores for the choice alone; with `renorm_eps` the weights are the chosen scores over (their sum + renorm_eps)."""
+    _need_cuda(correction, x, w_router, w_gate, chosen, weights, gate_out)
     n, H = x.shape
     E, top = w_router.shape[0], chosen.shape[1]
     assert x.is_contiguous() and w_router.dtype == torch.float32 and w_router.shape == (E, H) and w_router.is_contiguous()
@@ -1155,11 +1241,13 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, w_gate, chosen: torch.Ten
     if w_gate is not None:
         assert w_gate.dtype == torch.float32 and w_gate.shape == (H,) and w_gate.is_contiguous()
         assert gate_out.dtype == torch.float32 and gate_out.shape == (n,) and gate_out.is_contiguous()
+    assert correction is None or (correction.dtype == torch.float32 and correction.shape == (E,) and correction.is_contiguous())
     if scores not in ("softmax", "sigmoid"):
         raise KernelError(f"router scores {scores!r}: 'softmax' or 'sigmoid'")
     lib = load_family("moe")
-    _check(lib.wllm_moe_route(_ptr(x), _dt(x), _ptr(w_router), _ptr(w_gate), _ptr(chosen), _ptr(weights), _ptr(gate_out), n, H, E,
-                              top, groups, groups_kept, 1 if scores == "sigmoid" else 0, _stream()), f"moe_route(experts={E}, top={top}, groups={groups}/{groups_kept})")
+    _check(lib.wllm_moe_route_corrected(_ptr(x), _dt(x), _ptr(w_router), _ptr(w_gate), _ptr(chosen), _ptr(weights), _ptr(gate_out), n, H, E,
+                                        top, groups, groups_kept, 1 if scores == "sigmoid" else 0, _ptr(correction),
+                                        c_float(-1.0 if renorm_eps is None else renorm_eps), _stream()), f"moe_route(experts={E}, top={top}, groups={groups}/{groups_kept})")
 
 
 MOE_TILE_ROWS = 128      # rows of a row tile of the experts' products on the tensor-memory kernel
@@ -1174,11 +1262,12 @@ MOE_PLAN_SEGMENTS = 8     # warps an expert that scan a long list of pairs (csrc
 
 
 def moe_plan(chosen: torch.Tensor, count: torch.Tensor, offset: torch.Tensor, order: torch.Tensor, place: torch.Tensor,
-             tiles: torch.Tensor | None = None, scratch: torch.Tensor | None = None) -> None:
+             tiles: torch.Tensor | None = None, scratch: torch.Tensor | None = None, real_experts: int | None = None) -> None:
     """The (token, rank) pairs of `chosen` [n, top] sorted by expert, stably: count [E], offset [E + 1], order [pairs] (sorted
     row -> pair), place [pairs] (pair -> sorted row).  `tiles` (int32, 1 + 3 * moe_row_tiles(pairs, E)): the table of row
     tiles for gemm_bf16_tc_grouped: their number, then (expert, first sorted row, rows) a tile.  `scratch` (int32,
-    MOE_PLAN_SEGMENTS * E): with it a long list is scanned by several warps an expert; the result is the same."""
+    MOE_PLAN_SEGMENTS * E): with it a long list is scanned by several warps an expert; the result is the same.  `real_experts`: the
+    experts that have matrices (the first ones of the E; None: all): the table lists their tiles."""
     _need_cuda(chosen, count, offset, order, place, tiles, scratch)
     pairs, E = chosen.numel(), count.shape[0]
     assert offset.shape == (E + 1,) and order.shape == place.shape == (pairs,)
@@ -1187,8 +1276,8 @@ def moe_plan(chosen: torch.Tensor, count: torch.Tensor, offset: torch.Tensor, or
     assert tiles is None or (tiles.dtype == torch.int32 and tiles.is_contiguous() and tiles.numel() >= 1 + 3 * moe_row_tiles(pairs, E))
     lib = load_family("moe")
     assert scratch is None or (scratch.dtype == torch.int32 and scratch.is_contiguous() and scratch.numel() >= MOE_PLAN_SEGMENTS * E)
-    _check(lib.wllm_moe_plan_tiles(_ptr(chosen), pairs, E, _ptr(count), _ptr(offset), _ptr(order), _ptr(place), _ptr(tiles),
-                                   MOE_TILE_ROWS, _ptr(scratch), _stream()), "moe_plan")
+    _check(lib.wllm_moe_plan_real(_ptr(chosen), pairs, E, _ptr(count), _ptr(offset), _ptr(order), _ptr(place), _ptr(tiles),
+                                  MOE_TILE_ROWS, _ptr(scratch), E if real_experts is None else real_experts, _stream()), "moe_plan")
     global launches
     launches += 1
 
@@ -1259,18 +1348,142 @@ def gemm_bf16_tc_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, ti
     return out
 
 
-def moe_combine(y: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, shared, gate, out: torch.Tensor) -> torch.Tensor:
+def moe_combine(y: torch.Tensor, place: torch.Tensor, weights: torch.Tensor, shared, gate, out: torch.Tensor,
+                chosen: torch.Tensor | None = None, real_experts: int = 0, x: torch.Tensor | None = None) -> torch.Tensor:
     """out[t] = sum over ranks k, in order, of weights[t, k] * y[place[t * top + k]]  (+ gate[t] * shared[t]; `shared`:
-    None or (tensor [n, H] | float32 partial sums [P, n, H], P or 0)).  `weights` None: the outputs are added as they are."""
-    _need_cuda(y, place, weights, gate, out, shared[0] if shared is not None else None)
+    None or (tensor [n, H] | float32 partial sums [P, n, H], P or 0); `gate` None: 1).  `weights` None: the outputs are added as they
+    are.  With `chosen` [n, top], ranks whose expert is `real_experts` or above (identity experts) take the token's row of `x` [n, H]
+    in place of y."""
+    _need_cuda(y, place, weights, gate, out, chosen, x, shared[0] if shared is not None else None)
     n, H = out.shape
     top = place.shape[0] // max(n, 1)
     assert y.dtype == torch.float32 == out.dtype and y.is_contiguous() and out.is_contiguous() and y.shape[1] == H
     assert place.shape == (n * top,) and (weights is None or (weights.shape == (n, top) and weights.dtype == torch.float32 and weights.is_contiguous()))
+    assert chosen is None or (chosen.shape == (n, top) and chosen.is_contiguous() and x is not None and x.shape == (n, H) and x.is_contiguous())
     ps = _branch_args(shared, n, H) if shared is not None else (_ptr(None), _F32, 1, ctypes.c_longlong(0))
     lib = load_family("moe")
-    _check(lib.wllm_moe_combine(_ptr(y), _ptr(_int32(place, "place")), _ptr(weights), top, *ps, _ptr(gate), _ptr(out), n, H,
-                                _stream()), "moe_combine")
+    _check(lib.wllm_moe_combine_own(_ptr(y), _ptr(_int32(place, "place")), _ptr(weights), top, *ps, _ptr(gate), _ptr(out), n, H,
+                                    _ptr(_int32(chosen, "chosen") if chosen is not None else None), real_experts,
+                                    _ptr(x if chosen is not None else None), _dt(x) if chosen is not None else _F32, _stream()), "moe_combine")
+    return out
+
+
+def token_blend(h: torch.Tensor, mu: torch.Tensor, ctx, kept: torch.Tensor, out: torch.Tensor, tiles: torch.Tensor | None = None,
+                groups: int = 0) -> torch.Tensor:
+    """out[s, t] = h[t] + (h[t - 1] - h[t]) * mu[s] for every stream s (csrc/token_blend.cu); the row before a portion's first token is the
+    one `kept` [slots, 2, H] holds for its request (zeros in front of the sequence), and the portion's last row is left there.
+    `ctx`: the step's index arrays.  `tiles` (int32, 1 + 3 * groups * ceil(n / MOE_TILE_ROWS)): the table of row tiles for
+    gemm_bf16_tc_grouped over the first `groups` streams."""
+    _need_cuda(h, mu, kept, out, tiles)
+    n, H = h.shape
+    S = mu.shape[0]
+    assert h.is_contiguous() and mu.dtype == torch.float32 and mu.shape == (S, H) and mu.is_contiguous()
+    assert kept.dtype == h.dtype == out.dtype and kept.is_contiguous() and kept.shape[1:] == (2, H) and out.shape == (S, n, H) and out.is_contiguous()
+    assert tiles is None or (tiles.dtype == torch.int32 and tiles.is_contiguous() and 0 < groups <= S and
+                             tiles.numel() >= 1 + 3 * groups * -(-n // MOE_TILE_ROWS))
+    lib = load_family("token_blend")
+    _check(lib.wllm_token_blend(_ptr(h), _dt(h), n, H, _ptr(mu), S, _ptr(_int32(ctx.positions, "positions")),
+                                _ptr(_int32(ctx.token_req, "token_req")), _ptr(_int32(ctx.req_q_start, "req_q_start")),
+                                _ptr(_int32(ctx.req_q_len, "req_q_len")), _ptr(_int32(ctx.req_slot, "req_slot")), _ptr(kept), _ptr(out),
+                                _ptr(tiles), groups, MOE_TILE_ROWS, _stream()), "token_blend")
+    return out
+
+
+BLENDED_MAX_ROWS = 32      # tokens of a step up to which the blends and their products are one kernel
+
+
+def blended_product_ok(h: torch.Tensor, w: torch.Tensor) -> bool:
+    """Whether the blends' products of a step of single tokens can run as one kernel."""
+    return h.dtype == torch.bfloat16 == w.dtype and h.shape[0] <= BLENDED_MAX_ROWS and h.shape[1] % 8 == 0
+
+
+def blended_product(h: torch.Tensor, mu: torch.Tensor, w: torch.Tensor, segments, ctx, kept: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out[t, o] = w[o] . (h[t] + (h[t - 1] - h[t]) * mu[s]) for steps in which no request brings more than one token
+    (csrc/token_blend.cu).  `segments`: (rows, stream) of the matrices that lie one below the other in w [N, H]; stream -1 reads h itself.
+    `kept` as for token_blend; out float32 [n, N]."""
+    _need_cuda(h, mu, w, kept, out)
+    n, H = h.shape
+    rows, streams = [r for r, _ in segments], [s for _, s in segments]
+    assert h.dtype == torch.bfloat16 == w.dtype == kept.dtype and h.is_contiguous() and w.is_contiguous() and w.shape == (sum(rows), H)
+    assert mu.dtype == torch.float32 and mu.is_contiguous() and mu.shape[1] == H and max(streams) < mu.shape[0]
+    assert kept.is_contiguous() and kept.shape[1:] == (2, H) and out.dtype == torch.float32 and out.shape == (n, sum(rows)) and out.is_contiguous()
+    lib = load_family("token_blend")
+    ints = ctypes.c_int * len(rows)
+    _check(lib.wllm_blended_product(_ptr(h), n, H, _ptr(mu), _ptr(w), ints(*rows), ints(*streams), len(rows),
+                                    _ptr(_int32(ctx.positions, "positions")), _ptr(_int32(ctx.token_req, "token_req")),
+                                    _ptr(_int32(ctx.req_q_len, "req_q_len")), _ptr(_int32(ctx.req_slot, "req_slot")), _ptr(kept), _ptr(out),
+                                    _stream()), f"blended_product({n}x{sum(rows)}x{H})")
+    return out
+
+
+RGLRU_RUNS_FROM = 128      # portions of at least this many tokens are walked as runs side by side
+RGLRU_STEP_MAX_BLOCK = 1024
+
+
+def _rglru_input(fused, parts: int, unit: dict, ctx, ring: torch.Tensor) -> tuple:
+    """The projection of a gated linear recurrent unit and what goes with it, as the kernels take it.  `unit`: y_off, x_off, x_bias, y_bias,
+    taps [T, W], conv_bias (all 32-bit)."""
+    ptr, dt, row_stride, nparts, part_stride, n = _fused_args(fused, parts)
+    T, W = unit["taps"].shape
+    for key in ("x_bias", "y_bias", "conv_bias"):
+        assert unit[key].dtype == torch.float32 and unit[key].shape == (W,) and unit[key].is_contiguous()
+    assert unit["taps"].dtype == torch.float32 and unit["taps"].is_contiguous() and max(unit["y_off"], unit["x_off"]) + W <= fused.shape[-1]
+    assert ring.dtype == torch.float32 and ring.is_contiguous() and ring.shape[1:] == (T, W)
+    _need_cuda(fused, ring, *[unit[k] for k in ("x_bias", "y_bias", "taps", "conv_bias")])
+    return (ptr, dt, row_stride, nparts, part_stride, unit["y_off"], unit["x_off"], _ptr(unit["x_bias"]), _ptr(unit["y_bias"]),
+            _ptr(unit["taps"]), _ptr(unit["conv_bias"]), T, W, _ptr(_int32(ctx.positions, "positions")),
+            _ptr(_int32(ctx.token_req, "token_req")), _ptr(_int32(ctx.req_q_start, "req_q_start")),
+            _ptr(_int32(ctx.req_slot, "req_slot")), _ptr(ring)), n, W
+
+
+def _rglru_gates(gates: dict, W: int) -> tuple:
+    """`gates`: ra, ri [B, s, s], ra_bias, ri_bias, lam [W] (32-bit), c."""
+    B, s, _ = gates["ra"].shape
+    assert gates["ra"].shape == gates["ri"].shape == (B, s, s) and B * s == W and gates["ra"].dtype == gates["ri"].dtype
+    assert gates["ra"].is_contiguous() and gates["ri"].is_contiguous()
+    for key in ("ra_bias", "ri_bias", "lam"):
+        assert gates[key].dtype == torch.float32 and gates[key].shape == (W,) and gates[key].is_contiguous()
+    _need_cuda(*[gates[k] for k in ("ra", "ri", "ra_bias", "ri_bias", "lam")])
+    return (_ptr(gates["ra"]), _ptr(gates["ri"]), _dt(gates["ra"]), _ptr(gates["ra_bias"]), _ptr(gates["ri_bias"]), _ptr(gates["lam"]),
+            c_float(gates["c"]), B)
+
+
+def rglru_gates(fused, parts: int, unit: dict, gates: dict, ctx, ring: torch.Tensor, ab: torch.Tensor) -> torch.Tensor:
+    """Convolution and gates of a real-gated linear recurrent unit (csrc/rg_lru.cu): ab [n, W, 2] = (a, sqrt(1 - a^2) i u), 32-bit."""
+    args, n, W = _rglru_input(fused, parts, unit, ctx, ring)
+    assert ab.dtype == torch.float32 and ab.shape == (n, W, 2) and ab.is_contiguous()
+    lib = load_family("rg_lru")
+    _check(lib.wllm_rglru_gates(*args, *_rglru_gates(gates, W), n, _ptr(ab), _stream()), "rglru_gates")
+    return ab
+
+
+def rglru_scan(fused, parts: int, unit: dict, ctx, ring: torch.Tensor, ab: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+               long_portions: bool) -> torch.Tensor:
+    """S <- a S + b over every request's tokens of the step, from and to its row of `state` [slots, W]; out = S * gelu_tanh(y + bias) [n, W]; the
+    convolution's newest inputs go to `ring`.  `long_portions`: runs of tokens side by side instead of token by token."""
+    args, n, W = _rglru_input(fused, parts, unit, ctx, ring)
+    assert ab.dtype == torch.float32 and ab.shape == (n, W, 2) and ab.is_contiguous() and out.shape == (n, W) and out.is_contiguous()
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (W,)
+    lib = load_family("rg_lru")
+    _check(lib.wllm_rglru_scan(*args, _ptr(ab), _ptr(_int32(ctx.req_q_len, "req_q_len")), ctx.req_q_len.shape[0], _ptr(state), _ptr(out),
+                               _dt(out), 1 if long_portions else 0, _stream()), "rglru_scan")
+    return out
+
+
+def rglru_step_ok(gates: dict, fused, x_off: int) -> bool:
+    """Whether convolution, gates and recurrence of a step of single tokens can run as one kernel."""
+    s = gates["ra"].shape[1]
+    return gates["ra"].dtype == torch.bfloat16 and s % 8 == 0 and s <= RGLRU_STEP_MAX_BLOCK and x_off % 8 == 0 and fused.stride(-2) % 8 == 0 \
+        and fused.data_ptr() % 16 == 0
+
+
+def rglru_step(fused, parts: int, unit: dict, gates: dict, ctx, ring: torch.Tensor, state: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """rglru_gates and rglru_scan in one kernel for steps in which no request brings more than one token."""
+    args, n, W = _rglru_input(fused, parts, unit, ctx, ring)
+    assert out.shape == (n, W) and out.is_contiguous() and state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (W,)
+    lib = load_family("rg_lru")
+    _check(lib.wllm_rglru_step(*args, *_rglru_gates(gates, W), n, _ptr(_int32(ctx.req_q_len, "req_q_len")), _ptr(state), _ptr(out), _dt(out),
+                               _stream()), "rglru_step")
     return out
 
 

@@ -27,11 +27,16 @@ finished sums in 32-bit; with row_norm), distance_slopes (one number per query h
 loses slope_h * (i - j), after the scale and the cap), value_mix ({"weight": name, "role": 'first' | 'later', "key":
 label}: the layers that share a label blend their values with those of the layer whose role is 'first', for the same
 token: v <- (1 - w) v + w v_first with w the scalar tensor `weight`, in 32-bit; the blended values are what is cached.  The
-first layer leaves its values in a buffer of the step; its own `weight` tensor is read and not used).
+first layer leaves its values in a buffer of the step; its own `weight` tensor is read and not used), head_norm ({"eps": e, and
+any of "q": name, "k": name, "values": True}: every query and key head is divided by its root mean square and multiplied by the
+gain [head_dim] of that name, shared by the heads, in front of the turn; with `values` every value head is divided by its root mean
+square before it is cached), query_temperature ({"coef": c, "every": m}: queries are multiplied by
+1 + c * ln(floor((p + 1) / m) + 1) at position p; with head_norm).
 
 A mixer may be one of several that read the same input (a block that runs two mixers side
 by side): `input_weights()` lists the matrices that read the input, `mix(fused, parts,
-col0, ...)` runs the mixer on its columns of a fused product that somebody else made.
+col0, ...)` runs the mixer on its columns of a fused product that somebody else made, and `heads(...)` does so up to the output
+projection (a mixer that projects two mixers' heads at once).
 
 One forward serves whole prompts, portions and decoded tokens alike: the step's keys
 and values go into the pages first, then every token attends through its request's
@@ -83,6 +88,14 @@ class PagedAttention:
             raise ValueError("projection biases and blended values are built into the kernel that norms q and k as whole rows (row_norm)")
         if self.slope_values is not None and len(self.slope_values) != self.nq:
             raise ValueError(f"{len(self.slope_values)} distance slopes for {self.nq} query heads")
+        self.head_norm = spec.options.get("head_norm")
+        self.temperature = spec.options.get("query_temperature")
+        if self.head_norm is not None and (self.row_norm is not None or self.borrows or spec.options.get("qk_unit_norm_eps") is not None):
+            raise ValueError("head norms stand for themselves: no row norms, no unit norms, and a key projection of the mixer's own")
+        if self.head_norm is not None and (("q" in self.head_norm) != ("k" in self.head_norm)):
+            raise ValueError("head norms carry gains for q and k, or for neither")
+        if self.temperature is not None and self.head_norm is None:
+            raise ValueError("a query temperature is built into the kernel that norms heads (head_norm)")
         if self.row_norm is not None and self.borrows:
             raise ValueError("row norms of q and k need the mixer's own key projection")
         self.position = POSITIONS.build(spec.position)
@@ -122,6 +135,8 @@ class PagedAttention:
         if self.row_norm is not None:
             out += [ParamSpec(self.row_norm["q"], (self.nq * self.hd_file,), "vector"),
                     ParamSpec(self.row_norm["k"], (self.nkv * self.hd_file,), "vector")]
+        if self.head_norm is not None and "q" in self.head_norm:
+            out += [ParamSpec(self.head_norm[k], (self.hd_file,), "vector") for k in ("q", "k")]
         if self.bias_names is not None:
             out += [ParamSpec(self.bias_names["q"], (self.nq * self.hd_file,), "vector"),
                     ParamSpec(self.bias_names["k"], (self.nkv * self.hd_file,), "vector"),
@@ -150,6 +165,9 @@ class PagedAttention:
             gains = [heads_padded(fetch(self.row_norm[k])[:, None], heads, self.hd_file, self.hd)[:, 0].contiguous()
                      for k, heads in (("q", self.nq), ("k", self.nkv))]
             self.q_gain, self.k_gain = gains
+        if self.head_norm is not None and "q" in self.head_norm:
+            self.q_gain, self.k_gain = (heads_padded(fetch(self.head_norm[k])[:, None], 1, self.hd_file, self.hd)[:, 0].contiguous()
+                                        for k in ("q", "k"))
         if self.bias_names is not None:
             rows = [heads_padded(fetch(self.bias_names[k]).to(torch.float32)[:, None], heads, size, to)[:, 0]
                     for k, heads, size, to in (("q", self.nq, self.hd_file, self.hd), ("k", self.nkv, self.hd_file, self.hd),
@@ -174,6 +192,13 @@ class PagedAttention:
 
     def mix(self, fused: torch.Tensor, parts: int, col0: int, ctx, cache: CacheRef):
         """The mixer on columns col0 .. col0 + width of a fused product [n, W] (or partial sums [parts, n, W])."""
+        attn = ctx.buffer(self.tag + "attn", (fused.shape[-2], self.nq * self.vd), self.model_dtype)
+        self.heads(fused, parts, col0, ctx, cache, attn)
+        return as_branch(ops.project(attn, self.wo, lambda name, shape, dt: ctx.buffer(self.tag + "branch_" + name, shape, dt)))
+
+    def heads(self, fused: torch.Tensor, parts: int, col0: int, ctx, cache: CacheRef, attn: torch.Tensor) -> None:
+        """The heads' outputs (what the output projection reads) into `attn` [n, num_heads * value size], whose rows may be columns of
+        wider rows."""
         if self.borrows and cache.writes:
             raise ValueError("an attention mixer without key and value projections must stand in a run that reads another run's cache")
         n = fused.shape[-2]
@@ -195,15 +220,19 @@ class PagedAttention:
                                        self.hd, self.position.rotary_dim, group.page_size, self.q_gain, self.k_gain,
                                        float(self.row_norm["eps"]), self.nq * self.hd_file, self.nkv * self.hd_file,
                                        in_splits=parts, pairing=pairing, vd=self.vd, bias=self.bias, **self._blend_args(n, ctx))
+        elif self.head_norm is not None:
+            t = self.temperature or {"coef": 0.0, "every": 0}
+            ops.rope_head_norm_kv_write(qkv, q, ctx.positions, slots, self.position.inv_freq, k_pages, v_pages, self.nq, self.nkv, self.hd,
+                                        self.position.rotary_dim, group.page_size, float(self.head_norm["eps"]), self.q_gain, self.k_gain,
+                                        self.hd_file, self.vd_file, bool(self.head_norm.get("values")), float(t["coef"]), int(t["every"]),
+                                        in_splits=parts, pairing=pairing, vd=self.vd)
         else:
             ops.rope_kv_write(qkv[..., :self.qkv_width] if self.width != self.qkv_width else qkv, q, ctx.positions, slots,
                               self.position.inv_freq, k_pages, v_pages, self.nq, 0 if self.borrows else self.nkv, self.hd,
                               self.position.rotary_dim, group.page_size, in_splits=parts, pairing=pairing, **extra)
-        attn = ctx.buffer(self.tag + "attn", (n, self.nq * self.vd), self.model_dtype)
         self.attend(q, attn, k_pages, v_pages, ctx, cache.group)
         if self.gate_name is not None:
             ops.sigmoid_gate(attn, qkv, parts, self.qkv_width)
-        return as_branch(ops.project(attn, self.wo, lambda name, shape, dt: ctx.buffer(self.tag + "branch_" + name, shape, dt)))
 
     def _blend_args(self, n: int, ctx) -> dict:
         """The buffer of the step in which the first layer of a label leaves its values, and this layer's part in it."""

@@ -125,6 +125,34 @@ class MeanOfNormed:
         return ops.branch_norm(pa, self.gain_a, out, self.eps, center=False, factor=self.factor, b=pb, weight_b=self.gain_b)
 
 
+class BranchSum:
+    """Several branch outputs that join the residual at once, each times a factor: terms of (tensor [n, hidden], `Partials`,
+    `MeanOfNormed` or `BranchSum`; factor).  A norm that takes several addends folds them in one kernel; `materialize` adds them alone."""
+
+    def __init__(self, terms):
+        self.terms = []
+        for branch, factor in terms:
+            self.terms += [(b, f * factor) for b, f in branch.terms] if isinstance(branch, BranchSum) else [(branch, factor)]
+
+    def addends(self, ctx) -> list:
+        """(tensor, parts, factor) of every term, as the norm kernels take them."""
+        out = []
+        for i, (branch, factor) in enumerate(self.terms):
+            if hasattr(branch, "materialize"):
+                branch = branch.materialize(ctx, f"branch_sum_{i}")
+            out.append((*branch_pair(branch), factor))
+        return out
+
+    def materialize(self, ctx, name: str = "branch_sum") -> torch.Tensor:
+        from ..kernels import ops
+        terms = self.addends(ctx)
+        out = ctx.buffer(name, tuple(terms[0][0].shape[-2:]), torch.float32)
+        out.zero_()
+        for i in range(0, len(terms), 3):
+            ops.fold_norm(out, terms[i:i + 3], [], 0.0, [])
+        return out
+
+
 class NormedBranch:
     """A branch output that is to pass a norm of its own before it joins the residual (a block that norms behind its
     sublayers): `branch` is a tensor, `Partials` or `MeanOfNormed`, `norm` the norm part.  The next norm of the
@@ -134,7 +162,7 @@ class NormedBranch:
         self.branch, self.norm = branch, norm
 
     def materialize(self, ctx, name: str = "branch_normed") -> torch.Tensor:
-        inner = self.branch.materialize(ctx) if isinstance(self.branch, MeanOfNormed) else self.branch
+        inner = self.branch.materialize(ctx) if hasattr(self.branch, "materialize") else self.branch
         return self.norm.branch(inner, ctx, name)
 
 

@@ -25,10 +25,17 @@ spec options: norm_in, mixer, norm_mixer_out, and norm_post, feed_forward, norm_
 rounding to the model's element type in one kernel).  `feed_forward` may be None.
 
 spec options: reader, mixer, norm_mixer_out, and feed_forward, norm_ff_out (both or none).
+
+'parallel': both sublayers read the same residual, each through a norm of its own, and are added together,
+    x = x + (mixer(norm_mixer(x)) + feed_forward(norm_ff(x)))
+The two norms (kind 'grouped_rmsnorm') are one kernel, which also folds in what the block before left pending: a `BranchSum` of its
+mixer's and its feed-forward's output.  `feed_forward` may be None.
+
+spec options: norm_mixer, mixer, and norm_ff, feed_forward (both or none).
 """
 from __future__ import annotations
 
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, CacheRef, NormedBranch, Residual
+from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, BranchSum, CacheRef, NormedBranch, Residual
 
 
 @BLOCKS.register("pre_norm")
@@ -120,3 +127,34 @@ class BranchNormedBlock:
         residual.pending = NormedBranch(self.mixer(self.reader(residual, ctx), ctx, cache), self.norm_mixer_out)
         if self.feed_forward is not None:
             residual.pending = NormedBranch(self.feed_forward(self.reader(residual, ctx), ctx), self.norm_ff_out)
+
+
+@BLOCKS.register("parallel")
+class ParallelBlock:
+    graph_safe = True
+
+    def __init__(self, spec, hidden_size: int, model_dtype):
+        kw = dict(hidden_size=hidden_size, model_dtype=model_dtype)
+        self.norm_mixer = NORMS.build(spec.norm_mixer, **kw)
+        self.mixer = MIXERS.build(spec.mixer, **kw)
+        self.feed_forward = None
+        if spec.options.get("feed_forward") is not None:
+            self.norm_ff = NORMS.build(spec.norm_ff, **kw)
+            self.feed_forward = FEED_FORWARDS.build(spec.feed_forward, **kw)
+            if not hasattr(self.norm_mixer, "pair"):
+                raise TypeError(f"the norms of a parallel block are worked out together; '{spec.norm_mixer.kind}' cannot do that")
+
+    def parts(self):
+        first = [self.norm_mixer, self.mixer]
+        return first if self.feed_forward is None else first + [self.norm_ff, self.feed_forward]
+
+    def cache_need(self):
+        return self.mixer.cache_need()
+
+    def __call__(self, residual: Residual, ctx, cache: CacheRef) -> None:
+        if self.feed_forward is None:
+            residual.pending = BranchSum([(self.mixer(self.norm_mixer(residual, ctx), ctx, cache), 1.0)])
+            return
+        h, g = self.norm_mixer.pair(residual, self.norm_ff, ctx)
+        mixed = self.mixer(h, ctx, cache)
+        residual.pending = BranchSum([(mixed, 1.0), (self.feed_forward(g, ctx), 1.0)])

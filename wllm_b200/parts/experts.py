@@ -7,8 +7,11 @@ is its best expert's and only experts of the `groups_kept` best groups can be ch
 the default, over all experts; 'sigmoid': expert by expert, not normalised), gated (default True; False: an expert is
 down(act(up x)) with tensors <prefix><j>.up / .down and activation 'relu_squared'), weight_on ('output', the default: the
 chosen experts' outputs are multiplied by their scores; 'input': their inputs are, the output is the sum of expert(s x)), shared (None, or
-the options of a 'gated_dense' unit that every token runs, plus gate_weight: the checkpoint name of one row [1, hidden]; the
-unit's output is multiplied by sigmoid(row . x)).
+the options of a 'gated_dense' unit that every token runs, plus gate_weight: the checkpoint name of one row [1, hidden], the
+unit's output is multiplied by sigmoid(row . x); without gate_weight it is added as it is), identity (so many further experts behind the
+num_experts, without tensors, whose output is the token's row itself; the router has a row for each), correction (checkpoint
+name of a vector [num_experts + identity] that joins the scores for the choice alone), renorm_eps (the weights are the chosen
+scores over their sum + renorm_eps; absent: the scores as they are).
 
 Router logits, the softmax over all experts, the choice and the weights (the chosen experts' scores as they are) are
 32-bit, against a 32-bit copy of the router matrix.  The tokens' (token, rank) pairs are sorted by expert on the device
@@ -32,9 +35,12 @@ class RoutedExperts:
 
     def __init__(self, spec, hidden_size: int, model_dtype: torch.dtype):
         self.E, self.top = int(spec.num_experts), int(spec.top)
+        self.identity = int(spec.options.get("identity") or 0)
+        self.slots = self.E + self.identity                       # what the router chooses from
+        self.correction_name, self.renorm_eps = spec.options.get("correction"), spec.options.get("renorm_eps")
         self.groups, self.groups_kept = int(spec.options.get("groups") or 1), int(spec.options.get("groups_kept") or 1)
-        if self.E % self.groups or not 1 <= self.groups_kept <= self.groups or not 1 <= self.top <= self.groups_kept * (self.E // self.groups):
-            raise ValueError(f"{self.E} experts in {self.groups} groups, {self.groups_kept} kept, top {self.top}: no such choice")
+        if self.slots % self.groups or not 1 <= self.groups_kept <= self.groups or not 1 <= self.top <= self.groups_kept * (self.slots // self.groups):
+            raise ValueError(f"{self.slots} experts in {self.groups} groups, {self.groups_kept} kept, top {self.top}: no such choice")
         self.inter, self.activation = int(spec.intermediate_size), spec.activation
         self.gated = bool(spec.options.get("gated", True))
         self.scores, self.weight_on = spec.options.get("scores") or "softmax", spec.options.get("weight_on") or "output"
@@ -43,6 +49,8 @@ class RoutedExperts:
         if self.activation != ("capped_swish" if self.gated else "relu_squared"):
             raise ValueError("the grouped expert products are built for gated experts with the activation capped_swish and for "
                              "experts without a gate with relu_squared")
+        if self.weight_on == "input" and self.identity:
+            raise ValueError("scores on the experts' inputs are built without identity experts")
         if self.weight_on == "input" and self.gated:
             raise ValueError("scores on the experts' inputs are built for experts without a gate")
         self.limit, self.slope = float(spec.options.get("limit") or 0.0), float(spec.options.get("slope") or 0.0)
@@ -52,25 +60,29 @@ class RoutedExperts:
         shared = spec.options.get("shared")
         if shared is not None:
             shared = dict(shared)
-            self.gate_name = shared.pop("gate_weight")
+            self.gate_name = shared.pop("gate_weight", None)
             self.shared = FEED_FORWARDS.build(make_spec("gated_dense", **shared), hidden_size=hidden_size, model_dtype=model_dtype)
-        self.w_router = self.w_gate = self.w_gu = self.w_down = None
+        self.w_router = self.w_gate = self.w_gu = self.w_down = self.correction = None
 
     def parts(self):
         return [] if self.shared is None else [self.shared]
 
     def param_specs(self):
         H, I = self.hidden_size, self.inter
-        out = [ParamSpec(self.router_name, (self.E, H))]
+        out = [ParamSpec(self.router_name, (self.slots, H))]
+        if self.correction_name is not None:
+            out.append(ParamSpec(self.correction_name, (self.slots,), "vector"))
         for j in range(self.E):
             p = f"{self.prefix}{j}."
             out += ([ParamSpec(p + "gate", (I, H))] if self.gated else []) + [ParamSpec(p + "up", (I, H)), ParamSpec(p + "down", (H, I))]
         if self.shared is not None:
-            out += self.shared.param_specs() + [ParamSpec(self.gate_name, (1, H))]
+            out += self.shared.param_specs() + ([ParamSpec(self.gate_name, (1, H))] if self.gate_name is not None else [])
         return out
 
     def load(self, fetch):
         self.w_router = fetch(self.router_name).to(torch.float32).contiguous()
+        if self.correction_name is not None:
+            self.correction = fetch(self.correction_name).to(torch.float32).contiguous()
         names = [f"{self.prefix}{j}." for j in range(self.E)]
         if self.gated:
             self.w_gu = torch.stack([torch.cat([fetch(p + "gate"), fetch(p + "up")], dim=0) for p in names]).contiguous()
@@ -79,6 +91,7 @@ class RoutedExperts:
         self.w_down = torch.stack([fetch(p + "down") for p in names]).contiguous()
         if self.shared is not None:
             self.shared.load(fetch)
+        if self.gate_name is not None:
             self.w_gate = fetch(self.gate_name).to(torch.float32).reshape(-1).contiguous()
 
     def __call__(self, x: torch.Tensor, ctx):
@@ -86,13 +99,16 @@ class RoutedExperts:
         pairs = n * top
         chosen = ctx.buffer("moe_chosen", (n, top), torch.int32)
         weights = ctx.buffer("moe_weights", (n, top), torch.float32)
-        gate = ctx.buffer("moe_gate", (n,), torch.float32) if self.shared is not None else None
-        ops.moe_route(x, self.w_router, self.w_gate, chosen, weights, gate, self.groups, self.groups_kept, scores=self.scores)
+        gate = ctx.buffer("moe_gate", (n,), torch.float32) if self.gate_name is not None else None
+        ops.moe_route(x, self.w_router, self.w_gate, chosen, weights, gate, self.groups, self.groups_kept, scores=self.scores,
+                      correction=self.correction, renorm_eps=self.renorm_eps)
         unit = None if self.gated else self.activation
         on_input = weights.view(-1) if self.weight_on == "input" else None
-        index = ctx.buffer("moe_index", (2 * self.E + 1 + 2 * pairs,), torch.int32)
-        count, offset = index[:self.E], index[self.E:2 * self.E + 1]
-        order, place = index[2 * self.E + 1:2 * self.E + 1 + pairs], index[2 * self.E + 1 + pairs:]
+        slots = self.slots
+        index = ctx.buffer("moe_index", (2 * slots + 1 + 2 * pairs,), torch.int32)
+        count, offset = index[:slots], index[slots:2 * slots + 1]
+        order, place = index[2 * slots + 1:2 * slots + 1 + pairs], index[2 * slots + 1 + pairs:]
+        real = offset[:self.E + 1]          # identity experts' pairs lie behind all others: the products see the first E experts
         act = ctx.buffer("moe_act", (pairs, self.inter), self.model_dtype)
         y = ctx.buffer("moe_y", (pairs, H), torch.float32)
         # Many rows (portions of prompts): the products run on the tensor-memory kernel over row tiles of one expert each, on
@@ -100,7 +116,8 @@ class RoutedExperts:
         # the kernel on mma.sync does from rows gathered on the fly.
         if pairs >= self.TC_FROM_PAIRS and x.dtype == torch.bfloat16 and ops.tc_grouped_ok(x, self.w_gu) and self.inter % 8 == 0:
             tiles = ctx.buffer("moe_tiles", (1 + 3 * ops.moe_row_tiles(pairs, self.E),), torch.int32)
-            ops.moe_plan(chosen, count, offset, order, place, tiles, ctx.buffer("moe_plan", (ops.MOE_PLAN_SEGMENTS * self.E,), torch.int32))
+            ops.moe_plan(chosen, count, offset, order, place, tiles, ctx.buffer("moe_plan", (ops.MOE_PLAN_SEGMENTS * slots,), torch.int32),
+                         real_experts=self.E)
             # (scores on the inputs: the rows are multiplied while they are copied, rounded once)
             rows = ops.moe_gather(x, order, top, ctx.buffer("moe_rows", (pairs, H), self.model_dtype), row_weights=on_input)
             ops.gemm_bf16_tc_grouped(rows, self.w_gu, act, tiles, self.gated, self.limit, self.slope, unit=unit)
@@ -108,8 +125,9 @@ class RoutedExperts:
         else:
             ops.moe_plan(chosen, count, offset, order, place)
             # (scores on the inputs: the up product is linear, so the score multiplies its 32-bit sums in front of the activation)
-            ops.moe_grouped(x, self.w_gu, act, offset, order, top, self.gated, self.limit, self.slope, unit=unit, row_weights=on_input)
-            ops.moe_grouped(act, self.w_down, y, offset, order, top, False)
+            ops.moe_grouped(x, self.w_gu, act, real, order, top, self.gated, self.limit, self.slope, unit=unit, row_weights=on_input)
+            ops.moe_grouped(act, self.w_down, y, real, order, top, False)
         shared = branch_pair(self.shared(x, ctx)) if self.shared is not None else None
         out = ctx.buffer("moe_out", (n, H), torch.float32)
-        return ops.moe_combine(y, place, None if self.weight_on == "input" else weights, shared, gate, out)
+        own = dict(chosen=chosen, real_experts=self.E, x=x) if self.identity else {}
+        return ops.moe_combine(y, place, None if self.weight_on == "input" else weights, shared, gate, out, **own)

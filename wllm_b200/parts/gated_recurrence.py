@@ -1,0 +1,82 @@
+"""A gated linear recurrent unit behind a short convolution.
+
+'rg_lru': two branches of `width` channels, y = gelu_tanh(y_proj x + y_bias) and u = conv(x_proj x + x_bias), a causal convolution per
+channel with `conv_taps` taps that look back only (the last tap weighs the token itself; inputs in front of the sequence are zero)
+and a bias; u in `blocks` equal parts, each with two square maps,
+
+    r = sigmoid(r_gate u + r_bias),  i = sigmoid(i_gate u + i_bias),  log a = -c r softplus(decay),  a = exp(log a)
+    S_t = a S_(t-1) + sqrt(1 - a^2) i u,    output = o_proj(S * y)
+
+S starts at zero and lives, per channel, in 32-bit in the request's state slot, beside the convolution's last inputs (a ring of
+conv_taps rows, the input of position p in row p mod conv_taps).  Convolution, gates and recurrence are 32-bit (csrc/rg_lru.cu).
+
+spec options: width, blocks, conv_taps, gate_factor (c), y_proj / x_proj [width, hidden], y_bias, x_bias [width], conv [width,
+conv_taps], conv_bias [width], r_gate / i_gate [blocks, width / blocks, width / blocks] (out, in), r_bias / i_bias [blocks, width /
+blocks], decay [width], o_proj [hidden, width] (checkpoint names).  One product makes y | x.
+"""
+from __future__ import annotations
+
+import torch
+
+from ..kernels import ops
+from .base import MIXERS, CacheRef, ParamSpec, StateNeed, as_branch
+
+_NAMES = ("y_proj", "x_proj", "y_bias", "x_bias", "conv", "conv_bias", "r_gate", "i_gate", "r_bias", "i_bias", "decay", "o_proj")
+
+
+@MIXERS.register("rg_lru")
+class GatedRecurrence:
+    graph_safe = True
+
+    def __init__(self, spec, hidden_size: int, model_dtype: torch.dtype):
+        self.width, self.blocks, self.taps = int(spec.width), int(spec.blocks), int(spec.conv_taps)
+        if self.width % self.blocks:
+            raise ValueError(f"{self.width} channels in {self.blocks} equal blocks: no such cut")
+        self.c = float(spec.gate_factor)
+        self.hidden_size, self.model_dtype = hidden_size, model_dtype
+        self.names = {k: spec.options[k] for k in _NAMES}
+        self.w_in = self.wo = self.conv = self.conv_bias = self.x_bias = self.y_bias = None
+        self.ra = self.ri = self.ra_bias = self.ri_bias = self.decay = None
+        self.x_off = 0
+        self.tag = ""
+
+    def cache_need(self):
+        return StateNeed((("state", (self.width,), torch.float32), ("conv", (self.taps, self.width), torch.float32)))
+
+    def param_specs(self):
+        H, W, B, n = self.hidden_size, self.width, self.blocks, self.names
+        s = W // B
+        return [ParamSpec(n["y_proj"], (W, H)), ParamSpec(n["y_bias"], (W,), "vector"), ParamSpec(n["x_proj"], (W, H)),
+                ParamSpec(n["x_bias"], (W,), "vector"), ParamSpec(n["conv"], (W, self.taps)), ParamSpec(n["conv_bias"], (W,), "vector"),
+                ParamSpec(n["r_gate"], (B, s, s)), ParamSpec(n["r_bias"], (B, s), "vector"), ParamSpec(n["i_gate"], (B, s, s)),
+                ParamSpec(n["i_bias"], (B, s), "vector"), ParamSpec(n["decay"], (W,), "vector"), ParamSpec(n["o_proj"], (H, W))]
+
+    def load(self, fetch):
+        n = self.names
+        def vector(name):
+            return fetch(n[name]).to(torch.float32).reshape(-1).contiguous()
+        y = fetch(n["y_proj"])
+        pad = -self.width % 8                 # x's columns begin on a multiple of 8 (16 bytes of the matrix type), and so do the rows
+        gap = [y.new_zeros((pad, self.hidden_size))] if pad else []
+        self.x_off = self.width + pad
+        self.w_in = torch.cat([y] + gap + [fetch(n["x_proj"])] + gap, dim=0).contiguous()
+        self.wo = fetch(n["o_proj"]).contiguous()
+        self.conv = fetch(n["conv"]).to(torch.float32).t().contiguous()
+        self.x_bias, self.y_bias, self.conv_bias, self.decay = vector("x_bias"), vector("y_bias"), vector("conv_bias"), vector("decay")
+        self.ra, self.ri = fetch(n["r_gate"]).contiguous(), fetch(n["i_gate"]).contiguous()
+        self.ra_bias, self.ri_bias = vector("r_bias"), vector("i_bias")
+
+    def __call__(self, x: torch.Tensor, ctx, cache: CacheRef):
+        n, W = x.shape[0], self.width
+        fused, parts = ops.project(x, self.w_in, lambda name, shape, dt: ctx.buffer(self.tag + "lru_in_" + name, shape, dt))
+        unit = dict(y_off=0, x_off=self.x_off, x_bias=self.x_bias, y_bias=self.y_bias, taps=self.conv, conv_bias=self.conv_bias)
+        gates = dict(ra=self.ra, ri=self.ri, ra_bias=self.ra_bias, ri_bias=self.ri_bias, lam=self.decay, c=self.c)
+        state, ring = ctx.state(cache.state_names["state"]), ctx.state(cache.state_names["conv"])
+        out = ctx.buffer(self.tag + "lru_out", (n, W), self.model_dtype)
+        if ctx.num_multi == 0 and self.model_dtype == torch.bfloat16 and ops.rglru_step_ok(gates, fused, self.x_off):
+            ops.rglru_step(fused, parts, unit, gates, ctx, ring, state, out)
+        else:
+            ab = ctx.buffer(self.tag + "lru_pairs", (n, W, 2), torch.float32)
+            ops.rglru_gates(fused, parts, unit, gates, ctx, ring, ab)
+            ops.rglru_scan(fused, parts, unit, ctx, ring, ab, state, out, ctx.max_q_len >= ops.RGLRU_RUNS_FROM)
+        return as_branch(ops.project(out, self.wo, lambda name, shape, dt: ctx.buffer(self.tag + "lru_branch_" + name, shape, dt)))

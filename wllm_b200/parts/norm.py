@@ -4,6 +4,9 @@
              1 + w, as Gemma stores it, src/wllm/models/gemma.py:42-51; False: gain is w).
 'layernorm'  (x - mean(x)) / sqrt(mean((x - mean)^2) + eps) * w, a layer norm with a gain and no bias.
              spec options: weight, eps.
+'grouped_rmsnorm'  the row in `groups` equal parts, each x / sqrt(mean(x^2) + eps) over itself, the whole times the gain; it folds
+             up to three pending branches with factors (`BranchSum`) in its own kernel, and `pair` gives the outputs of two such norms
+             of the same residual at once (they must agree in eps, groups and offset).  spec options: weight, eps, groups, unit_offset.
 'identity'   nothing is normed: the residual (with the pending branch folded in) rounded to the model's element type, for
              blocks whose sublayers read the residual as it is.  No options, no tensors.
 The statistics and the gain are applied in 32-bit on the 32-bit residual; the result is rounded once to the model's
@@ -15,7 +18,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import NORMS, MeanOfNormed, NormedBranch, ParamSpec, Partials, Residual, branch_pair
+from .base import NORMS, BranchSum, MeanOfNormed, NormedBranch, ParamSpec, Partials, Residual, branch_pair
 
 
 @NORMS.register("rmsnorm")
@@ -53,6 +56,8 @@ class RMSNorm:
         if isinstance(pending, NormedBranch) and self._fusable(pending):
             # the branch's own norm, the add and this norm in one kernel; two mixers' outputs are normed and averaged there too
             post, inner, more = pending.norm, pending.branch, {}
+            if isinstance(inner, BranchSum):
+                inner = inner.materialize(ctx)
             if isinstance(inner, MeanOfNormed):
                 more = dict(gain_a=inner.gain_a, b=branch_pair(inner.b), gain_b=inner.gain_b, inner_eps=inner.eps, factor=inner.factor)
                 inner = inner.a
@@ -70,6 +75,8 @@ class RMSNorm:
         if not isinstance(post, RMSNorm) or post.weight is None or self.hidden_size > 24 * 1024 or \
                 (self.weight is not None and post.weight.dtype != self.weight.dtype):
             return False
+        if isinstance(post, GroupedRMSNorm):
+            return False
         inner = pending.branch
         return not isinstance(inner, MeanOfNormed) or inner.gain_a.dtype == post.weight.dtype == inner.gain_b.dtype
 
@@ -83,6 +90,45 @@ class RMSNorm:
 @NORMS.register("layernorm")
 class LayerNormNoBias(RMSNorm):
     center = True
+
+
+@NORMS.register("grouped_rmsnorm")
+class GroupedRMSNorm(RMSNorm):
+    def __init__(self, spec, hidden_size: int, model_dtype: torch.dtype):
+        super().__init__(spec, hidden_size, model_dtype)
+        self.groups = int(spec.options.get("groups") or 1)
+        if hidden_size % self.groups:
+            raise ValueError(f"a row of {hidden_size} in {self.groups} equal groups: no such cut")
+
+    def _run(self, residual: Residual, ctx, out, rows) -> None:
+        self._fold(residual, ctx, [self.weight], [out], rows)
+
+    def pair(self, residual: Residual, other: "GroupedRMSNorm", ctx) -> tuple:
+        """The outputs of this norm and of `other`, both of the residual with the pending branch folded in."""
+        if (other.eps, other.groups, other.offset) != (self.eps, self.groups, self.offset):
+            raise ValueError("two norms in one kernel share eps, groups and offset")
+        shape = (residual.stream.shape[0], self.hidden_size)
+        outs = [ctx.buffer("normed", shape, self.model_dtype), ctx.buffer("normed_second", shape, self.model_dtype)]
+        self._fold(residual, ctx, [self.weight, other.weight], outs, None)
+        residual.pending = None
+        return tuple(outs)
+
+    def _fold(self, residual: Residual, ctx, weights, outs, rows) -> None:
+        pending = residual.pending
+        if pending is None:
+            terms = []
+        elif isinstance(pending, BranchSum) and len(pending.terms) <= 3:
+            terms = pending.addends(ctx)
+        else:
+            terms = [(*residual.pending_args(ctx), 1.0)]
+        ops.fold_norm(residual.stream, terms, weights, self.eps, outs, groups=self.groups, offset=self.offset, rows=rows)
+
+    def branch(self, branch, ctx, name: str = "branch_normed") -> torch.Tensor:
+        t, parts = branch_pair(branch)
+        row, out = (ctx.buffer(name + which, tuple(t.shape[-2:]), torch.float32) for which in ("_row", ""))
+        row.zero_()
+        ops.fold_norm(row, [(t, parts, 1.0)], [self.weight], self.eps, [out], groups=self.groups, offset=self.offset)
+        return out
 
 
 @NORMS.register("identity")
