@@ -13,8 +13,8 @@
 //                           split-K slabs): q and k turned by the rotary angle of the token's position (optional),
 //                           scaled, v copied, and the decay of every key channel worked out from a low-rank map:
 //                               z = W2 (x W1^T) + b,   a = sigmoid(z)^(1/tau) = exp(log_sigmoid(z) / tau)
-//                           or (decay form 1)  z = W2 tanh(x W1^T) + b,   a = exp(-exp(z)); the decay alone where q, k and v are
-//                           read from the projections as they are
+//                           or (decay form 1)  z = W2 tanh(x W1^T) + b,   a = exp(-exp(z)), handed on as a - 1; the decay alone
+//                           where q, k and v are read from the projections as they are
 //   wllm_linattn_scan       the recurrence.  Grid (tiles of 64 value columns, heads, requests); a lane owns two
 //                           columns of S, a warp a run of at most 16 key channels of them, in registers.  Tokens
 //                           arrive in tiles of 8 through a two-stage cp.async ring; the warps' partial dot products of a
@@ -22,7 +22,9 @@
 //                           into segments that are walked side by side: from zero for their local end states, which a
 //                           small kernel chains into start states, and once more from those for the outputs.
 //                           With a bonus u per key channel the output is taken in front of the update, with the token's own
-//                           key and value counted u times: o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t (time mixing).
+//                           key and value counted u times: o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t (time mixing).  There
+//                           the decays come as a - 1 (S + ((a - 1) S + k v)): a channel that forgets slowly has a close to one, and
+//                           the rounding of a itself, the same at every token, would grow with its memory.
 //   wllm_head_gate_norm     per head: o / sqrt(mean(o^2) + eps) [* w] * silu(g) [* factor], rounded once to the matrix type
 //                           (the operand of the output projection).  w is shared by the heads or a gain of the whole row.
 #include "common.cuh"
@@ -159,14 +161,14 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
                 if (tt >= count) break;
                 // log(sigmoid(z)) = min(z, 0) - log(1 + e^-|z|), exact at both ends
                 const float log_sig = fminf(z[tt], 0.f) - log1pf(expf(-fabsf(z[tt])));
-                decay[((size_t)(t_lo + tt) * H + h) * D + c] = form == 1 ? expf(-expf(z[tt])) : expf(log_sig * inv_tau);
+                decay[((size_t)(t_lo + tt) * H + h) * D + c] = form == 1 ? expm1f(-expf(z[tt])) : expf(log_sig * inv_tau);
             }
         }
     }
 }
 
-// q null: q, k and v stay where they are and only the decay is worked out.  form 0: sigmoid(z)^(1/tau); 1: exp(-exp(z)) over tanh of
-// the low-rank columns (tau is not used).
+// q null: q, k and v stay where they are and only the decay is worked out.  form 0: sigmoid(z)^(1/tau); 1: exp(-exp(z)) - 1 over tanh
+// of the low-rank columns (tau is not used).
 WLLM_API int wllm_linattn_prepare_form(const void* fused, int in_dtype, int row_stride, int parts, long long part_stride, int q_off,
                                        int k_off, int v_off, int a_off, int n, int H, int D, int V, int rank, const int* positions,
                                        const float* inv_freq, int rot_dim, float q_scale, float k_scale, const void* w2,
@@ -227,7 +229,7 @@ __device__ __forceinline__ void la_cp16(float* smem_dst, const float* src) {    
 // a time, and with two columns a lane every such read feeds eight multiply-adds; one column a lane and one channel
 // a read left the kernel waiting for shared memory (a read a multiply-add).
 // FULL: every warp holds LA_CPT channels (the head's key size is a multiple of 16): the loops carry no guards.
-// BONUS: the output is S_(t-1)^T q + (q . (u k)) v, taken channel by channel in front of the update.
+// BONUS: the output is S_(t-1)^T q + (q . (u k)) v, taken channel by channel in front of the update, and the decays are a - 1.
 // q, k and v are rows `q_stride`, `k_stride`, `v_stride` elements apart.
 template <bool PER_CHANNEL, int MODE, bool FULL, bool BONUS>
 __global__ void __launch_bounds__(512)
@@ -268,7 +270,7 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
         const bool ch = MODE != 1 && (FULL || c_lo + i < c_hi);
         S0[i] = (ch && col0) ? St[(size_t)(c_lo + i) * V + j0] : 0.f;
         S1[i] = (ch && col1) ? St[(size_t)(c_lo + i) * V + j1] : 0.f;
-        P[i] = 1.f;
+        P[i] = BONUS ? 0.f : 1.f;
         U[i] = BONUS && (FULL || c_lo + i < c_hi) ? bonus[h * D + c_lo + i] : 0.f;
     }
     const float fixed = PER_CHANNEL ? 0.f : head_decay[h];
@@ -356,9 +358,14 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
                                     p0[tt] = fmaf(fmaf(uk, v0, S0[i4 + e]), qe[e], p0[tt]);
                                     p1[tt] = fmaf(fmaf(uk, v1, S1[i4 + e]), qe[e], p1[tt]);
                                 }
-                                S0[i4 + e] = fmaf(ae[e], S0[i4 + e], ke[e] * v0);
-                                S1[i4 + e] = fmaf(ae[e], S1[i4 + e], ke[e] * v1);
-                                if (MODE == 1) P[i4 + e] *= ae[e];
+                                if (BONUS) {
+                                    S0[i4 + e] += fmaf(ae[e], S0[i4 + e], ke[e] * v0);
+                                    S1[i4 + e] += fmaf(ae[e], S1[i4 + e], ke[e] * v1);
+                                } else {
+                                    S0[i4 + e] = fmaf(ae[e], S0[i4 + e], ke[e] * v0);
+                                    S1[i4 + e] = fmaf(ae[e], S1[i4 + e], ke[e] * v1);
+                                }
+                                if (MODE == 1) P[i4 + e] = BONUS ? P[i4 + e] + fmaf(ae[e], P[i4 + e], ae[e]) : P[i4 + e] * ae[e];
                                 else if (!BONUS) {
                                     p0[tt] = fmaf(S0[i4 + e], qe[e], p0[tt]);
                                     p1[tt] = fmaf(S1[i4 + e], qe[e], p1[tt]);
@@ -420,7 +427,7 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
 // start states of the segments 1 .. nseg-1 of every request, in place of their local end states; grid (D*V / 256, H, requests)
 __global__ void linattn_combine_kernel(const float* __restrict__ state, const int* __restrict__ req_q_len,
                                        const int* __restrict__ req_slot, int H, int D, int V, int seg_len, int max_seg,
-                                       float* __restrict__ seg_state, const float* __restrict__ seg_decay) {
+                                       float* __restrict__ seg_state, const float* __restrict__ seg_decay, int minus_one) {
     pdl_begin();
     const int r = blockIdx.z, h = blockIdx.y;
     const int req_len = req_q_len[r], slot = req_slot[r];
@@ -433,7 +440,8 @@ __global__ void linattn_combine_kernel(const float* __restrict__ state, const in
     seg_state[((size_t)(r * max_seg) * H + h) * D * V + e] = cur;
     for (int sgm = 1; sgm < nseg; ++sgm) {
         const size_t at = (size_t)(r * max_seg + sgm) * H + h;
-        cur = fmaf(seg_decay[at * D + d], cur, seg_state[at * D * V + e]);
+        const float next = fmaf(seg_decay[at * D + d], cur, seg_state[at * D * V + e]);
+        cur = minus_one ? cur + next : next;
         seg_state[at * D * V + e] = cur;
     }
 }
@@ -443,7 +451,7 @@ __global__ void linattn_combine_kernel(const float* __restrict__ state, const in
 // seg_len > 0: portions longer than that are cut into segments that run side by side (at most max_seg a request, which
 // must cover the longest portion); seg_state holds requests * max_seg * H * D * V floats, seg_decay requests * max_seg * H * D.
 // q_stride, k_stride, v_stride: elements between two tokens' rows (H * D, H * D and H * V where the rows lie one behind the other).
-// bonus [H, D] (null: none): time mixing, see above; with a decay per key channel.
+// bonus [H, D] (null: none): time mixing, see above; with a decay per key channel, given as a - 1.
 WLLM_API int wllm_linattn_scan_rows(const float* q, const float* k, const float* v, long long q_stride, long long k_stride,
                                     long long v_stride, const float* decay, const float* head_decay, const float* bonus, float* state,
                                     float* out, const int* req_q_start, const int* req_q_len, const int* req_slot, int requests, int H,
@@ -467,7 +475,7 @@ WLLM_API int wllm_linattn_scan_rows(const float* q, const float* k, const float*
 #define RAISE(PC, M, B) if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_scan_kernel<PC, M, true, B>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); \
         if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_scan_kernel<PC, M, false, B>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)
         RAISE(true, 0, false); RAISE(true, 1, false); RAISE(true, 2, false); RAISE(false, 0, false); RAISE(false, 1, false); RAISE(false, 2, false);
-        RAISE(true, 0, true); RAISE(true, 2, true);
+        RAISE(true, 0, true); RAISE(true, 1, true); RAISE(true, 2, true);
 #undef RAISE
         if (e != cudaSuccess) return 1000 + (int)e;
         raised = true;
@@ -482,10 +490,10 @@ WLLM_API int wllm_linattn_scan_rows(const float* q, const float* k, const float*
         return SCAN(0, grid);
     }
     const dim3 grid(vtiles, H, requests * max_seg);
-    int st = decay ? SCAN1(true, 1, false, grid) : SCAN1(false, 1, false, grid);      // (no outputs yet: the bonus does not matter)
+    int st = SCAN(1, grid);
     if (st != WLLM_OK) return st;
     st = wllm_launch(linattn_combine_kernel, dim3((D * V + 255) / 256, H, requests), 256, 0, stream, (const float*)state,
-                     req_q_len, req_slot, H, D, V, seg_len, max_seg, seg_state, (const float*)seg_decay);
+                     req_q_len, req_slot, H, D, V, seg_len, max_seg, seg_state, (const float*)seg_decay, bonus != nullptr ? 1 : 0);
     if (st != WLLM_OK) return st;
     return SCAN(2, grid);
 #undef SCAN

@@ -5,11 +5,13 @@
 //     log a = -c r softplus(lam);          S_t = a S_(t-1) + sqrt(1 - a^2) i u;                  out_t = S_t gelu_tanh(in_y + b_y)
 //
 // in_y and in_x are columns of one projection row (possibly still in split-K slabs).  The convolution, the gates and the
-// recurrence are 32-bit.  The state S [W] and the last inputs x of the convolution live in the cache manager's state slots.  The
+// recurrence are 32-bit.  A channel that forgets slowly has a close to one, and what counts is how far it is from one: a - 1 is
+// carried instead of a (e = expm1(log a), S + (e S + b), 1 - a^2 = -e (2 + e)), so that its error is relative to itself and does
+// not grow with the memory.  The state S [W] and the last inputs x of the convolution live in the cache manager's state slots.  The
 // kept inputs are a ring of T rows: the input of position p lies in row p mod T, so a step of single tokens reads the rows of
 // the T - 1 positions before and writes its own without meeting another CTA's reads.  A position before the start counts as zero.
 //
-//   wllm_rglru_gates   a step's tokens: convolution and gates, (a, sqrt(1 - a^2) i u) as pairs [n, W, 2].  Two forms: the block
+//   wllm_rglru_gates   a step's tokens: convolution and gates, (a - 1, sqrt(1 - a^2) i u) as pairs [n, W, 2].  Two forms: the block
 //                      maps on the tensor cores (mma.sync, bfloat16 maps: u in two bfloat16 pieces, high and low, so that the product
 //                      keeps some sixteen bits of u), and plain 32-bit chains (32-bit maps, sizes in no step of 8).
 //   wllm_rglru_scan    the recurrence over every request's tokens from and to its slot, the output gate, and the slot's kept
@@ -140,12 +142,14 @@ __device__ __forceinline__ void rg_conv8(const RgInput& in, int t, int i, int sl
         for (int e = 0; e < 8; ++e) u[e] = fmaf(w[e], x[e], u[e]);
     }
 }
-// (a, sqrt(1 - a^2) i u) from the gates' sums
+// (a - 1, sqrt(1 - a^2) i u) from the gates' sums
 __device__ __forceinline__ float2 rg_pair(const RgGates& g, int c, float zr, float zi, float u) {
     const float r = rg_sigmoid(zr + g.ra_bias[c]), i = rg_sigmoid(zi + g.ri_bias[c]);
-    const float log_a = -g.c * r * rg_softplus(g.lam[c]);
-    return make_float2(expf(log_a), sqrtf(-expm1f(2.0f * log_a)) * (i * u));
+    const float e = expm1f(-g.c * r * rg_softplus(g.lam[c]));
+    return make_float2(e, sqrtf(-e * (2.0f + e)) * (i * u));
 }
+// one step of the recurrence from such a pair
+__device__ __forceinline__ float rg_advance(float S, float2 p) { return S + fmaf(p.x, S, p.y); }
 
 // ---------------------------------------------------------------------------------------------------
 // gates, plain: grid (blocks of channels x tiles of 32 of their channels, tiles of 32 tokens), 256 threads; thread (ty, tx) of
@@ -362,13 +366,13 @@ rglru_walk_kernel(RgInput in, const float2* __restrict__ ab, const int* __restri
         float2 p[8];
         float y[8];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) p[u] = k0 + u < len ? ab[(size_t)(t0 + k0 + u) * in.W + c] : make_float2(1.f, 0.f);
+        for (int u = 0; u < 8; ++u) p[u] = k0 + u < len ? ab[(size_t)(t0 + k0 + u) * in.W + c] : make_float2(0.f, 0.f);
 #pragma unroll
         for (int u = 0; u < 8; ++u) y[u] = k0 + u < len ? rg_y(in, t0 + k0 + u, c) : 0.f;
 #pragma unroll
         for (int u = 0; u < 8; ++u)
             if (k0 + u < len) {
-                S = fmaf(p[u].x, S, p[u].y);
+                S = rg_advance(S, p[u]);
                 out[(size_t)(t0 + k0 + u) * in.W + c] = from_f32<TO>(S * y[u]);
             }
     }
@@ -382,7 +386,7 @@ template <typename TO>
 __global__ void __launch_bounds__(RG_RUNS * RG_COLS)
 rglru_runs_kernel(RgInput in, const float2* __restrict__ ab, const int* __restrict__ req_q_len, float* __restrict__ state,
                   TO* __restrict__ out) {
-    __shared__ float2 local[2][RG_RUNS][RG_COLS];       // a run's decay product and its end state from zero
+    __shared__ float2 local[2][RG_RUNS][RG_COLS];       // a run's decay product minus one and its end state from zero
     pdl_begin();
     const int r = blockIdx.y, len = req_q_len[r], slot = in.req_slot[r];
     if (len <= 0 || slot < 0) return;
@@ -397,7 +401,7 @@ rglru_runs_kernel(RgInput in, const float2* __restrict__ ab, const int* __restri
 #pragma unroll
         for (int u = 0; u < RG_RUN; ++u) {
             const int k = tile * TILE + run * RG_RUN + u;
-            p[u] = k < len ? ab[(size_t)(t0 + k) * in.W + cc] : make_float2(1.f, 0.f);
+            p[u] = k < len ? ab[(size_t)(t0 + k) * in.W + cc] : make_float2(0.f, 0.f);
         }
     };
     const int tiles = (len + TILE - 1) / TILE;
@@ -413,22 +417,21 @@ rglru_runs_kernel(RgInput in, const float2* __restrict__ ab, const int* __restri
             y[u] = k < len ? rg_in(in.fused, in.dtype, in.parts, in.part_stride, (size_t)(t0 + k) * in.row_stride + in.y_off + cc) + in.y_bias[cc] : 0.f;
         }
         if (tile + 1 < tiles) load(tile + 1);           // on its way while this tile is walked
-        float A = 1.f, L = 0.f;
+        float A = 0.f, L = 0.f;
 #pragma unroll
-        for (int u = 0; u < RG_RUN; ++u) { L = fmaf(mine[u].x, L, mine[u].y); A *= mine[u].x; }
+        for (int u = 0; u < RG_RUN; ++u) { L = rg_advance(L, mine[u]); A = A + fmaf(mine[u].x, A, mine[u].x); }      // (1 + A)(1 + e) - 1
         local[tile & 1][run][col] = make_float2(A, L);
         __syncthreads();                                // (the buffer of the tile before is read to its end by the time this one is full)
         float S = carry, end = carry;
         for (int q = 0; q < RG_RUNS; ++q) {
-            const float2 al = local[tile & 1][q][col];
-            end = fmaf(al.x, end, al.y);
+            end = rg_advance(end, local[tile & 1][q][col]);
             if (q + 1 == run) S = end;
         }
         carry = end;
 #pragma unroll
         for (int u = 0; u < RG_RUN; ++u) {
             const int k = tile * TILE + run * RG_RUN + u;
-            S = fmaf(mine[u].x, S, mine[u].y);
+            S = rg_advance(S, mine[u]);
             if (k < len && live) out[(size_t)(t0 + k) * in.W + c] = from_f32<TO>(S * rg_gelu_tanh(y[u]));
         }
     }
@@ -541,7 +544,7 @@ rglru_step_kernel(RgInput in, RgGates g, int n, const int* __restrict__ req_q_le
             zi += red[((size_t)w * 2 * RS_COLS + RS_COLS + cc) * (RS_TOK + 1) + tt];
         }
         const float2 p = rg_pair(g, c, zr, zi, us[tt * RS_COLS + cc]);
-        const float S = fmaf(p.x, state[(size_t)slot * in.W + c], p.y);
+        const float S = rg_advance(state[(size_t)slot * in.W + c], p);
         state[(size_t)slot * in.W + c] = S;
         out[(size_t)t * in.W + c] = from_f32<TO>(S * rg_y(in, t, c));
         in.ring[((size_t)slot * in.T + in.positions[t] % in.T) * in.W + c] = rg_x(in, t, 0, slot, in.positions[t], 0, c);

@@ -1071,7 +1071,7 @@ def linattn_prepare(fused, parts: int, q_off: int, k_off: int, v_off: int, heads
 
 def linattn_decay(low: torch.Tensor, parts: int, low_off: int, w2: torch.Tensor, b2: torch.Tensor, heads: int, dim: int,
                   decay: torch.Tensor) -> torch.Tensor:
-    """The decay per key channel of time mixing, decay [n, heads*dim] = exp(-exp(w2 @ tanh(low) + b2)), where `low` are the
+    """The decay per key channel of time mixing, minus one: decay [n, heads*dim] = expm1(-exp(w2 @ tanh(low) + b2)), where `low` are the
     rank = w2.shape[1] columns of the projection `low` [n, W] (or partial sums [parts, n, W]) from `low_off`; 32-bit."""
     _need_cuda(low, w2, b2, decay)
     ptr, dt, row_stride, nparts, part_stride, n = _fused_args(low, parts)
@@ -1116,7 +1116,7 @@ def linattn_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay, head_
     with `head_decay` [heads].  With seg_len > 0 and max_seg > 1 (linattn_segment_plan) portions are cut into segments
     of seg_len tokens that run side by side; seg_state (requests * max_seg * heads * dim * vdim floats) and seg_decay
     (requests * max_seg * heads * dim) are their scratch.  q, k and v may be columns of wider rows.  `bonus` [heads*dim]
-    (time mixing): o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t, the output in front of the update."""
+    (time mixing): o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t, the output in front of the update; `decay` then holds a - 1."""
     _need_cuda(bonus, q, k, v, decay, head_decay, state, out, req_q_start, req_q_len, req_slot, seg_state, seg_decay)
     R = req_q_len.shape[0]
     if seg_len > 0 and max_seg > 1:
@@ -1273,7 +1273,7 @@ def moe_plan(chosen: torch.Tensor, count: torch.Tensor, offset: torch.Tensor, or
     assert offset.shape == (E + 1,) and order.shape == place.shape == (pairs,)
     for t in (chosen, count, offset, order, place):
         assert t.dtype == torch.int32 and t.is_contiguous()
-    assert tiles is None or (tiles.dtype == torch.int32 and tiles.is_contiguous() and tiles.numel() >= 1 + 3 * moe_row_tiles(pairs, E))
+    assert tiles is None or (tiles.dtype == torch.int32 and tiles.is_contiguous() and tiles.numel() >= 1 + 3 * moe_row_tiles(pairs, real_experts or E))
     lib = load_family("moe")
     assert scratch is None or (scratch.dtype == torch.int32 and scratch.is_contiguous() and scratch.numel() >= MOE_PLAN_SEGMENTS * E)
     _check(lib.wllm_moe_plan_real(_ptr(chosen), pairs, E, _ptr(count), _ptr(offset), _ptr(order), _ptr(place), _ptr(tiles),
@@ -1449,7 +1449,7 @@ def _rglru_gates(gates: dict, W: int) -> tuple:
 
 
 def rglru_gates(fused, parts: int, unit: dict, gates: dict, ctx, ring: torch.Tensor, ab: torch.Tensor) -> torch.Tensor:
-    """Convolution and gates of a real-gated linear recurrent unit (csrc/rg_lru.cu): ab [n, W, 2] = (a, sqrt(1 - a^2) i u), 32-bit."""
+    """Convolution and gates of a real-gated linear recurrent unit (csrc/rg_lru.cu): ab [n, W, 2] = (a - 1, sqrt(1 - a^2) i u), 32-bit."""
     args, n, W = _rglru_input(fused, parts, unit, ctx, ring)
     assert ab.dtype == torch.float32 and ab.shape == (n, W, 2) and ab.is_contiguous()
     lib = load_family("rg_lru")
@@ -1459,7 +1459,7 @@ def rglru_gates(fused, parts: int, unit: dict, gates: dict, ctx, ring: torch.Ten
 
 def rglru_scan(fused, parts: int, unit: dict, ctx, ring: torch.Tensor, ab: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
                long_portions: bool) -> torch.Tensor:
-    """S <- a S + b over every request's tokens of the step, from and to its row of `state` [slots, W]; out = S * gelu_tanh(y + bias) [n, W]; the
+    """S <- a S + b, with (a - 1, b) from `ab`, over every request's tokens of the step, from and to its row of `state` [slots, W]; out = S * gelu_tanh(y + bias) [n, W]; the
     convolution's newest inputs go to `ring`.  `long_portions`: runs of tokens side by side instead of token by token."""
     args, n, W = _rglru_input(fused, parts, unit, ctx, ring)
     assert ab.dtype == torch.float32 and ab.shape == (n, W, 2) and ab.is_contiguous() and out.shape == (n, W) and out.is_contiguous()
