@@ -134,8 +134,8 @@ def time_mixing(m, w, p, h, eps):
 
 
 def parallel(m, w, p, h, eps):
-    return float(m["left_scale"]) * attention(m["left"], w, p + "left.", h, eps) + \
-        float(m["right_scale"]) * time_mixing(m["right"], w, p + "right.", h, eps)
+    return float(m.get("left_scale", 1.0)) * attention(m["left"], w, p + "left.", h, eps) + \
+        float(m.get("right_scale", 1.0)) * time_mixing(m["right"], w, p + "right.", h, eps)
 
 
 def expert(w, p, h, limit):
