@@ -28,6 +28,11 @@ beside the like kernel of the Gemma layer.  One JSON line.
 
 Gudarax beside a Zafilix of equal layer sizes (the closest of the other designs), and its kernels one by one beside their like kernels.
 
+    python bench.py --design fusanex [--steps K] [--warmup W] [--batch 8] [--context 2048] [--sizes 2k,4k]
+
+Fusanex beside a Gudarax of equal layer sizes (the closest of the other designs: recurrences behind short convolutions, attention,
+routed experts in every layer), and its kernels one by one beside their like kernels.
+
     python bench.py --design taritar [--steps K] [--warmup W] [--batch 8] [--context 2048] [--sizes 2k,4k]
 
 the same for Taritar (several residual streams, attention with a score cap behind a window that keeps first keys, layers
@@ -1208,6 +1213,237 @@ def gudarax_bench(args) -> int:
     return 0
 
 
+FUSANEX_SIZES = {
+    # width, attention (heads, kv heads, head size), time mixing (heads, head size, rank), gated recurrence (channels, blocks, taps),
+    # experts (matrices, identity, chosen, feed-forward), the shared expert's feed-forward
+    "2k": dict(width=2048, attn=(16, 4, 128), mix=(32, 64, 64), lru=(2560, 10, 4), experts=(16, 4, 2, 2048), shared=2048, groups=2, vocab=32000),
+    "4k": dict(width=4096, attn=(32, 8, 128), mix=(64, 64, 128), lru=(4096, 16, 4), experts=(16, 4, 2, 3584), shared=4096, groups=2, vocab=32000),
+}
+
+
+def fusanex_config(size: dict) -> dict:
+    """Four layers: a gated recurrence, attention beside time mixing, and both again; routed experts with a shared one in every layer."""
+    nq, nkv, hd = size["attn"]
+    mh, md, rank = size["mix"]
+    W, blocks, taps = size["lru"]
+    E, identity, top, eff = size["experts"]
+    moe = {"kind": "moe", "expert": {"ff": eff, "limit": 7.0}, "router": {"experts": E, "top": top, "identity": identity},
+           "shared": {"ff": size["shared"], "limit": 7.0}}
+    lru = {"type": "rglru", "mixer": {"width": W, "blocks": blocks, "conv": taps}, "mlp": moe}
+    par = {"type": "parallel", "mlp": moe,
+           "mixer": {"left": {"heads": nq, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "q_temp": {"coef": 0.3, "every": 1024}},
+                     "right": {"heads": mh, "dim": md, "rank": rank}, "left_scale": 0.7, "right_scale": 0.7}}
+    return {"architecture": "Fusanex", "vocab": size["vocab"], "width": size["width"], "embedding": {"scale": 1.0},
+            "norm": {"eps": 1e-6, "groups": size["groups"]}, "layers": [lru, par, lru, par]}
+
+
+def fusanex_like_config(size: dict) -> dict:
+    """The closest of the other designs at equal sizes, a Gudarax of four layers: the delta rule (with short convolutions and as many state
+    elements as the time mixing) and attention alternating, routed experts of the same number and size behind all of them."""
+    nq, nkv, hd = size["attn"]
+    mh, md, _ = size["mix"]
+    E, _, top, eff = size["experts"]
+    moe = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}}
+    att = {"type": "attention", "mixer": {"heads": nq, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5}, "mlp": moe}
+    dlt = {"type": "delta", "mixer": {"heads": mh, "kv_heads": mh, "dim": md, "vdim": md, "conv": size["lru"][2]}, "mlp": moe}
+    return {"architecture": "Gudarax", "vocab": size["vocab"], "width": size["width"], "max_positions": 16384, "embedding": {"scale": 1.0},
+            "norm": {"eps": 1e-6}, "layers": [dlt, att, dlt, att]}
+
+
+def fusanex_kernel_table(size: dict, pk: dict, T: int, batch: int, context: int) -> dict:
+    """Fusanex's kernels alone at one size's shapes, each with its like kernel of the framework's other designs: microseconds, the time the
+    bytes each must move (or its arithmetic) take at the measured peaks (`floor_us`), how many times that it takes (`x_floor`), and, in a
+    design's own row, the like kernel's name and the ratio of the two `x_floor`."""
+    import torch
+    from types import SimpleNamespace
+    from wllm_b200.kernels import ops
+    dev, bf, f32, i32 = "cuda:0", torch.bfloat16, torch.float32, torch.int32
+    flush = torch.zeros(160 << 20, dtype=f32, device=dev)
+    H = size["width"]
+    nq, nkv, hd = size["attn"]
+    mh, md, rank = size["mix"]
+    W, blocks, taps = size["lru"]
+    E, identity, top, eff = size["experts"]
+    HD, ps = mh * md, 64
+    out = {}
+
+    def row(name, fn, bytes_moved, flops=0.0, like=None):
+        us = timed_us(fn, flush)
+        floor = max(bytes_moved / (pk["hbm_gbs"] * 1e3), flops / (pk["bf16_tflops"] * 1e6))
+        out[name] = {"us": round(us, 1), "floor_us": round(floor, 2), "x_floor": round(us / max(floor, 1e-9), 1)}
+        if like is not None:
+            out[name].update(like=like, ratio=round(us / max(floor, 1e-9) * out[like]["floor_us"] / out[like]["us"] if out[like]["floor_us"] else 0.0, 2))
+    g = torch.Generator(device=dev).manual_seed(1)
+
+    def rnd(*shape, dtype=f32, scale=1.0):
+        return (torch.randn(*shape, generator=g, device=dev, dtype=f32) * scale).to(dtype)
+    none = torch.empty(0, dtype=f32, device=dev)
+    ints = lambda v: torch.tensor(v, dtype=i32, device=dev)
+    pages = batch * (-(-(context + 1) // ps)) + -(-T // ps) + 1
+    kp, vp = rnd(pages, nkv, ps, hd, dtype=bf), rnd(pages, nkv, ps, hd, dtype=bf)
+    for n, tag in ((T, "prefill"), (batch, "decode")):
+        R = 1 if tag == "prefill" else batch
+        ctx = SimpleNamespace(positions=torch.arange(n, dtype=i32, device=dev) if R == 1 else ints([context] * n),
+                              token_req=ints([0] * n if R == 1 else list(range(n))), req_q_start=ints([0] if R == 1 else list(range(n))),
+                              req_q_len=ints([n] if R == 1 else [1] * n), req_slot=ints(list(range(R))))
+        slots = torch.arange(n, dtype=i32, device=dev)
+        # ---- norms: one pending branch and one norm; the design's two branches, two outputs, rows in groups
+        resid, gain, gain2 = rnd(n, H), rnd(H, dtype=bf), rnd(H, dtype=bf)
+        one_b, two_b = rnd(n, H, dtype=bf), rnd(n, H)
+        n1, n2 = torch.empty(n, H, dtype=bf, device=dev), torch.empty(n, H, dtype=bf, device=dev)
+        row(f"{tag}/norm of the residual with one branch folded in", lambda: ops.rmsnorm(resid, one_b, gain, 1e-6, 0.0, n1), n * H * (4 + 4 + 2 + 2))
+        row(f"{tag}/two norms in groups of the residual with two branches folded in",
+            lambda: ops.fold_norm(resid, [(one_b, 0, 0.7), (two_b, 0, 1.0)], [gain, gain2], 1e-6, [n1, n2], groups=size["groups"]),
+            n * H * (4 + 4 + 2 + 4 + 2 + 2), like=f"{tag}/norm of the residual with one branch folded in")
+        # ---- q | k | v into the pages
+        qkv, qo = rnd(n, (nq + 2 * nkv) * hd, dtype=bf), torch.empty(n, nq * hd, dtype=bf, device=dev)
+        hg = rnd(hd, dtype=bf)
+        moved = n * (nq + 2 * nkv) * hd * 2 * 2
+        row(f"{tag}/unit norms of q and k heads+cache write (no turn)",
+            lambda: ops.rope_kv_write(qkv, qo, ctx.positions, slots, none, kp, vp, nq, nkv, hd, 0, ps, unit_norm_eps=1e-6), moved)
+        row(f"{tag}/head norms with gains, normed values, query temperature+cache write",
+            lambda: ops.rope_head_norm_kv_write(qkv, qo, ctx.positions, slots, none, kp, vp, nq, nkv, hd, 0, ps, 1e-6, hg, hg, hd, hd, True, 0.3, 1024),
+            moved, like=f"{tag}/unit norms of q and k heads+cache write (no turn)")
+        # ---- short convolutions and gates: the delta rule's inputs, and the gated recurrence's
+        G = mh
+        off = {"q": 0, "k": HD, "v": 2 * HD, "g": 3 * HD, "b": 4 * HD, "a": 4 * HD + G}
+        conv = [rnd(HD, taps, dtype=bf) for _ in range(3)]
+        a_log, dt_bias = rnd(G, dtype=bf), rnd(G, dtype=bf)
+        dfused = rnd(n, 4 * HD + 2 * G, dtype=bf)
+        dq, dk, dv = (torch.empty(n, HD, device=dev) for _ in range(3))
+        beta, ddecay = torch.empty(n, G, device=dev), torch.empty(n, G, device=dev)
+        conv_state = torch.zeros(batch + 1, taps - 1, 3 * HD, device=dev)
+        row(f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)",
+            lambda: ops.delta_prepare(dfused, 0, off, G, G, md, md, taps, *conv, a_log, dt_bias, ctx.token_req, ctx.req_q_start, ctx.req_slot, conv_state,
+                                      1e-6, md ** -0.5, dq, dk, dv, beta, ddecay), n * (3 * HD + 2 * G) * (2 + 4))
+        dstate, do = torch.zeros(batch + 1, G, md, md, device=dev), torch.empty(n, HD, device=dev)
+        row(f"{tag}/delta rule: recurrence", lambda: ops.delta_scan(dq, dk, dv, beta, ddecay, dstate, do, ctx.req_q_start, ctx.req_q_len, ctx.req_slot, G, G, md, md),
+            n * (4 * HD + 2 * G) * 4 + R * 2 * G * md * md * 4, 6.0 * n * G * md * md)
+        s = W // blocks
+        fused = rnd(n, 2 * W, dtype=bf)
+        unit = dict(y_off=0, x_off=W, x_bias=rnd(W), y_bias=rnd(W), taps=rnd(taps, W), conv_bias=rnd(W))
+        gates = dict(ra=rnd(blocks, s, s, dtype=bf, scale=0.05), ri=rnd(blocks, s, s, dtype=bf, scale=0.05), ra_bias=rnd(W), ri_bias=rnd(W), lam=rnd(W), c=8.0)
+        ring, lstate = torch.zeros(batch + 1, taps, W, device=dev), torch.zeros(batch + 1, W, device=dev)
+        ab, lout = torch.empty(n, W, 2, device=dev), torch.empty(n, W, dtype=bf, device=dev)
+        maps = 2 * W * s * 2
+        if R == 1:
+            row(f"{tag}/gated recurrence: convolution and gates", lambda: ops.rglru_gates(fused, 0, unit, gates, ctx, ring, ab), n * W * (2 + 8) + maps,
+                2.0 * n * 2 * W * s, like=f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)")
+            row(f"{tag}/gated recurrence: runs side by side", lambda: ops.rglru_scan(fused, 0, unit, ctx, ring, ab, lstate, lout, True), n * W * (8 + 2 + 2),
+                like=f"{tag}/delta rule: recurrence")
+        else:
+            row(f"{tag}/gated recurrence: one step (convolution, gates, state, output gate)",
+                lambda: ops.rglru_step(fused, 0, unit, gates, ctx, ring, lstate, lout), n * W * (4 + 2 + 4 * (taps + 2)) + maps, 2.0 * n * 2 * W * s,
+                like=f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)")
+        # ---- time mixing: blends and their products, decay, recurrence with a bonus, head norm and gate
+        h, mu = rnd(n, H, dtype=bf), torch.rand(5, H, device=dev)
+        kept = rnd(batch + 1, 2, H, dtype=bf)
+        qkv_rows = (nq + 2 * nkv) * hd
+        w_all = rnd(qkv_rows + 4 * HD + rank, H, dtype=bf, scale=0.02)
+        if R == 1:
+            blends = torch.empty(5, n, H, dtype=bf, device=dev)
+            tiles = torch.empty(1 + 3 * ops.moe_row_tiles(4 * n, 4), dtype=i32, device=dev)
+            order = torch.randperm(5 * n, generator=g, device=dev).to(i32)
+            row(f"{tag}/experts: rows into sorted order (five a token)", lambda: ops.moe_gather(h, order, 5, blends.view(5 * n, H)), n * H * 2 * 6)
+            row(f"{tag}/blends of neighbouring tokens (five streams)", lambda: ops.token_blend(h, mu, ctx, kept, blends, tiles, 4), n * H * 2 * 6,
+                like=f"{tag}/experts: rows into sorted order (five a token)")
+            wide, rkvg = torch.empty(n, 4 * HD, dtype=bf, device=dev), torch.empty(4 * n, HD, device=dev)
+            w4 = w_all[qkv_rows:qkv_rows + 4 * HD]
+            row(f"{tag}/one product of that many columns", lambda: ops.gemm_bf16_tc(h, w4, wide), 4 * HD * H * 2 + n * (H + 4 * HD) * 2, 2.0 * n * 4 * HD * H)
+            row(f"{tag}/r, k, v, g: one grouped product of four blends", lambda: ops.gemm_bf16_tc_grouped(blends[:4].view(4 * n, H), w4.view(4, HD, H), rkvg, tiles, False),
+                4 * HD * H * 2 + 4 * n * (H * 2 + HD * 4), 2.0 * n * 4 * HD * H, like=f"{tag}/one product of that many columns")
+        else:
+            N = w_all.shape[0]
+            bufs = {}
+            row(f"{tag}/one product of that many columns", lambda: ops.project(h, w_all, lambda name, shape, dt: bufs.setdefault(name, torch.empty(shape, dtype=dt, device=dev))),
+                N * H * 2 + n * (H * 2 + N * 4), 2.0 * n * N * H)
+            fz = torch.empty(n, N, device=dev)
+            segments = [(qkv_rows, -1)] + [(HD, i) for i in range(4)] + [(rank, 4)]
+            row(f"{tag}/q, k, v and the products of five blends in one kernel", lambda: ops.blended_product(h, mu, w_all, segments, ctx, kept, fz),
+                N * H * 2 + n * (H * 2 * 2 + N * 4), 2.0 * n * N * H, like=f"{tag}/one product of that many columns")
+        r, k, v, gate = (rnd(n, HD) for _ in range(4))
+        low, w2, b2 = rnd(n, rank, dtype=bf), rnd(HD, rank, dtype=bf, scale=0.1), rnd(HD, dtype=bf)
+        decay = torch.empty(n, HD, device=dev)
+        lq, lk, lv = (torch.empty(n, HD, device=dev) for _ in range(3))
+        wide_la = rnd(n, 3 * HD + rank, dtype=bf)
+        row(f"{tag}/decayed state: inputs with the low-rank decay",
+            lambda: ops.linattn_prepare(wide_la, 0, 0, HD, 2 * HD, mh, md, md, ctx.positions, lq, lk, lv, low_off=3 * HD, w2=w2, b2=b2, tau=16.0, decay=decay),
+            n * (3 * HD * (2 + 4) + rank * 2 + HD * 4) + HD * rank * 2)
+        row(f"{tag}/time mixing: the decay", lambda: ops.linattn_decay(low, 0, 0, w2, b2, mh, md, decay), n * (rank * 2 + HD * 4) + HD * rank * 2,
+            like=f"{tag}/decayed state: inputs with the low-rank decay")
+        state, o = torch.zeros(batch + 1, mh, md, md, device=dev), torch.empty(n, HD, device=dev)
+        seg_len, max_seg = ops.linattn_segment_plan(n, 1, mh, md) if R == 1 else (0, 1)
+        ss, sd = torch.empty(R * max_seg * HD * md, device=dev), torch.empty(R * max_seg * HD, device=dev)
+        bonus, decay01 = rnd(HD), torch.rand(n, HD, device=dev) * 0.2 + 0.8
+        moved = n * 5 * HD * 4 + R * 2 * HD * md * 4
+        row(f"{tag}/decayed state: recurrence (decay per key channel)",
+            lambda: ops.linattn_scan(r, k, v, decay01, None, state, o, ctx.req_q_start, ctx.req_q_len, ctx.req_slot, mh, md, md, seg_len, max_seg, ss, sd), moved,
+            4.0 * n * HD * md)
+        minus = decay01 - 1.0
+        row(f"{tag}/time mixing: recurrence with a bonus",
+            lambda: ops.linattn_scan(r, k, v, minus, None, state, o, ctx.req_q_start, ctx.req_q_len, ctx.req_slot, mh, md, md, seg_len, max_seg, ss, sd, bonus=bonus),
+            moved, 4.0 * n * HD * md, like=f"{tag}/decayed state: recurrence (decay per key channel)")
+        both = torch.empty(n, nq * hd + HD, dtype=bf, device=dev)
+        plain_out = torch.empty(n, HD, dtype=bf, device=dev)
+        hw, rw = rnd(md, dtype=bf), rnd(HD, dtype=bf)
+        row(f"{tag}/head norm and gate", lambda: ops.head_gate_norm(o, gate, 0, 0, hw, 1e-6, plain_out, mh, md), n * HD * (4 + 4 + 2))
+        row(f"{tag}/head norm, gain of the whole row and gate, beside the attention's heads",
+            lambda: ops.head_gate_norm(o, gate, 0, 0, rw, 1e-6, both[:, nq * hd:], mh, md, 0.8), n * HD * (4 + 4 + 2), like=f"{tag}/head norm and gate")
+        # ---- experts
+        x = rnd(n, H, dtype=bf)
+        wr, corr = rnd(E + identity, H, scale=0.05), rnd(E + identity, scale=0.02)
+        chosen, weights = torch.empty(n, top, dtype=i32, device=dev), torch.empty(n, top, device=dev)
+        row(f"{tag}/router (softmax scores, choice)", lambda: ops.moe_route(x, wr, None, chosen, weights, None), n * H * 2 + (E + identity) * H * 4)
+        row(f"{tag}/router with a correction, weights over their sum",
+            lambda: ops.moe_route(x, wr, None, chosen, weights, None, correction=corr, renorm_eps=1e-20), n * H * 2 + (E + identity) * H * 4,
+            like=f"{tag}/router (softmax scores, choice)")
+        pairs, slots_e = n * top, E + identity
+        y, shared = rnd(pairs, H), rnd(n, H, dtype=bf)
+        place, sgate, o32 = torch.randperm(pairs, generator=g, device=dev).to(i32), torch.rand(n, device=dev), torch.empty(n, H, device=dev)
+        row(f"{tag}/experts' outputs weighted and summed, gated shared unit", lambda: ops.moe_combine(y, place, weights, (shared, 0), sgate, o32), pairs * H * 4 + n * H * (4 + 2))
+        own = int((chosen >= E).sum())
+        row(f"{tag}/experts' outputs weighted and summed, identity experts, shared unit",
+            lambda: ops.moe_combine(y, place, weights, (shared, 0), None, o32, chosen=chosen, real_experts=E, x=x),
+            (pairs - own) * H * 4 + own * H * 2 + n * H * (4 + 2), like=f"{tag}/experts' outputs weighted and summed, gated shared unit")
+    return out
+
+
+def fusanex_bench(args) -> int:
+    import torch
+    from wllm_b200.config import EngineConfig, FusanexConfig, GudaraxConfig
+    from wllm_b200.engine import build_model
+    pk = peaks()
+    ps, T = args.page_size, 2048
+    context = args.context or 2048
+    engine_cfg = EngineConfig(dtype="bfloat16", block_size=ps, max_num_seqs=max(64, args.batch), cuda_graphs=not args.no_graphs)
+    sizes = {}
+    for name in (args.sizes if args.sizes != "2b,7b" else "2k,4k").split(","):
+        size = FUSANEX_SIZES[name]
+        models = {"gudarax": GudaraxConfig.from_dict(fusanex_like_config(size)), "fusanex": FusanexConfig.from_dict(fusanex_config(size))}
+        res = {}
+        for label, cfg in models.items():
+            model = build_model(None, engine_cfg.dtype, engine_cfg.device, config=cfg, random_seed=1)
+            pre_ms = prefill_run(model, engine_cfg, T, ps)
+            ms, launches, _, clocks, _ = decode_run(model, engine_cfg, args.batch, context, min(args.steps, 32), args.warmup, ps, 3)
+            res[label] = {"weights_gb": round(model.weight_bytes() / 1e9, 3), "prefill_tok_s": round(T / (pre_ms / 1e3), 1),
+                          "prefill_ms": round(pre_ms, 3), "decode_tok_s": round(args.batch / (ms / 1e3), 1),
+                          "decode_ms_per_step": round(ms, 4), "decode_launches": launches,
+                          "decode_weights_hbm_frac": round(model.weight_bytes() / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 3), "clocks": clocks}
+            del model
+            torch.cuda.empty_cache()
+        sizes[name] = {"shape": size, "models": res}
+        if not args.no_points:
+            sizes[name]["kernels"] = fusanex_kernel_table(size, pk, T, args.batch, context)
+    print(json.dumps({"metric": "Fusanex beside Gudarax at equal layer sizes: prefill tok/s @ 2048 tokens, decode tok/s",
+                      "design": "fusanex", "unit": "tokens/s", "n_gpus": 1, "steps": min(args.steps, 32), "warmup": args.warmup,
+                      "dtype": "bf16", "data": "synthetic (random weights, random token ids, random cached keys/values)",
+                      "config": {"global_batch": args.batch, "seq_len": context, "prefill_tokens": T, "page_size": ps,
+                                 "cuda_graphs": not args.no_graphs, "peaks": pk["source"],
+                                 "l2": "kernel table: a 640 MB buffer is written before every timed launch"},
+                      "peaks": pk, "sizes": sizes}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1222,9 +1458,9 @@ def main() -> int:
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-points", action="store_true")
     ap.add_argument("--regions", type=int, default=5, help="timed regions of --steps steps each; the median is reported")
-    ap.add_argument("--design", default="gemma", choices=["gemma", "pesanex", "taritar", "zafilix", "gudarax"],
-                    help="gemma: the default workload; pesanex, taritar, zafilix, gudarax: models of that design beside a Gemma of equal layer sizes (another line)")
-    ap.add_argument("--sizes", default="2b,7b", help="which of the layer sizes to run (--design pesanex: 2b, 7b; taritar, zafilix, gudarax: 2k, 4k)")
+    ap.add_argument("--design", default="gemma", choices=["gemma", "pesanex", "taritar", "zafilix", "gudarax", "fusanex"],
+                    help="gemma: the default workload; the others: models of that design beside a model of an earlier design of equal layer sizes (another line)")
+    ap.add_argument("--sizes", default="2b,7b", help="which of the layer sizes to run (--design pesanex: 2b, 7b; the others: 2k, 4k)")
     args = ap.parse_args()
     if args.gpus != 1:
         print(f"bench.py: this engine runs on one GPU; --gpus {args.gpus} is not supported")
@@ -1240,6 +1476,8 @@ def main() -> int:
         return zafilix_bench(args)
     if args.design == "gudarax":
         return gudarax_bench(args)
+    if args.design == "fusanex":
+        return fusanex_bench(args)
     import torch
     from wllm_b200.config import EngineConfig, GemmaConfig
     from wllm_b200.engine import build_model
