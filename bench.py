@@ -1322,15 +1322,17 @@ def fusanex_kernel_table(size: dict, pk: dict, T: int, batch: int, context: int)
         s = W // blocks
         fused = rnd(n, 2 * W, dtype=bf)
         unit = dict(y_off=0, x_off=W, x_bias=rnd(W), y_bias=rnd(W), taps=rnd(taps, W), conv_bias=rnd(W))
-        gates = dict(ra=rnd(blocks, s, s, dtype=bf, scale=0.05), ri=rnd(blocks, s, s, dtype=bf, scale=0.05), ra_bias=rnd(W), ri_bias=rnd(W), lam=rnd(W), c=8.0)
+        gates = dict(maps=rnd(blocks, 2 * s, s, dtype=bf, scale=0.05).repeat(1, 1, 2), ra_bias=rnd(W), ri_bias=rnd(W), rate=rnd(W).abs())
         ring, lstate = torch.zeros(batch + 1, taps, W, device=dev), torch.zeros(batch + 1, W, device=dev)
-        ab, lout = torch.empty(n, W, 2, device=dev), torch.empty(n, W, dtype=bf, device=dev)
+        lout = torch.empty(n, W, dtype=bf, device=dev)
+        uv, z = torch.empty(blocks * n, 2 * s, dtype=bf, device=dev), torch.empty(blocks * n, 2 * s, device=dev)
+        ltiles = torch.empty(1 + 3 * ops.moe_row_tiles(blocks * n, blocks), dtype=i32, device=dev)
         maps = 2 * W * s * 2
         if R == 1:
-            row(f"{tag}/gated recurrence: convolution and gates", lambda: ops.rglru_gates(fused, 0, unit, gates, ctx, ring, ab), n * W * (2 + 8) + maps,
-                2.0 * n * 2 * W * s, like=f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)")
-            row(f"{tag}/gated recurrence: runs side by side", lambda: ops.rglru_scan(fused, 0, unit, ctx, ring, ab, lstate, lout, True), n * W * (8 + 2 + 2),
-                like=f"{tag}/delta rule: recurrence")
+            row(f"{tag}/gated recurrence: convolution and the gates' sums (two kernels)", lambda: ops.rglru_gate_sums(fused, 0, unit, gates, ctx, ring, uv, ltiles, z),
+                n * W * (2 + 4 + 4 + 8) + 2 * maps, 4.0 * n * 2 * W * s, like=f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)")
+            row(f"{tag}/gated recurrence: gates and runs side by side", lambda: ops.rglru_scan(fused, 0, unit, gates, ctx, ring, (z, uv), lstate, lout, True),
+                n * W * (8 + 4 + 2 + 2), like=f"{tag}/delta rule: recurrence")
         else:
             row(f"{tag}/gated recurrence: one step (convolution, gates, state, output gate)",
                 lambda: ops.rglru_step(fused, 0, unit, gates, ctx, ring, lstate, lout), n * W * (4 + 2 + 4 * (taps + 2)) + maps, 2.0 * n * 2 * W * s,

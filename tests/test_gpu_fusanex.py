@@ -4,8 +4,8 @@ Whole models: the residual after every layer; every way of cutting the work (who
 portions down to two tokens and one, mixed batches whose pages and state slots are used again), bit for bit against one
 another in 32-bit; long decoding; decoding from captured graphs; batches of unequal requests against each alone; one key far back
 or at a page's border that decides the logits; greedy generation through the scheduler; the trace runner.  Mechanisms alone: norms in
-groups of one residual with several branches folded in, head norms with gains and a temperature, the gated recurrence (both
-forms of its gates, all three of its walks, a write far back read much later), blends of neighbouring tokens and their products,
+groups of one residual with several branches folded in, head norms with gains and a temperature, the gated recurrence (all
+forms of its gates and of its walk, a write far back read much later), blends of neighbouring tokens and their products,
 the recurrence with a bonus, the router's correction and renormalised weights, identity experts.
 """
 import copy
@@ -406,7 +406,9 @@ def lru_unit(W, B, T, g, dtype):
     w = {k: v.to(torch.bfloat16).float() for k, v in w.items()}
     dev = lambda k: w[k].reshape(-1).contiguous().to(DEV)
     unit = dict(x_bias=dev("x.b"), y_bias=dev("y.b"), conv_bias=dev("conv.b"), taps=w["conv"].t().contiguous().to(DEV))
-    gates = dict(ra=w["ra"].to(dtype).to(DEV), ri=w["ri"].to(dtype).to(DEV), ra_bias=dev("ra.b"), ri_bias=dev("ri.b"), lam=dev("lam"), c=8.0)
+    maps = torch.cat([w["ra"], w["ri"]], 1)
+    gates = dict(maps=(torch.cat([maps, maps], 2) if dtype == torch.bfloat16 else maps).to(dtype).contiguous().to(DEV), ra_bias=dev("ra.b"),
+                 ri_bias=dev("ri.b"), rate=(8.0 * torch.nn.functional.softplus(w["lam"].double())).float().to(DEV))
     return w, unit, gates
 
 
@@ -422,7 +424,7 @@ def plain_lru(w, y, x):
 @pytest.mark.parametrize("W,B,T", [(48, 3, 4), (30, 3, 2), (21, 1, 5), (160, 1, 1), (256, 2, 4), (144, 2, 3)])
 def test_the_gated_recurrence_across_portions_and_slots(W, B, T, dtype):
     """Three requests in slots of a pool of six, in steps that cut them anywhere: portions shorter than the taps, single tokens (the one
-    kernel for them, and the two for portions, which must agree), long portions as runs side by side.  One early input is a hundred
+    kernel for them, and those for portions, which must agree), the gates' maps on the grouped product, long portions as runs side by side.  One early input is a hundred
     times the others and the slowest channels forget a few thousandths of their state in a hundred tokens, so it still shows at the end.
     The slots of nobody stay as they were."""
     from wllm_b200.kernels import ops
@@ -460,16 +462,22 @@ def test_the_gated_recurrence_across_portions_and_slots(W, B, T, dtype):
             forms.append((parts.to(DEV), 3))
             answers = []
             for fused, p in forms:
-                ways = [False] + ([True] if max(lens) == 1 and ops.rglru_step_ok(gates, fused, off) else [])
-                for step in ways:
-                    rg, st, out = ring.clone(), state.clone(), torch.empty(n, W, dtype=dtype, device=DEV)
-                    if step:
-                        ops.rglru_step(fused, p, unit, gates, ctx, rg, st, out)
-                    else:
-                        ab = torch.empty(n, W, 2, device=DEV)
-                        ops.rglru_gates(fused, p, unit, gates, ctx, rg, ab)
-                        ops.rglru_scan(fused, p, unit, ctx, rg, ab, st, out, max(lens) >= ops.RGLRU_RUNS_FROM)
-                    answers.append((out, rg, st))
+                ways = ["pairs"] + (["step"] if max(lens) == 1 and ops.rglru_step_ok(gates, fused, off) else []) + \
+                    (["grouped"] if ops.rglru_grouped_ok(gates, fused, off) else [])
+                for way in ways:
+                    for long in {max(lens) >= ops.RGLRU_RUNS_FROM, way == "grouped"}:
+                        rg, st, out = ring.clone(), state.clone(), torch.empty(n, W, dtype=dtype, device=DEV)
+                        if way == "step":
+                            ops.rglru_step(fused, p, unit, gates, ctx, rg, st, out)
+                        elif way == "pairs":
+                            ab = torch.empty(n, W, 2, device=DEV)
+                            ops.rglru_gates(fused, p, unit, gates, ctx, rg, ab)
+                            ops.rglru_scan(fused, p, unit, gates, ctx, rg, ab, st, out, long)
+                        else:
+                            uv, z = torch.empty(B * n, 2 * W // B, dtype=dtype, device=DEV), torch.empty(B * n, 2 * W // B, device=DEV)
+                            ops.rglru_gate_sums(fused, p, unit, gates, ctx, rg, uv, torch.empty(1 + 3 * ops.moe_row_tiles(B * n, B), dtype=torch.int32, device=DEV), z)
+                            ops.rglru_scan(fused, p, unit, gates, ctx, rg, (z, uv), st, out, long)
+                        answers.append((out, rg, st))
             for out, rg, st in answers[1:]:
                 tol = 2e-4 if dtype == torch.float32 else 0.02
                 big = max(1.0, float(answers[0][0].abs().max()))
@@ -575,8 +583,9 @@ def test_the_recurrence_with_a_bonus(H, D):
     rows = torch.randn(n, wide, generator=g)
     rows[2, H * D:2 * H * D] *= 30
     r, k, v = (rows[:, i * H * D:(i + 1) * H * D] for i in range(3))
-    low, rank = torch.randn(n, 12, generator=g), 9
-    w2, b2 = torch.randn(H * D, rank, generator=g), torch.rand(H * D, generator=g) * 8 - 8
+    rank = {24: 9, 10: 5, 64: 16, 128: 64}[D]
+    low = torch.randn(n, rank + 3, generator=g)
+    w2, b2 = torch.randn(H * D, rank, generator=g) * (9 / rank) ** 0.5, torch.rand(H * D, generator=g) * 8 - 8
     bonus = torch.randn(H * D, generator=g) * 4
     decay = torch.exp(-torch.exp(torch.tanh(low[:, 2:2 + rank].double()) @ w2.double().T + b2.double()))
     shaped = lambda t: t.double().view(n, H, D)
@@ -585,6 +594,15 @@ def test_the_recurrence_with_a_bonus(H, D):
     rd, kd, vd = (dev[:, i * H * D:(i + 1) * H * D] for i in range(3))
     dd = ops.linattn_decay(low.to(DEV), 0, 2, w2.to(DEV), b2.to(DEV), H, D, torch.empty(n, H * D, device=DEV))
     assert (dd.cpu().double() + 1 - decay).abs().max() < 1e-6
+    if rank % 8 == 0:          # many tokens, bfloat16 maps: the tensor-core form, from one tensor and from partial sums
+        wb, bb = w2.bfloat16(), b2.bfloat16()
+        ref = torch.expm1(-torch.exp(torch.tanh(low[:, 2:2 + rank].double()) @ wb.double().T + bb.double()))
+        slabs = torch.randn(3, n, rank + 3, generator=g)
+        slabs[-1] = low - slabs[:-1].sum(0)
+        for src, parts in ((low, 0), (slabs, 3)):
+            for m in (n, 70, 20):
+                got = ops.linattn_decay(src[..., :m, :].contiguous().to(DEV), parts, 2, wb.to(DEV), bb.to(DEV), H, D, torch.empty(m, H * D, device=DEV))
+                assert ((got.cpu().double() - ref[:m]) / ref[:m]).abs().max() < 2e-3, (parts, m)
     small = decay > 0.999
     assert bool(small.any()) and ((dd.cpu().double() - (decay - 1))[small] / (decay - 1)[small]).abs().max() < 1e-5     # relative to itself
     for cuts, seg in (([n], 0), ([n], 32), ([100, 1, 2, 157], 0), ([130, 130], 48)):

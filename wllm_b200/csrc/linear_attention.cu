@@ -167,6 +167,92 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
     }
 }
 
+// The decay of time mixing for many tokens, bfloat16 maps, on the tensor cores (mma.sync): a CTA takes 64 tokens, whose tanh'd low-rank
+// rows it holds in shared memory as a high and a low bfloat16 piece each (together some sixteen bits), and walks tiles of 128
+// channels; 2 x 4 warps, 32 tokens by 32 channels each.  grid (CTAs that share the channels' tiles, tiles of tokens), 256 threads.
+constexpr int DEC_TM = 64, DEC_TN = 128, DEC_MAX_RANK = 256;
+
+__device__ __forceinline__ void dec_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void dec_ldsm4(const bf16* p, uint32_t (&r)[4]) {
+    const unsigned addr = (unsigned)__cvta_generic_to_shared(p);
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+
+template <bool MULTI>
+__global__ void __launch_bounds__(256)
+linattn_decay_mma_kernel(const void* __restrict__ low, int in_dtype, int row_stride, int parts, size_t part_stride, int a_off, int n, int HD,
+                         int rank, const bf16* __restrict__ w2, const bf16* __restrict__ b2, float* __restrict__ decay) {
+    extern __shared__ __align__(16) unsigned char dec_smem[];
+    const int kp = (rank + 15) & ~15, pitch = kp + 8;
+    bf16* hi = reinterpret_cast<bf16*>(dec_smem);        // [64][pitch]
+    bf16* lo = hi + DEC_TM * pitch;
+    bf16* ws = lo + DEC_TM * pitch;                      // [128][pitch]
+    pdl_begin();
+    const int t0 = blockIdx.y * DEC_TM, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wm = warp & 1, wn = warp >> 1;
+    for (int idx = threadIdx.x; idx < DEC_TM * kp; idx += 256) {
+        const int tt = idx / kp, r = idx - tt * kp;
+        float v = 0.f;
+        if (t0 + tt < n && r < rank) v = tanhf(la_in<MULTI>(low, in_dtype, parts, part_stride, (size_t)(t0 + tt) * row_stride + a_off + r));
+        const bf16 h = __float2bfloat16_rn(v);
+        hi[tt * pitch + r] = h;
+        lo[tt * pitch + r] = __float2bfloat16_rn(v - __bfloat162float(h));
+    }
+    const int tiles = (HD + DEC_TN - 1) / DEC_TN;
+    for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x) {
+        __syncthreads();                                 // the tokens' rows are here; the tile before is read to its end
+        for (int idx = threadIdx.x; idx < DEC_TN * (kp / 8); idx += 256) {
+            const int c = idx / (kp / 8), k = (idx % (kp / 8)) * 8, ch = tile * DEC_TN + c;
+            *reinterpret_cast<uint4*>(ws + c * pitch + k) =
+                (ch < HD && k < rank) ? *reinterpret_cast<const uint4*>(w2 + (size_t)ch * rank + k) : make_uint4(0u, 0u, 0u, 0u);
+        }
+        __syncthreads();
+        float acc[2][4][4];
+#pragma unroll
+        for (int mi = 0; mi < 2; ++mi)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[mi][j][0] = acc[mi][j][1] = acc[mi][j][2] = acc[mi][j][3] = 0.f;
+        for (int k = 0; k < kp; k += 16) {
+            uint32_t ah[2][4], al[2][4], bw[2][4];
+#pragma unroll
+            for (int mi = 0; mi < 2; ++mi) {
+                const int at = (wm * 32 + mi * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * pitch + k + (lane >> 4) * 8;
+                dec_ldsm4(hi + at, ah[mi]);
+                dec_ldsm4(lo + at, al[mi]);
+            }
+#pragma unroll
+            for (int nj = 0; nj < 2; ++nj)
+                dec_ldsm4(ws + (wn * 32 + nj * 16 + (lane & 7) + (lane >> 4) * 8) * pitch + k + ((lane >> 3) & 1) * 8, bw[nj]);
+#pragma unroll
+            for (int mi = 0; mi < 2; ++mi)
+#pragma unroll
+                for (int nj = 0; nj < 2; ++nj) {
+                    dec_mma(acc[mi][2 * nj], al[mi], bw[nj][0], bw[nj][1]);
+                    dec_mma(acc[mi][2 * nj + 1], al[mi], bw[nj][2], bw[nj][3]);
+                    dec_mma(acc[mi][2 * nj], ah[mi], bw[nj][0], bw[nj][1]);
+                    dec_mma(acc[mi][2 * nj + 1], ah[mi], bw[nj][2], bw[nj][3]);
+                }
+        }
+#pragma unroll
+        for (int mi = 0; mi < 2; ++mi)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                const int t = t0 + wm * 32 + mi * 16 + (lane >> 2) + half * 8;
+                if (t >= n) continue;
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const int ch = tile * DEC_TN + wn * 32 + j * 8 + (lane & 3) * 2 + e;
+                        if (ch < HD) decay[(size_t)t * HD + ch] = expm1f(-expf(acc[mi][j][half * 2 + e] + __bfloat162float(b2[ch])));
+                    }
+            }
+    }
+}
+
 // q null: q, k and v stay where they are and only the decay is worked out.  form 0: sigmoid(z)^(1/tau); 1: exp(-exp(z)) - 1 over tanh
 // of the low-rank columns (tau is not used).
 WLLM_API int wllm_linattn_prepare_form(const void* fused, int in_dtype, int row_stride, int parts, long long part_stride, int q_off,
@@ -179,6 +265,23 @@ WLLM_API int wllm_linattn_prepare_form(const void* fused, int in_dtype, int row_
     if (a_off >= 0 && (rank <= 0 || !(tau > 0.f) || !w2 || !b2 || !decay)) return WLLM_BAD_SIZE;
     if ((in_dtype != WLLM_BF16 && in_dtype != WLLM_F32) || (a_off >= 0 && w_dtype != WLLM_BF16 && w_dtype != WLLM_F32))
         return WLLM_BAD_DTYPE;
+    if (q == nullptr && form == 1 && a_off >= 0 && n >= 64 && w_dtype == WLLM_BF16 && rank % 8 == 0 && rank <= DEC_MAX_RANK && ((uintptr_t)w2 & 15) == 0) {
+        const int HD = H * D, row_tiles = (n + DEC_TM - 1) / DEC_TM, col_tiles = (HD + DEC_TN - 1) / DEC_TN;
+        int share = (2 * 148 + row_tiles - 1) / row_tiles;           // CTAs that share a tile of tokens: some two CTAs an SM in all
+        if (share > col_tiles) share = col_tiles;
+        const size_t smem = (size_t)(2 * DEC_TM + DEC_TN) * (((rank + 15) & ~15) + 8) * sizeof(bf16);
+        static bool raised = false;
+        if (!raised) {
+            cudaError_t e = cudaFuncSetAttribute(linattn_decay_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+            if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_decay_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+            if (e != cudaSuccess) return 1000 + (int)e;
+            raised = true;
+        }
+#define DEC(M) wllm_launch(linattn_decay_mma_kernel<M>, dim3(share, row_tiles), 256, smem, stream, fused, in_dtype, row_stride, parts, \
+        (size_t)part_stride, a_off, n, HD, rank, (const bf16*)w2, (const bf16*)b2, decay)
+        return parts > 1 ? DEC(true) : DEC(false);
+#undef DEC
+    }
 #define PREP2(TT, M) wllm_launch(linattn_prepare_kernel<TT, M>, dim3((n + TT - 1) / TT, H), 128, 0, stream, fused, \
         in_dtype, row_stride, parts, (size_t)part_stride, q_off, k_off, v_off, a_off, n, H, D, V, rank, positions, \
         inv_freq, rot_dim, q_scale, k_scale, w2, b2, w_dtype, a_off >= 0 ? 1.0f / tau : 0.f, q, k, v, decay, form)
@@ -510,14 +613,15 @@ WLLM_API int wllm_linattn_scan(const float* q, const float* k, const float* v, c
 }
 
 // ---------------------------------------------------------------------------------------------------
-// head norm and gate: grid (tokens, heads), one warp
+// head norm and gate: grid (tokens, groups of four heads), a warp a head
 // ---------------------------------------------------------------------------------------------------
 template <typename TO, bool MULTI>
 __global__ void head_gate_norm_kernel(const float* __restrict__ o, const void* __restrict__ fused, int in_dtype, int row_stride,
                                       int parts, size_t part_stride, int g_off, const void* __restrict__ w, int w_dtype,
                                       float eps, TO* __restrict__ out, int H, int V, int w_head_stride, size_t out_stride, float factor) {
     pdl_begin();
-    const int t = blockIdx.x, h = blockIdx.y, lane = threadIdx.x;
+    const int t = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (h >= H) return;
     const float* orow = o + ((size_t)t * H + h) * V;
     float ss = 0.f;
     for (int c = lane; c < V; c += 32) ss = fmaf(orow[c], orow[c], ss);
@@ -540,7 +644,7 @@ WLLM_API int wllm_head_gate_norm_rows(const float* o, const void* fused, int in_
     if (n <= 0) return WLLM_OK;
     if (H <= 0 || H > 65535 || V <= 0 || parts < 1 || out_stride < H * V) return WLLM_BAD_SIZE;
     if ((in_dtype != WLLM_BF16 && in_dtype != WLLM_F32) || (w && w_dtype != WLLM_BF16 && w_dtype != WLLM_F32)) return WLLM_BAD_DTYPE;
-#define GATE(TO, M) wllm_launch(head_gate_norm_kernel<TO, M>, dim3(n, H), 32, 0, stream, o, fused, in_dtype, row_stride, parts, \
+#define GATE(TO, M) wllm_launch(head_gate_norm_kernel<TO, M>, dim3(n, (H + 3) / 4), 128, 0, stream, o, fused, in_dtype, row_stride, parts, \
         (size_t)part_stride, g_off, w, w_dtype, eps, (TO*)out, H, V, per_head ? V : 0, (size_t)out_stride, factor)
     if (out_dtype == WLLM_BF16) return parts > 1 ? GATE(bf16, true) : GATE(bf16, false);
     if (out_dtype == WLLM_F32) return parts > 1 ? GATE(float, true) : GATE(float, false);

@@ -14,10 +14,14 @@
 //   wllm_rglru_gates   a step's tokens: convolution and gates, (a - 1, sqrt(1 - a^2) i u) as pairs [n, W, 2].  Two forms: the block
 //                      maps on the tensor cores (mma.sync, bfloat16 maps: u in two bfloat16 pieces, high and low, so that the product
 //                      keeps some sixteen bits of u), and plain 32-bit chains (32-bit maps, sizes in no step of 8).
+//   wllm_rglru_conv    many tokens, bfloat16 maps: the convolution alone, u as its two pieces in the layout that the grouped
+//                      tensor-memory product (gemm_bf16_tc.cu) reads: a group a block, rows [high | low] of 2 s elements, times the
+//                      block's rows [R R; I I] gives both gates' sums in 32-bit.  It writes that product's table of row tiles too.
 //   wllm_rglru_scan    the recurrence over every request's tokens from and to its slot, the output gate, and the slot's kept
-//                      inputs.  Short portions: a thread a channel walks the tokens.  Long ones: 32 runs of 8 tokens at a time; a run's
-//                      decay product and end state from zero come first, then its true start state from the runs before it, then
-//                      its outputs; all of it from registers, so the pairs are read once.
+//                      inputs, from the pairs or from the gates' sums and u's pieces.  Short portions: a thread a channel walks the
+//                      tokens.  Long ones: 64 runs of 8 tokens at a time; a run's decay product and end state from zero come first,
+//                      then its true start state from the runs before it, then its outputs; all of it from registers, so that
+//                      everything is read once.
 //   wllm_rglru_step    both at once for a step in which no request brings more than one token (decoding).
 #include "common.cuh"
 
@@ -74,7 +78,6 @@ __device__ __forceinline__ void rg_f8(const float* p, float (&v)[8]) {
     v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
 }
 __device__ __forceinline__ float rg_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float rg_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ float rg_gelu_tanh(float x) {
     const float k = 0.7978845608028654f;  // sqrt(2/pi)
     return 0.5f * x * (1.0f + tanhf(k * (x + 0.044715f * x * x * x)));
@@ -99,13 +102,13 @@ struct RgInput {
 };
 // gates' parameters
 struct RgGates {
-    const void* ra;           // [B][s][s], [out, in]
+    const void* ra;           // B blocks of s rows of s elements ([out, in]), `pitch` elements from row to row, `block` from block to block
     const void* ri;
-    int w_dtype;
+    int w_dtype, pitch;
+    size_t block;
     const float* ra_bias;     // [W]
     const float* ri_bias;
-    const float* lam;         // [W]
-    float c;                  // log a = -c r softplus(lam)
+    const float* rate;        // [W] c softplus(lam): log a = -rate r
     int B, s;
 };
 
@@ -145,7 +148,7 @@ __device__ __forceinline__ void rg_conv8(const RgInput& in, int t, int i, int sl
 // (a - 1, sqrt(1 - a^2) i u) from the gates' sums
 __device__ __forceinline__ float2 rg_pair(const RgGates& g, int c, float zr, float zi, float u) {
     const float r = rg_sigmoid(zr + g.ra_bias[c]), i = rg_sigmoid(zi + g.ri_bias[c]);
-    const float e = expm1f(-g.c * r * rg_softplus(g.lam[c]));
+    const float e = expm1f(-g.rate[c] * r);
     return make_float2(e, sqrtf(-e * (2.0f + e)) * (i * u));
 }
 // one step of the recurrence from such a pair
@@ -171,7 +174,7 @@ rglru_gates_plain_kernel(RgInput in, RgGates g, int n, float2* __restrict__ ab) 
         for (int idx = threadIdx.x; idx < TN * TK; idx += 256) {
             const int c = idx / TK, k = idx % TK;
             const bool ok = col0 + c < g.s && k0 + k < g.s;
-            const size_t at = ((size_t)base + col0 + c) * g.s + k0 + k;
+            const size_t at = b * g.block + (size_t)(col0 + c) * g.pitch + k0 + k;
             Wr[k][c] = ok ? rg_any(g.ra, g.w_dtype, at) : 0.f;
             Wi[k][c] = ok ? rg_any(g.ri, g.w_dtype, at) : 0.f;
         }
@@ -247,7 +250,7 @@ rglru_gates_mma_kernel(RgInput in, RgGates g, int n, float2* __restrict__ ab) {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
         const int r = (threadIdx.x >> 2) + 64 * h, col = col0 + 16 * (r >> 5) + (r & 15);
-        w_src[h] = col < g.s ? reinterpret_cast<const bf16*>((r >> 4) & 1 ? g.ri : g.ra) + ((size_t)base + col) * g.s : nullptr;
+        w_src[h] = col < g.s ? reinterpret_cast<const bf16*>((r >> 4) & 1 ? g.ri : g.ra) + b * g.block + (size_t)col * g.pitch : nullptr;
     }
     auto load_w = [&](int kb, int buf) {
         const int k = kb * RG_TK + w_piece * 8;
@@ -339,9 +342,50 @@ rglru_gates_mma_kernel(RgInput in, RgGates g, int n, float2* __restrict__ ab) {
         }
 }
 
+// the convolution alone: grid (tiles of 4 tokens, tiles of 512 channels), 256 threads = 4 tokens by 64 runs of eight channels.
+// uv [B][n][2 s]; tiles (null: none): the table of row tiles of `tile_rows` rows of one block each
+__global__ void __launch_bounds__(256)
+rglru_conv_kernel(RgInput in, int n, int B, int s, bf16* __restrict__ uv, int* __restrict__ tiles, int tile_rows) {
+    pdl_begin();
+    if (tiles != nullptr && blockIdx.x == 0 && blockIdx.y == 0) {
+        const int per = (n + tile_rows - 1) / tile_rows;
+        for (int i = threadIdx.x; i < B * per; i += blockDim.x) {
+            const int b = i / per, k = i % per;
+            tiles[1 + 3 * i] = b;
+            tiles[2 + 3 * i] = b * n + k * tile_rows;
+            tiles[3 + 3 * i] = min(tile_rows, n - k * tile_rows);
+        }
+        if (threadIdx.x == 0) tiles[0] = B * per;
+    }
+    const int t = blockIdx.x * 4 + (threadIdx.x >> 6), c = (blockIdx.y * 64 + (threadIdx.x & 63)) * 8;
+    if (t >= n || c >= in.W) return;
+    const int r = in.token_req[t];
+    float u[8];
+    rg_conv8(in, t, t - in.req_q_start[r], max(in.req_slot[r], 0), in.positions[t], c, u);
+    uint4 hi, lo;
+    rg_split2(u[0], u[1], hi.x, lo.x); rg_split2(u[2], u[3], hi.y, lo.y);
+    rg_split2(u[4], u[5], hi.z, lo.z); rg_split2(u[6], u[7], hi.w, lo.w);
+    bf16* dst = uv + ((size_t)(c / s) * n + t) * 2 * s + c % s;          // (s is a multiple of 8: the eight channels share a block)
+    *reinterpret_cast<uint4*>(dst) = hi;
+    *reinterpret_cast<uint4*>(dst + s) = lo;
+}
+
 // ---------------------------------------------------------------------------------------------------
 // scan
 // ---------------------------------------------------------------------------------------------------
+// where the recurrence finds a token's pair: made already, or the gates' sums z [B][n][2 s] (R's s, then I's) and u's pieces
+struct RgPairs {
+    const float2* ab;
+    const float* z;
+    const bf16* uv;
+    int n, s;
+};
+template <bool MADE>
+__device__ __forceinline__ float2 rg_pair_at(const RgPairs& src, const RgGates& g, int W, int t, int c) {
+    if (MADE) return src.ab[(size_t)t * W + c];
+    const size_t at = ((size_t)(c / src.s) * src.n + t) * 2 * src.s + c % src.s;
+    return rg_pair(g, c, src.z[at], src.z[at + src.s], __bfloat162float(src.uv[at]) + __bfloat162float(src.uv[at + src.s]));
+}
 // the newest inputs of the convolution after this step: rows of the ring (positions base + len - T .. base + len - 1)
 __device__ __forceinline__ void rg_keep_inputs(const RgInput& in, int t0, int len, int slot, int first_pos, int c) {
     for (int k = max(0, len - in.T); k < len; ++k)
@@ -353,10 +397,9 @@ __device__ __forceinline__ float rg_y(const RgInput& in, int t, int c) {
 }
 
 // a thread a channel: grid (ceil(W / 128), requests)
-template <typename TO>
+template <typename TO, bool MADE>
 __global__ void __launch_bounds__(128)
-rglru_walk_kernel(RgInput in, const float2* __restrict__ ab, const int* __restrict__ req_q_len, float* __restrict__ state,
-                  TO* __restrict__ out) {
+rglru_walk_kernel(RgInput in, RgGates g, RgPairs src, const int* __restrict__ req_q_len, float* __restrict__ state, TO* __restrict__ out) {
     pdl_begin();
     const int r = blockIdx.y, len = req_q_len[r], slot = in.req_slot[r], c = blockIdx.x * 128 + threadIdx.x;
     if (len <= 0 || slot < 0 || c >= in.W) return;
@@ -366,7 +409,7 @@ rglru_walk_kernel(RgInput in, const float2* __restrict__ ab, const int* __restri
         float2 p[8];
         float y[8];
 #pragma unroll
-        for (int u = 0; u < 8; ++u) p[u] = k0 + u < len ? ab[(size_t)(t0 + k0 + u) * in.W + c] : make_float2(0.f, 0.f);
+        for (int u = 0; u < 8; ++u) p[u] = k0 + u < len ? rg_pair_at<MADE>(src, g, in.W, t0 + k0 + u, c) : make_float2(0.f, 0.f);
 #pragma unroll
         for (int u = 0; u < 8; ++u) y[u] = k0 + u < len ? rg_y(in, t0 + k0 + u, c) : 0.f;
 #pragma unroll
@@ -380,59 +423,61 @@ rglru_walk_kernel(RgInput in, const float2* __restrict__ ab, const int* __restri
     rg_keep_inputs(in, t0, len, slot, in.positions[t0], c);
 }
 
-// runs side by side: grid (ceil(W / 16), requests), 512 threads = 32 runs of 8 tokens by 16 channels
-constexpr int RG_RUNS = 32, RG_RUN = 8, RG_COLS = 16;
-template <typename TO>
+// runs side by side: grid (ceil(W / 8), requests), 512 threads = 64 runs of 8 tokens by 8 channels; a warp has four runs
+constexpr int RG_RUNS = 64, RG_RUN = 8, RG_COLS = 8, RG_WARPS = RG_RUNS * RG_COLS / 32;
+// two stretches of the recurrence one behind the other, each as (decay product - 1, end state from zero)
+__device__ __forceinline__ float2 rg_join(float2 first, float2 second) {
+    return make_float2(first.x + fmaf(second.x, first.x, second.x), rg_advance(first.y, second));
+}
+template <typename TO, bool MADE>
 __global__ void __launch_bounds__(RG_RUNS * RG_COLS)
-rglru_runs_kernel(RgInput in, const float2* __restrict__ ab, const int* __restrict__ req_q_len, float* __restrict__ state,
-                  TO* __restrict__ out) {
-    __shared__ float2 local[2][RG_RUNS][RG_COLS];       // a run's decay product minus one and its end state from zero
+rglru_runs_kernel(RgInput in, RgGates g, RgPairs src, const int* __restrict__ req_q_len, float* __restrict__ state, TO* __restrict__ out) {
+    __shared__ float2 local[2][RG_WARPS][RG_COLS];       // a warp's four runs joined
     pdl_begin();
     const int r = blockIdx.y, len = req_q_len[r], slot = in.req_slot[r];
     if (len <= 0 || slot < 0) return;
     const int run = threadIdx.x / RG_COLS, col = threadIdx.x % RG_COLS, c = blockIdx.x * RG_COLS + col;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool live = c < in.W;
     const int cc = live ? c : in.W - 1;
     const int t0 = in.req_q_start[r];
     float carry = state[(size_t)slot * in.W + cc];      // the state in front of the tile
     constexpr int TILE = RG_RUNS * RG_RUN;
-    float2 p[RG_RUN];
-    auto load = [&](int tile) {
-#pragma unroll
-        for (int u = 0; u < RG_RUN; ++u) {
-            const int k = tile * TILE + run * RG_RUN + u;
-            p[u] = k < len ? ab[(size_t)(t0 + k) * in.W + cc] : make_float2(0.f, 0.f);
-        }
-    };
     const int tiles = (len + TILE - 1) / TILE;
-    load(0);
     for (int tile = 0; tile < tiles; ++tile) {
-        float2 mine[RG_RUN];
+        float2 p[RG_RUN];
         float y[RG_RUN];
+        const int k0 = tile * TILE + run * RG_RUN;
 #pragma unroll
-        for (int u = 0; u < RG_RUN; ++u) mine[u] = p[u];
+        for (int u = 0; u < RG_RUN; ++u) p[u] = k0 + u < len ? rg_pair_at<MADE>(src, g, in.W, t0 + k0 + u, cc) : make_float2(0.f, 0.f);
 #pragma unroll
-        for (int u = 0; u < RG_RUN; ++u) {
-            const int k = tile * TILE + run * RG_RUN + u;
-            y[u] = k < len ? rg_in(in.fused, in.dtype, in.parts, in.part_stride, (size_t)(t0 + k) * in.row_stride + in.y_off + cc) + in.y_bias[cc] : 0.f;
+        for (int u = 0; u < RG_RUN; ++u)
+            y[u] = k0 + u < len ? rg_in(in.fused, in.dtype, in.parts, in.part_stride, (size_t)(t0 + k0 + u) * in.row_stride + in.y_off + cc) + in.y_bias[cc] : 0.f;
+        float2 mine = p[0];
+#pragma unroll
+        for (int u = 1; u < RG_RUN; ++u) mine = rg_join(mine, p[u]);
+        // the runs of the warp that lie before this one, and the warp's four together
+        float2 upto = mine;
+#pragma unroll
+        for (int o = RG_COLS; o < 32; o <<= 1) {
+            const float2 before = make_float2(__shfl_up_sync(0xffffffffu, upto.x, o), __shfl_up_sync(0xffffffffu, upto.y, o));
+            if (lane >= o) upto = rg_join(before, upto);
         }
-        if (tile + 1 < tiles) load(tile + 1);           // on its way while this tile is walked
-        float A = 0.f, L = 0.f;
-#pragma unroll
-        for (int u = 0; u < RG_RUN; ++u) { L = rg_advance(L, mine[u]); A = A + fmaf(mine[u].x, A, mine[u].x); }      // (1 + A)(1 + e) - 1
-        local[tile & 1][run][col] = make_float2(A, L);
+        if (lane >= 32 - RG_COLS) local[tile & 1][warp][col] = upto;
         __syncthreads();                                // (the buffer of the tile before is read to its end by the time this one is full)
-        float S = carry, end = carry;
-        for (int q = 0; q < RG_RUNS; ++q) {
-            end = rg_advance(end, local[tile & 1][q][col]);
-            if (q + 1 == run) S = end;
-        }
+        float S = carry;
+#pragma unroll 4
+        for (int w = 0; w < warp; ++w) S = rg_advance(S, local[tile & 1][w][col]);
+        float end = S;
+#pragma unroll 4
+        for (int w = warp; w < RG_WARPS; ++w) end = rg_advance(end, local[tile & 1][w][col]);
         carry = end;
+        const float2 before = make_float2(__shfl_up_sync(0xffffffffu, upto.x, RG_COLS), __shfl_up_sync(0xffffffffu, upto.y, RG_COLS));
+        if (lane >= RG_COLS) S = rg_advance(S, before);
 #pragma unroll
         for (int u = 0; u < RG_RUN; ++u) {
-            const int k = tile * TILE + run * RG_RUN + u;
-            S = rg_advance(S, mine[u]);
-            if (k < len && live) out[(size_t)(t0 + k) * in.W + c] = from_f32<TO>(S * rg_gelu_tanh(y[u]));
+            S = rg_advance(S, p[u]);
+            if (k0 + u < len && live) out[(size_t)(t0 + k0 + u) * in.W + c] = from_f32<TO>(S * rg_gelu_tanh(y[u]));
         }
     }
     if (run == 0 && live) {
@@ -473,7 +518,7 @@ rglru_step_kernel(RgInput in, RgGates g, int n, const int* __restrict__ req_q_le
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
                 const int col = col0 + (m & 1) * 16 + (lane >> 2) + (q & 1) * 8, k = ks * 16 + (lane & 3) * 2 + (q >> 1) * 8;
-                a[m][q] = (col < g.s && k < g.s) ? *reinterpret_cast<const uint32_t*>(w + ((size_t)base + col) * g.s + k) : 0u;
+                a[m][q] = (col < g.s && k < g.s) ? *reinterpret_cast<const uint32_t*>(w + b * g.block + (size_t)col * g.pitch + k) : 0u;
             }
         }
     };
@@ -561,7 +606,7 @@ static int rg_check(const RgInput& in) {
 }
 // rows, vectors and maps whose eight neighbouring elements may be read with 16-byte loads
 static bool rg_wide(const RgInput& in, const RgGates& g) {
-    return g.w_dtype == WLLM_BF16 && g.s % 8 == 0 && in.W % 8 == 0 && in.x_off % 8 == 0 && in.row_stride % 8 == 0 && in.part_stride % 4 == 0 &&
+    return g.w_dtype == WLLM_BF16 && g.s % 8 == 0 && g.pitch % 8 == 0 && g.block % 8 == 0 && in.W % 8 == 0 && in.x_off % 8 == 0 && in.row_stride % 8 == 0 && in.part_stride % 4 == 0 &&
            !(((uintptr_t)in.fused | (uintptr_t)in.x_bias | (uintptr_t)in.taps | (uintptr_t)in.conv_bias | (uintptr_t)in.ring | (uintptr_t)g.ra |
               (uintptr_t)g.ri) & 15);
 }
@@ -571,10 +616,12 @@ static bool rg_wide(const RgInput& in, const RgGates& g) {
     const int* token_req, const int* req_q_start, const int* req_slot, float* ring
 #define RG_INPUT RgInput{fused, in_dtype, row_stride, parts, (size_t)part_stride, y_off, x_off, x_bias, y_bias, taps, conv_bias, T, W, \
     positions, token_req, req_q_start, req_slot, ring}
-#define RG_GATE_ARGS const void* ra, const void* ri, int w_dtype, const float* ra_bias, const float* ri_bias, const float* lam, float c, int B
+#define RG_GATE_ARGS const void* ra, const void* ri, int w_dtype, int w_pitch, long long w_block, const float* ra_bias, const float* ri_bias, \
+    const float* rate, int B
+#define RG_GATES RgGates{ra, ri, w_dtype, w_pitch, (size_t)w_block, ra_bias, ri_bias, rate, B, B > 0 ? W / B : 0}
 
 static int rg_gates_ok(const RgGates& g, int W) {
-    if (g.B < 1 || W % g.B != 0 || !g.ra || !g.ri || !g.ra_bias || !g.ri_bias || !g.lam) return WLLM_BAD_SIZE;
+    if (g.B < 1 || W % g.B != 0 || !g.ra || !g.ri || !g.ra_bias || !g.ri_bias || !g.rate || g.pitch < g.s) return WLLM_BAD_SIZE;
     return g.w_dtype == WLLM_BF16 || g.w_dtype == WLLM_F32 ? WLLM_OK : WLLM_BAD_DTYPE;
 }
 
@@ -584,7 +631,7 @@ WLLM_API int wllm_rglru_gates(RG_INPUT_ARGS, RG_GATE_ARGS, int n, float* ab, cud
     const RgInput in = RG_INPUT;
     int st = rg_check(in);
     if (st != WLLM_OK) return st;
-    const RgGates g{ra, ri, w_dtype, ra_bias, ri_bias, lam, c, B, B > 0 ? W / B : 0};
+    const RgGates g = RG_GATES;
     st = rg_gates_ok(g, W);
     if (st != WLLM_OK) return st;
     if (rg_wide(in, g) && ((uintptr_t)ab & 15) == 0) {
@@ -603,20 +650,39 @@ WLLM_API int wllm_rglru_gates(RG_INPUT_ARGS, RG_GATE_ARGS, int n, float* ab, cud
     return wllm_launch(rglru_gates_plain_kernel, grid, 256, 0, stream, in, g, n, (float2*)ab);
 }
 
-// long_portions: the step holds portions long enough for runs side by side (else every request is walked token by token)
-WLLM_API int wllm_rglru_scan(RG_INPUT_ARGS, const float* ab, const int* req_q_len, int requests, float* state, void* out, int out_dtype,
-                             int long_portions, cudaStream_t stream) {
-    if (requests <= 0) return WLLM_OK;
+// uv [B][n][2 W / B] (see above); tiles (null: none): 1 + 3 * B * ceil(n / tile_rows) ints.  W / B in steps of 8, aligned rows.
+WLLM_API int wllm_rglru_conv(RG_INPUT_ARGS, int B, int n, void* uv, int* tiles, int tile_rows, cudaStream_t stream) {
+    if (n <= 0) return WLLM_OK;
     const RgInput in = RG_INPUT;
     const int st = rg_check(in);
     if (st != WLLM_OK) return st;
-    if (requests > 65535 || !ab || !state || !out) return WLLM_BAD_SIZE;
-#define GO(TO) (long_portions \
-        ? wllm_launch(rglru_runs_kernel<TO>, dim3((W + RG_COLS - 1) / RG_COLS, requests), RG_RUNS * RG_COLS, 0, stream, in, (const float2*)ab, req_q_len, state, (TO*)out) \
-        : wllm_launch(rglru_walk_kernel<TO>, dim3((W + 127) / 128, requests), 128, 0, stream, in, (const float2*)ab, req_q_len, state, (TO*)out))
+    if (B < 1 || W % B != 0 || (W / B) % 8 != 0 || in.x_off % 8 != 0 || in.row_stride % 8 != 0 || in.part_stride % 4 != 0 || (tiles && tile_rows < 1))
+        return WLLM_BAD_SIZE;
+    if (((uintptr_t)fused | (uintptr_t)x_bias | (uintptr_t)taps | (uintptr_t)conv_bias | (uintptr_t)ring | (uintptr_t)uv) & 15) return WLLM_BAD_ALIGN;
+    return wllm_launch(rglru_conv_kernel, dim3((n + 3) / 4, (W + 511) / 512), 256, 0, stream, in, n, B, W / B, (bf16*)uv, tiles, tile_rows);
+}
+
+// ab [n, W, 2], or (ab null) z [B][n][2 W / B] and uv of the same shape: n tokens.  long_portions: the step holds portions long enough
+// for runs side by side (else every request is walked token by token)
+WLLM_API int wllm_rglru_scan(RG_INPUT_ARGS, RG_GATE_ARGS, int n, const float* ab, const float* z, const void* uv, const int* req_q_len,
+                             int requests, float* state, void* out, int out_dtype, int long_portions, cudaStream_t stream) {
+    if (requests <= 0) return WLLM_OK;
+    const RgInput in = RG_INPUT;
+    int st = rg_check(in);
+    if (st != WLLM_OK) return st;
+    const RgGates g = RG_GATES;
+    st = rg_gates_ok(g, W);
+    if (st != WLLM_OK) return st;
+    if (requests > 65535 || (!ab && (!z || !uv)) || !state || !out) return WLLM_BAD_SIZE;
+    const RgPairs src{(const float2*)ab, z, (const bf16*)uv, n, g.s};
+#define GO2(TO, M) (long_portions \
+        ? wllm_launch(rglru_runs_kernel<TO, M>, dim3((W + RG_COLS - 1) / RG_COLS, requests), RG_RUNS * RG_COLS, 0, stream, in, g, src, req_q_len, state, (TO*)out) \
+        : wllm_launch(rglru_walk_kernel<TO, M>, dim3((W + 127) / 128, requests), 128, 0, stream, in, g, src, req_q_len, state, (TO*)out))
+#define GO(TO) (ab ? GO2(TO, true) : GO2(TO, false))
     if (out_dtype == WLLM_BF16) return GO(bf16);
     if (out_dtype == WLLM_F32) return GO(float);
 #undef GO
+#undef GO2
     return WLLM_BAD_DTYPE;
 }
 
@@ -627,7 +693,7 @@ WLLM_API int wllm_rglru_step(RG_INPUT_ARGS, RG_GATE_ARGS, int n, const int* req_
     const RgInput in = RG_INPUT;
     int st = rg_check(in);
     if (st != WLLM_OK) return st;
-    const RgGates g{ra, ri, w_dtype, ra_bias, ri_bias, lam, c, B, B > 0 ? W / B : 0};
+    const RgGates g = RG_GATES;
     st = rg_gates_ok(g, W);
     if (st != WLLM_OK) return st;
     if (!rg_wide(in, g) || g.s > RS_MAX_S) return WLLM_BAD_SIZE;

@@ -1437,15 +1437,17 @@ def _rglru_input(fused, parts: int, unit: dict, ctx, ring: torch.Tensor) -> tupl
 
 
 def _rglru_gates(gates: dict, W: int) -> tuple:
-    """`gates`: ra, ri [B, s, s], ra_bias, ri_bias, lam [W] (32-bit), c."""
-    B, s, _ = gates["ra"].shape
-    assert gates["ra"].shape == gates["ri"].shape == (B, s, s) and B * s == W and gates["ra"].dtype == gates["ri"].dtype
-    assert gates["ra"].is_contiguous() and gates["ri"].is_contiguous()
-    for key in ("ra_bias", "ri_bias", "lam"):
+    """`gates`: maps [blocks, 2 s, s or 2 s]: in every block the rows of R, then those of I, and (2 s columns, for the grouped product)
+    each row twice side by side; ra_bias, ri_bias, rate [W] (32-bit; log a = -rate * r)."""
+    maps = gates["maps"]
+    B, rows, cols = maps.shape
+    s = rows // 2
+    assert B * s == W and cols in (s, 2 * s) and maps.is_contiguous()
+    for key in ("ra_bias", "ri_bias", "rate"):
         assert gates[key].dtype == torch.float32 and gates[key].shape == (W,) and gates[key].is_contiguous()
-    _need_cuda(*[gates[k] for k in ("ra", "ri", "ra_bias", "ri_bias", "lam")])
-    return (_ptr(gates["ra"]), _ptr(gates["ri"]), _dt(gates["ra"]), _ptr(gates["ra_bias"]), _ptr(gates["ri_bias"]), _ptr(gates["lam"]),
-            c_float(gates["c"]), B)
+    _need_cuda(*[gates[k] for k in ("maps", "ra_bias", "ri_bias", "rate")])
+    return (_ptr(maps), c_void_p(maps.data_ptr() + s * cols * maps.element_size()), _dt(maps), cols, ctypes.c_longlong(rows * cols),
+            _ptr(gates["ra_bias"]), _ptr(gates["ri_bias"]), _ptr(gates["rate"]), B)
 
 
 def rglru_gates(fused, parts: int, unit: dict, gates: dict, ctx, ring: torch.Tensor, ab: torch.Tensor) -> torch.Tensor:
@@ -1457,23 +1459,54 @@ def rglru_gates(fused, parts: int, unit: dict, gates: dict, ctx, ring: torch.Ten
     return ab
 
 
-def rglru_scan(fused, parts: int, unit: dict, ctx, ring: torch.Tensor, ab: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
-               long_portions: bool) -> torch.Tensor:
-    """S <- a S + b, with (a - 1, b) from `ab`, over every request's tokens of the step, from and to its row of `state` [slots, W]; out = S * gelu_tanh(y + bias) [n, W]; the
-    convolution's newest inputs go to `ring`.  `long_portions`: runs of tokens side by side instead of token by token."""
+RGLRU_GROUPED_FROM = 256      # tokens of a step from which the gates' maps run on the grouped tensor-memory product
+
+
+def rglru_grouped_ok(gates: dict, fused, x_off: int) -> bool:
+    """Whether the gates' maps can run on the grouped tensor-memory product: bfloat16, blocks in steps of 8, rows held twice."""
+    maps = gates["maps"]
+    return maps.dtype == torch.bfloat16 and maps.shape[2] == maps.shape[1] and maps.shape[1] % 16 == 0 and x_off % 8 == 0 and \
+        fused.stride(-2) % 8 == 0 and fused.data_ptr() % 16 == 0
+
+
+def rglru_gate_sums(fused, parts: int, unit: dict, gates: dict, ctx, ring: torch.Tensor, uv: torch.Tensor, tiles: torch.Tensor,
+                    z: torch.Tensor) -> None:
+    """The convolution and the gates' sums for many tokens: u as two bfloat16 pieces in uv [blocks * n, 2 s] (high, low), z [blocks * n, 2 s]
+    float32 = the sums of R and I, by one grouped product (the row tiles go to `tiles`, int32, 1 + 3 * moe_row_tiles(blocks * n, blocks))."""
     args, n, W = _rglru_input(fused, parts, unit, ctx, ring)
-    assert ab.dtype == torch.float32 and ab.shape == (n, W, 2) and ab.is_contiguous() and out.shape == (n, W) and out.is_contiguous()
-    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (W,)
+    maps = gates["maps"]
+    B = maps.shape[0]
+    _need_cuda(uv, tiles, z)
+    assert uv.shape == z.shape == (B * n, maps.shape[1]) and uv.dtype == torch.bfloat16 and z.dtype == torch.float32 and uv.is_contiguous() and z.is_contiguous()
+    assert tiles.dtype == torch.int32 and tiles.numel() >= 1 + 3 * B * -(-n // MOE_TILE_ROWS)
     lib = load_family("rg_lru")
-    _check(lib.wllm_rglru_scan(*args, _ptr(ab), _ptr(_int32(ctx.req_q_len, "req_q_len")), ctx.req_q_len.shape[0], _ptr(state), _ptr(out),
-                               _dt(out), 1 if long_portions else 0, _stream()), "rglru_scan")
+    _check(lib.wllm_rglru_conv(*args, B, n, _ptr(uv), _ptr(tiles), MOE_TILE_ROWS, _stream()), "rglru_conv")
+    gemm_bf16_tc_grouped(uv, maps, z, tiles, False)
+
+
+def rglru_scan(fused, parts: int, unit: dict, gates: dict, ctx, ring: torch.Tensor, pairs, state: torch.Tensor, out: torch.Tensor,
+               long_portions: bool) -> torch.Tensor:
+    """S <- a S + b over every request's tokens of the step, from and to its row of `state` [slots, W]; out = S * gelu_tanh(y + bias) [n, W];
+    the convolution's newest inputs go to `ring`.  `pairs`: what rglru_gates made (a - 1, b), or (z, uv) as rglru_gate_sums left them.
+    `long_portions`: runs of tokens side by side instead of token by token."""
+    args, n, W = _rglru_input(fused, parts, unit, ctx, ring)
+    made = isinstance(pairs, torch.Tensor)
+    z, uv = (None, None) if made else pairs
+    assert not made or (pairs.dtype == torch.float32 and pairs.shape == (n, W, 2) and pairs.is_contiguous())
+    assert made or (z.numel() == uv.numel() == 2 * n * W and z.dtype == torch.float32 and uv.dtype == torch.bfloat16)
+    assert out.shape == (n, W) and out.is_contiguous() and state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (W,)
+    lib = load_family("rg_lru")
+    _check(lib.wllm_rglru_scan(*args, *_rglru_gates(gates, W), n, _ptr(pairs if made else None), _ptr(z), _ptr(uv),
+                               _ptr(_int32(ctx.req_q_len, "req_q_len")), ctx.req_q_len.shape[0], _ptr(state), _ptr(out), _dt(out),
+                               1 if long_portions else 0, _stream()), "rglru_scan")
     return out
 
 
 def rglru_step_ok(gates: dict, fused, x_off: int) -> bool:
     """Whether convolution, gates and recurrence of a step of single tokens can run as one kernel."""
-    s = gates["ra"].shape[1]
-    return gates["ra"].dtype == torch.bfloat16 and s % 8 == 0 and s <= RGLRU_STEP_MAX_BLOCK and x_off % 8 == 0 and fused.stride(-2) % 8 == 0 \
+    maps = gates["maps"]
+    s = maps.shape[1] // 2
+    return maps.dtype == torch.bfloat16 and s % 8 == 0 and s <= RGLRU_STEP_MAX_BLOCK and x_off % 8 == 0 and fused.stride(-2) % 8 == 0 \
         and fused.data_ptr() % 16 == 0
 
 

@@ -36,7 +36,7 @@ class GatedRecurrence:
         self.hidden_size, self.model_dtype = hidden_size, model_dtype
         self.names = {k: spec.options[k] for k in _NAMES}
         self.w_in = self.wo = self.conv = self.conv_bias = self.x_bias = self.y_bias = None
-        self.ra = self.ri = self.ra_bias = self.ri_bias = self.decay = None
+        self.maps = self.ra_bias = self.ri_bias = self.rate = None
         self.x_off = 0
         self.tag = ""
 
@@ -62,21 +62,33 @@ class GatedRecurrence:
         self.w_in = torch.cat([y] + gap + [fetch(n["x_proj"])] + gap, dim=0).contiguous()
         self.wo = fetch(n["o_proj"]).contiguous()
         self.conv = fetch(n["conv"]).to(torch.float32).t().contiguous()
-        self.x_bias, self.y_bias, self.conv_bias, self.decay = vector("x_bias"), vector("y_bias"), vector("conv_bias"), vector("decay")
-        self.ra, self.ri = fetch(n["r_gate"]).contiguous(), fetch(n["i_gate"]).contiguous()
+        self.x_bias, self.y_bias, self.conv_bias = vector("x_bias"), vector("y_bias"), vector("conv_bias")
+        # log a = -rate r: what the gate does not touch is worked out once (in 64-bit, rounded once)
+        self.rate = (self.c * torch.nn.functional.softplus(fetch(n["decay"]).to(torch.float64))).to(torch.float32).contiguous()
+        # both gates' rows of a block one below the other; in bfloat16 each row twice side by side, for the two pieces of u
+        maps = torch.cat([fetch(n["r_gate"]), fetch(n["i_gate"])], dim=1)
+        self.maps = (torch.cat([maps, maps], dim=2) if self.model_dtype == torch.bfloat16 else maps).contiguous()
         self.ra_bias, self.ri_bias = vector("r_bias"), vector("i_bias")
 
     def __call__(self, x: torch.Tensor, ctx, cache: CacheRef):
         n, W = x.shape[0], self.width
         fused, parts = ops.project(x, self.w_in, lambda name, shape, dt: ctx.buffer(self.tag + "lru_in_" + name, shape, dt))
         unit = dict(y_off=0, x_off=self.x_off, x_bias=self.x_bias, y_bias=self.y_bias, taps=self.conv, conv_bias=self.conv_bias)
-        gates = dict(ra=self.ra, ri=self.ri, ra_bias=self.ra_bias, ri_bias=self.ri_bias, lam=self.decay, c=self.c)
+        gates = dict(maps=self.maps, ra_bias=self.ra_bias, ri_bias=self.ri_bias, rate=self.rate)
         state, ring = ctx.state(cache.state_names["state"]), ctx.state(cache.state_names["conv"])
         out = ctx.buffer(self.tag + "lru_out", (n, W), self.model_dtype)
         if ctx.num_multi == 0 and self.model_dtype == torch.bfloat16 and ops.rglru_step_ok(gates, fused, self.x_off):
             ops.rglru_step(fused, parts, unit, gates, ctx, ring, state, out)
         else:
-            ab = ctx.buffer(self.tag + "lru_pairs", (n, W, 2), torch.float32)
-            ops.rglru_gates(fused, parts, unit, gates, ctx, ring, ab)
-            ops.rglru_scan(fused, parts, unit, ctx, ring, ab, state, out, ctx.max_q_len >= ops.RGLRU_RUNS_FROM)
+            if n >= ops.RGLRU_GROUPED_FROM and ops.rglru_grouped_ok(gates, fused, self.x_off):
+                B, rows = self.blocks, self.maps.shape[1]
+                uv = ctx.buffer(self.tag + "lru_pieces", (B * n, rows), torch.bfloat16)
+                z = ctx.buffer(self.tag + "lru_gate_sums", (B * n, rows), torch.float32)
+                tiles = ctx.buffer(self.tag + "lru_tiles", (1 + 3 * ops.moe_row_tiles(B * n, B),), torch.int32)
+                ops.rglru_gate_sums(fused, parts, unit, gates, ctx, ring, uv, tiles, z)
+                pairs = (z, uv)
+            else:
+                pairs = ctx.buffer(self.tag + "lru_pairs", (n, W, 2), torch.float32)
+                ops.rglru_gates(fused, parts, unit, gates, ctx, ring, pairs)
+            ops.rglru_scan(fused, parts, unit, gates, ctx, ring, pairs, state, out, ctx.max_q_len >= ops.RGLRU_RUNS_FROM)
         return as_branch(ops.project(out, self.wo, lambda name, shape, dt: ctx.buffer(self.tag + "lru_branch_" + name, shape, dt)))
