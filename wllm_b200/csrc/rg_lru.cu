@@ -19,9 +19,9 @@
 //                      block's rows [R R; I I] gives both gates' sums in 32-bit.  It writes that product's table of row tiles too.
 //   wllm_rglru_scan    the recurrence over every request's tokens from and to its slot, the output gate, and the slot's kept
 //                      inputs, from the pairs or from the gates' sums and u's pieces.  Short portions: a thread a channel walks the
-//                      tokens.  Long ones: 64 runs of 8 tokens at a time; a run's decay product and end state from zero come first,
+//                      tokens.  Long ones: 32 runs of 4 tokens at a time; a run's decay product and end state from zero come first,
 //                      then its true start state from the runs before it, then its outputs; all of it from registers, so that
-//                      everything is read once.
+//                      everything is read once, and the next tokens' values are on their way meanwhile.
 //   wllm_rglru_step    both at once for a step in which no request brings more than one token (decoding).
 #include "common.cuh"
 
@@ -344,7 +344,7 @@ rglru_gates_mma_kernel(RgInput in, RgGates g, int n, float2* __restrict__ ab) {
 
 // the convolution alone: grid (tiles of 4 tokens, tiles of 512 channels), 256 threads = 4 tokens by 64 runs of eight channels.
 // uv [B][n][2 s]; tiles (null: none): the table of row tiles of `tile_rows` rows of one block each
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 rglru_conv_kernel(RgInput in, int n, int B, int s, bf16* __restrict__ uv, int* __restrict__ tiles, int tile_rows) {
     pdl_begin();
     if (tiles != nullptr && blockIdx.x == 0 && blockIdx.y == 0) {
@@ -423,14 +423,40 @@ rglru_walk_kernel(RgInput in, RgGates g, RgPairs src, const int* __restrict__ re
     rg_keep_inputs(in, t0, len, slot, in.positions[t0], c);
 }
 
-// runs side by side: grid (ceil(W / 8), requests), 512 threads = 64 runs of 8 tokens by 8 channels; a warp has four runs
-constexpr int RG_RUNS = 64, RG_RUN = 8, RG_COLS = 8, RG_WARPS = RG_RUNS * RG_COLS / 32;
+// runs side by side: grid (ceil(W / 8), requests), 256 threads = 32 runs of 4 tokens by 8 channels; a warp has four runs
+constexpr int RG_RUNS = 32, RG_RUN = 4, RG_COLS = 8, RG_WARPS = RG_RUNS * RG_COLS / 32;
+// what a run's tokens bring, as it comes from memory
+template <bool MADE> struct RgRaw;
+template <> struct RgRaw<true> {
+    float2 p[RG_RUN];
+    __device__ __forceinline__ void load(const RgPairs& src, int W, int t0, int k0, int len, int c) {
+#pragma unroll
+        for (int u = 0; u < RG_RUN; ++u) p[u] = src.ab[(size_t)(t0 + min(k0 + u, len - 1)) * W + c];
+    }
+    __device__ __forceinline__ float2 pair(const RgGates&, int, int u) const { return p[u]; }
+};
+template <> struct RgRaw<false> {
+    float zr[RG_RUN], zi[RG_RUN];
+    bf16 hi[RG_RUN], lo[RG_RUN];
+    __device__ __forceinline__ void load(const RgPairs& src, int, int t0, int k0, int len, int c) {
+        const size_t base = (size_t)(c / src.s) * src.n * 2 * src.s + c % src.s;
+#pragma unroll
+        for (int u = 0; u < RG_RUN; ++u) {
+            const size_t at = base + (size_t)(t0 + min(k0 + u, len - 1)) * 2 * src.s;
+            zr[u] = src.z[at]; zi[u] = src.z[at + src.s];
+            hi[u] = src.uv[at]; lo[u] = src.uv[at + src.s];
+        }
+    }
+    __device__ __forceinline__ float2 pair(const RgGates& g, int c, int u) const {
+        return rg_pair(g, c, zr[u], zi[u], __bfloat162float(hi[u]) + __bfloat162float(lo[u]));
+    }
+};
 // two stretches of the recurrence one behind the other, each as (decay product - 1, end state from zero)
 __device__ __forceinline__ float2 rg_join(float2 first, float2 second) {
     return make_float2(first.x + fmaf(second.x, first.x, second.x), rg_advance(first.y, second));
 }
 template <typename TO, bool MADE>
-__global__ void __launch_bounds__(RG_RUNS * RG_COLS)
+__global__ void __launch_bounds__(RG_RUNS * RG_COLS, 3)
 rglru_runs_kernel(RgInput in, RgGates g, RgPairs src, const int* __restrict__ req_q_len, float* __restrict__ state, TO* __restrict__ out) {
     __shared__ float2 local[2][RG_WARPS][RG_COLS];       // a warp's four runs joined
     pdl_begin();
@@ -442,17 +468,30 @@ rglru_runs_kernel(RgInput in, RgGates g, RgPairs src, const int* __restrict__ re
     const int cc = live ? c : in.W - 1;
     const int t0 = in.req_q_start[r];
     float carry = state[(size_t)slot * in.W + cc];      // the state in front of the tile
+    const float y_bias = in.y_bias[cc];
     constexpr int TILE = RG_RUNS * RG_RUN;
     const int tiles = (len + TILE - 1) / TILE;
-    for (int tile = 0; tile < tiles; ++tile) {
-        float2 p[RG_RUN];
-        float y[RG_RUN];
+    RgRaw<MADE> raw;
+    float y_raw[RG_RUN];
+    auto load = [&](int tile) {
         const int k0 = tile * TILE + run * RG_RUN;
-#pragma unroll
-        for (int u = 0; u < RG_RUN; ++u) p[u] = k0 + u < len ? rg_pair_at<MADE>(src, g, in.W, t0 + k0 + u, cc) : make_float2(0.f, 0.f);
+        raw.load(src, in.W, t0, k0, len, cc);
 #pragma unroll
         for (int u = 0; u < RG_RUN; ++u)
-            y[u] = k0 + u < len ? rg_in(in.fused, in.dtype, in.parts, in.part_stride, (size_t)(t0 + k0 + u) * in.row_stride + in.y_off + cc) + in.y_bias[cc] : 0.f;
+            y_raw[u] = rg_in(in.fused, in.dtype, in.parts, in.part_stride, (size_t)(t0 + min(k0 + u, len - 1)) * in.row_stride + in.y_off + cc);
+    };
+    load(0);
+    for (int tile = 0; tile < tiles; ++tile) {
+        const int k0 = tile * TILE + run * RG_RUN;
+        float2 p[RG_RUN];
+        float y[RG_RUN];
+#pragma unroll
+        for (int u = 0; u < RG_RUN; ++u) {
+            p[u] = raw.pair(g, cc, u);
+            if (k0 + u >= len) p[u] = make_float2(0.f, 0.f);
+            y[u] = y_raw[u];
+        }
+        if (tile + 1 < tiles) load(tile + 1);           // on its way while this tile is walked
         float2 mine = p[0];
 #pragma unroll
         for (int u = 1; u < RG_RUN; ++u) mine = rg_join(mine, p[u]);
@@ -465,19 +504,19 @@ rglru_runs_kernel(RgInput in, RgGates g, RgPairs src, const int* __restrict__ re
         }
         if (lane >= 32 - RG_COLS) local[tile & 1][warp][col] = upto;
         __syncthreads();                                // (the buffer of the tile before is read to its end by the time this one is full)
-        float S = carry;
-#pragma unroll 4
-        for (int w = 0; w < warp; ++w) S = rg_advance(S, local[tile & 1][w][col]);
-        float end = S;
-#pragma unroll 4
-        for (int w = warp; w < RG_WARPS; ++w) end = rg_advance(end, local[tile & 1][w][col]);
+        float S = carry, end = carry;
+#pragma unroll
+        for (int w = 0; w < RG_WARPS; ++w) {
+            if (w == warp) S = end;
+            end = rg_advance(end, local[tile & 1][w][col]);
+        }
         carry = end;
         const float2 before = make_float2(__shfl_up_sync(0xffffffffu, upto.x, RG_COLS), __shfl_up_sync(0xffffffffu, upto.y, RG_COLS));
         if (lane >= RG_COLS) S = rg_advance(S, before);
 #pragma unroll
         for (int u = 0; u < RG_RUN; ++u) {
             S = rg_advance(S, p[u]);
-            if (k0 + u < len && live) out[(size_t)(t0 + k0 + u) * in.W + c] = from_f32<TO>(S * rg_gelu_tanh(y[u]));
+            if (k0 + u < len && live) out[(size_t)(t0 + k0 + u) * in.W + c] = from_f32<TO>(S * rg_gelu_tanh(y[u] + y_bias));
         }
     }
     if (run == 0 && live) {

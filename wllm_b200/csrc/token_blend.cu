@@ -10,9 +10,10 @@
 //                         channels (or one) of a run of tokens.
 //   wllm_blended_product  few tokens, one a request (decoding), bfloat16: the products themselves, each reading its own blend.  The
 //                         matrices lie one below the other, [N, H], in segments that name their stream (or none: h itself);
-//                         out [n, N] 32-bit.  A CTA has 32 rows of one segment: it blends the tokens' rows into shared memory, its
-//                         eight warps share K (32 columns at a time, every lane 16 contiguous bytes of a row, asked for while the
-//                         kernel before still runs), and their sums meet in shared memory in warp order.
+//                         out [n, N] 32-bit.  A CTA has some rows of one segment, so many that all CTAs run at once: it blends the
+//                         tokens' rows into shared memory once and walks its rows sixteen at a time; its eight warps share K (32
+//                         columns at a time, every lane 16 contiguous bytes of a row, the first asked for while the kernel before
+//                         still runs, the next rows' while these are multiplied), and their sums meet in shared memory in warp order.
 #include "common.cuh"
 
 constexpr int TB_MAX_STREAMS = 8, TB_TOKENS = 8;
@@ -125,9 +126,9 @@ struct BlendSegments {
     int count;
     int row0[TB_MAX_STREAMS + 1];        // first row of a segment; row0[count] = N
     int stream[TB_MAX_STREAMS + 1];      // the stream it reads, -1: h itself
-    int tile0[TB_MAX_STREAMS + 1];       // first tile of 32 rows
+    int tile0[TB_MAX_STREAMS + 1];       // first CTA
 };
-constexpr int BP_ROWS = 32, BP_WARPS = 8, BP_DEPTH = 4;
+constexpr int BP_ROWS = 16, BP_WARPS = 8, BP_CTAS = 2 * 148;
 
 __device__ __forceinline__ void bp_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
@@ -139,46 +140,40 @@ __device__ __forceinline__ uint4 bp_stream(const bf16* p) {              // weig
     return v;
 }
 
-// NT: tiles of eight tokens.  KC: columns of the tokens' blends that lie in shared memory at a time (a multiple of 256).
-template <int NT>
+// NT: tiles of eight tokens; DEPTH: runs of 32 columns a warp has on their way.  KC: columns of the tokens' blends that lie in shared memory
+// at a time (all of them, or a multiple of 256 * DEPTH); subs: groups of sixteen rows of a CTA (1 when the blends do not fit at once).
+template <int NT, int DEPTH>
 __global__ void __launch_bounds__(BP_WARPS * 32, 2)
 blended_product_kernel(const bf16* __restrict__ h, int n, int H, const float* __restrict__ mu, const bf16* __restrict__ w, BlendSegments seg,
                        const int* __restrict__ positions, const int* __restrict__ token_req, const int* __restrict__ req_q_len,
-                       const int* __restrict__ req_slot, bf16* __restrict__ kept, float* __restrict__ out, int N, int KC) {
+                       const int* __restrict__ req_slot, bf16* __restrict__ kept, float* __restrict__ out, int N, int KC, int subs) {
     extern __shared__ __align__(16) unsigned char bp_smem[];
-    bf16* xs = reinterpret_cast<bf16*>(bp_smem);                // [8 NT][KC + 8]
-    float* red = reinterpret_cast<float*>(bp_smem);             // [8 warps][32 rows][8 NT + 1], once the products are done
+    constexpr int RP = 8 * NT + 1;
+    bf16* xs = reinterpret_cast<bf16*>(bp_smem);                                      // [8 NT][KC + 8]
+    float* red = reinterpret_cast<float*>(bp_smem + (size_t)8 * NT * (KC + 8) * 2);   // [2][8 warps][16 rows][8 NT + 1]
     pdl_launch_dependents();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pitch = KC + 8;
     int sg = 0;
     while (sg + 1 < seg.count && (int)blockIdx.x >= seg.tile0[sg + 1]) ++sg;
-    const int row0 = seg.row0[sg] + ((int)blockIdx.x - seg.tile0[sg]) * BP_ROWS, row_end = seg.row0[sg + 1], stream = seg.stream[sg];
-    // this lane's rows of the tile (lane / 4 + 8 j) and its 16-byte piece of a run of 32 columns
-    const bf16* src[4];
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-        const int row = row0 + (lane >> 2) + 8 * j;
-        src[j] = row < row_end ? w + (size_t)row * H + (lane & 3) * 8 : nullptr;
-    }
-    const int steps = (H + 31) / 32, mine = steps > warp ? (steps - warp + BP_WARPS - 1) / BP_WARPS : 0;      // this warp's runs: warp, warp + 8, ..
-    uint4 a[BP_DEPTH][4];
-    auto fetch = [&](int q, uint4 (&to)[4]) {
+    const int row0 = seg.row0[sg] + ((int)blockIdx.x - seg.tile0[sg]) * BP_ROWS * subs, row_end = min(seg.row0[sg + 1], row0 + BP_ROWS * subs);
+    const int stream = seg.stream[sg];
+    // this lane's rows of a group (lane / 4 and that + 8) and its 16-byte piece of a run of 32 columns; a warp's runs are warp, warp + 8, ..,
+    // padded to whole rounds of DEPTH
+    const int steps = (H + 31) / 32, mine = steps > warp ? (steps - warp + BP_WARPS - 1) / BP_WARPS : 0;
+    const int rounds = ((steps + BP_WARPS - 1) / BP_WARPS + DEPTH - 1) / DEPTH;
+    uint4 a[DEPTH][2];
+    auto fetch = [&](int sub, int q, uint4 (&to)[2]) {
         const int k = (warp + q * BP_WARPS) * 32 + (lane & 3) * 8;
 #pragma unroll
-        for (int j = 0; j < 4; ++j)
-            to[j] = (q < mine && src[j] != nullptr && k < H) ? bp_stream(src[j] + (warp + q * BP_WARPS) * 32) : make_uint4(0u, 0u, 0u, 0u);
+        for (int j = 0; j < 2; ++j) {
+            const int row = row0 + sub * BP_ROWS + (lane >> 2) + 8 * j;
+            to[j] = (q < mine && row < row_end && k < H) ? bp_stream(w + (size_t)row * H + k) : make_uint4(0u, 0u, 0u, 0u);
+        }
     };
 #pragma unroll
-    for (int q = 0; q < BP_DEPTH; ++q) fetch(q, a[q]);
+    for (int q = 0; q < DEPTH; ++q) fetch(0, q, a[q]);
     pdl_wait();
-    float acc[2][NT][4];
-#pragma unroll
-    for (int m = 0; m < 2; ++m)
-#pragma unroll
-        for (int j = 0; j < NT; ++j) acc[m][j][0] = acc[m][j][1] = acc[m][j][2] = acc[m][j][3] = 0.f;
-    const int per_chunk = KC / (32 * BP_WARPS);                 // runs a warp has in a chunk
-    for (int k0 = 0, q0 = 0; k0 < H; k0 += KC, q0 += per_chunk) {
-        if (k0 > 0) __syncthreads();
+    auto blend = [&](int k0) {
         for (int idx = threadIdx.x; idx < 8 * NT * (KC / 8); idx += blockDim.x) {
             const int tt = idx / (KC / 8), c = k0 + (idx % (KC / 8)) * 8;
             uint4 packed = make_uint4(0u, 0u, 0u, 0u);
@@ -202,45 +197,57 @@ blended_product_kernel(const bf16* __restrict__ h, int n, int H, const float* __
             }
             *reinterpret_cast<uint4*>(xs + tt * pitch + (c - k0)) = packed;
         }
-        __syncthreads();
-        for (int qq = 0; qq < per_chunk; qq += BP_DEPTH) {
+    };
+    const int per_chunk = KC / (32 * BP_WARPS);                 // runs a warp has in a chunk
+    const bool whole = KC >= H;
+    if (whole) { blend(0); __syncthreads(); }
+    for (int sub = 0; sub < subs && row0 + sub * BP_ROWS < row_end; ++sub) {
+        float acc[NT][4];
 #pragma unroll
-            for (int d = 0; d < BP_DEPTH; ++d) {
-                const int q = q0 + qq + d;
-                if (qq + d < per_chunk && q < mine) {
+        for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+        int k0 = 0, base = 0;                                   // first column and first run of the chunk that lies in shared memory
+        if (!whole) { blend(0); __syncthreads(); }
+        for (int round = 0; round < rounds; ++round) {
+            if (!whole && round * DEPTH >= base + per_chunk) {  // (a chunk holds whole rounds)
+                __syncthreads();
+                k0 += KC; base += per_chunk;
+                blend(k0);
+                __syncthreads();
+            }
+#pragma unroll
+            for (int d = 0; d < DEPTH; ++d) {
+                const int q = round * DEPTH + d;
+                if (q < mine) {
                     const int col = (warp + q * BP_WARPS) * 32 - k0 + (lane & 3) * 8;
 #pragma unroll
                     for (int j = 0; j < NT; ++j) {
                         const uint4 b = *reinterpret_cast<const uint4*>(xs + (j * 8 + (lane >> 2)) * pitch + col);
                         // a lane's eight columns of a run are the columns of two steps of 16: which of them stands where does
                         // not matter to the sum, as long as both operands agree
-                        bp_mma(acc[0][j], a[d][0].x, a[d][1].x, a[d][0].y, a[d][1].y, b.x, b.y);
-                        bp_mma(acc[0][j], a[d][0].z, a[d][1].z, a[d][0].w, a[d][1].w, b.z, b.w);
-                        bp_mma(acc[1][j], a[d][2].x, a[d][3].x, a[d][2].y, a[d][3].y, b.x, b.y);
-                        bp_mma(acc[1][j], a[d][2].z, a[d][3].z, a[d][2].w, a[d][3].w, b.z, b.w);
+                        bp_mma(acc[j], a[d][0].x, a[d][1].x, a[d][0].y, a[d][1].y, b.x, b.y);
+                        bp_mma(acc[j], a[d][0].z, a[d][1].z, a[d][0].w, a[d][1].w, b.z, b.w);
                     }
-                    fetch(q + BP_DEPTH, a[d]);
                 }
+                if (round + 1 < rounds) fetch(sub, q + DEPTH, a[d]);
+                else if (sub + 1 < subs) fetch(sub + 1, d, a[d]);
             }
         }
-    }
-    __syncthreads();                                            // the blends are read to their end: their room takes the sums
-    constexpr int RP = 8 * NT + 1;
-#pragma unroll
-    for (int m = 0; m < 2; ++m)
+        // the warps' sums meet in one of two places: who writes the next ones does not meet who still reads these
+        float* meet = red + (size_t)(sub & 1) * BP_WARPS * BP_ROWS * RP;
 #pragma unroll
         for (int j = 0; j < NT; ++j)
 #pragma unroll
             for (int q = 0; q < 4; ++q)
-                red[((size_t)warp * BP_ROWS + m * 16 + (lane >> 2) + (q >> 1) * 8) * RP + j * 8 + (lane & 3) * 2 + (q & 1)] = acc[m][j][q];
-    __syncthreads();
-    for (int idx = threadIdx.x; idx < n * BP_ROWS; idx += blockDim.x) {
-        const int tt = idx / BP_ROWS, row = idx % BP_ROWS;
-        if (row0 + row >= row_end) continue;
-        float v = 0.f;
+                meet[((size_t)warp * BP_ROWS + (lane >> 2) + (q >> 1) * 8) * RP + j * 8 + (lane & 3) * 2 + (q & 1)] = acc[j][q];
+        __syncthreads();
+        for (int idx = threadIdx.x; idx < n * BP_ROWS; idx += blockDim.x) {
+            const int tt = idx / BP_ROWS, row = idx % BP_ROWS, at = row0 + sub * BP_ROWS + row;
+            if (at >= row_end) continue;
+            float v = 0.f;
 #pragma unroll
-        for (int k = 0; k < BP_WARPS; ++k) v += red[((size_t)k * BP_ROWS + row) * RP + tt];
-        out[(size_t)tt * N + row0 + row] = v;
+            for (int k = 0; k < BP_WARPS; ++k) v += meet[((size_t)k * BP_ROWS + row) * RP + tt];
+            out[(size_t)tt * N + at] = v;
+        }
     }
 }
 
@@ -254,35 +261,37 @@ WLLM_API int wllm_blended_product(const void* h, int n, int H, const float* mu, 
     if (((uintptr_t)h | (uintptr_t)w | (uintptr_t)kept | (uintptr_t)mu) & 15) return WLLM_BAD_ALIGN;
     BlendSegments seg = {};
     seg.count = count;
+    const int nt = n <= 8 ? 1 : (n <= 16 ? 2 : 4), depth = nt == 4 ? 4 : 8;
+    const int round = 32 * BP_WARPS * depth;
+    // the blends in shared memory: whole rows of the tokens where they fit in some 66 KB, else as many columns as do, in whole rounds
+    int kc = (H + 255) / 256 * 256;
+    const int most = (33 * 1024 / (8 * nt) - 8) / round * round;
+    if (kc > most) kc = most;
+    int groups = 0;
+    for (int i = 0; i < count; ++i) groups += (rows[i] + BP_ROWS - 1) / BP_ROWS;
+    const int subs = kc < H ? 1 : (groups + BP_CTAS - 1) / BP_CTAS;
     int tiles = 0;
     for (int i = 0; i < count; ++i) {
         if (rows[i] < 1 || streams[i] < -1 || streams[i] >= TB_MAX_STREAMS) return WLLM_BAD_SIZE;
         seg.stream[i] = streams[i];
         seg.tile0[i] = tiles;
         seg.row0[i + 1] = seg.row0[i] + rows[i];
-        tiles += (rows[i] + BP_ROWS - 1) / BP_ROWS;
+        tiles += (rows[i] + BP_ROWS * subs - 1) / (BP_ROWS * subs);
     }
-    const int N = seg.row0[count], nt = n <= 8 ? 1 : (n <= 16 ? 2 : 4);
-    constexpr int STEP = 32 * BP_WARPS;
-    // the blends in shared memory: whole rows of the tokens where they fit in some 66 KB, else as many columns as do
-    int kc = (H + STEP - 1) / STEP * STEP;
-    const int most = (33 * 1024 / (8 * nt) - 8) / (STEP * BP_DEPTH) * (STEP * BP_DEPTH);
-    if (kc > most) kc = most;
-    size_t smem = (size_t)8 * nt * (kc + 8) * 2;
-    const size_t sums = (size_t)BP_WARPS * BP_ROWS * (8 * nt + 1) * 4;
-    if (smem < sums) smem = sums;
-#define GO(NT) do { \
+    const int N = seg.row0[count];
+    const size_t smem = (size_t)8 * nt * (kc + 8) * 2 + (size_t)2 * BP_WARPS * BP_ROWS * (8 * nt + 1) * 4;
+#define GO(NT, D) do { \
         static bool raised = false; \
         if (!raised) { \
-            const cudaError_t e = cudaFuncSetAttribute(blended_product_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024); \
+            const cudaError_t e = cudaFuncSetAttribute(blended_product_kernel<NT, D>, cudaFuncAttributeMaxDynamicSharedMemorySize, 110 * 1024); \
             if (e != cudaSuccess) return 1000 + (int)e; \
             raised = true; \
         } \
-        return wllm_launch(blended_product_kernel<NT>, tiles, BP_WARPS * 32, smem, stream, (const bf16*)h, n, H, mu, (const bf16*)w, seg, positions, \
-                           token_req, req_q_len, req_slot, (bf16*)kept, out, N, kc); \
+        return wllm_launch(blended_product_kernel<NT, D>, tiles, BP_WARPS * 32, smem, stream, (const bf16*)h, n, H, mu, (const bf16*)w, seg, positions, \
+                           token_req, req_q_len, req_slot, (bf16*)kept, out, N, kc, subs); \
     } while (0)
-    if (nt == 1) GO(1);
-    if (nt == 2) GO(2);
-    GO(4);
+    if (nt == 1) GO(1, 8);
+    if (nt == 2) GO(2, 8);
+    GO(4, 4);
 #undef GO
 }
