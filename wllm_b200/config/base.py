@@ -57,6 +57,17 @@ class ConfigReader:
     def optional_integer(self, key: str):
         return self._get(key, None, int)
 
+    def nested(self, value: Any, where: str):
+        """A reader for an object inside this one (None, with a complaint, when it is no object); `absorb` takes its problems over."""
+        if not isinstance(value, dict):
+            self.complain(f"{where} must be an object")
+            return None
+        return ConfigReader(value, where)
+
+    def absorb(self, inner: "ConfigReader") -> None:
+        self.problems.extend(f"{inner.where}: {p}" for p in inner.problems)
+        inner.problems = []
+
     def complain(self, text: str) -> None:
         self.problems.append(text)
 

@@ -120,16 +120,17 @@ WLLM_API int wllm_unit_act(const void* in, void* out, int dtype, int act, long l
     return WLLM_BAD_DTYPE;
 }
 
-// The heads' outputs times a sigmoid gate: x[n, c] *= sigmoid(g[n, c]), c < width.  The gate's row comes as `parts` partial
-// sums (slabs `part_stride` elements apart, added in order) or as one tensor; the sigmoid and the product are 32-bit, rounded once.
+// The heads' outputs times a sigmoid gate: x[n, c] *= sigmoid(g[n, c / per]), c < width (per 1: a gate per element; the head size: one
+// number per head).  The gate's row comes as `parts` partial sums (slabs `part_stride` elements apart, added in order) or as one
+// tensor; the sigmoid and the product are 32-bit, rounded once.
 template <typename TX, typename TG>
 __global__ void sigmoid_gate_kernel(TX* __restrict__ x, int x_stride, const TG* __restrict__ g, int g_stride, int parts,
-                                    size_t part_stride, int n, int width) {
+                                    size_t part_stride, int n, int width, int per) {
     pdl_begin();
     const size_t total = (size_t)n * width;
     for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
         const size_t t = idx / width, c = idx % width;
-        const TG* src = g + t * g_stride + c;
+        const TG* src = g + t * g_stride + (per == 1 ? c : c / per);
         float z = to_f32(src[0]);
         for (int s = 1; s < parts; ++s) z += to_f32(src[(size_t)s * part_stride]);
         TX* dst = x + t * x_stride + c;
@@ -138,13 +139,13 @@ __global__ void sigmoid_gate_kernel(TX* __restrict__ x, int x_stride, const TG* 
 }
 
 WLLM_API int wllm_sigmoid_gate(void* x, int x_dtype, int x_stride, const void* g, int g_dtype, int g_stride, int parts,
-                               long long part_stride, int n, int width, cudaStream_t stream) {
+                               long long part_stride, int n, int width, int per, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
-    if (width <= 0 || parts < 1) return WLLM_BAD_SIZE;
+    if (width <= 0 || parts < 1 || per < 1) return WLLM_BAD_SIZE;
     const long long want = ((long long)n * width + 255) / 256;
     const int blocks = (int)(want < 148 * 16 ? want : 148 * 16);
 #define GO(TX, TG) wllm_launch(sigmoid_gate_kernel<TX, TG>, blocks, 256, 0, stream, (TX*)x, x_stride, (const TG*)g, g_stride, parts, \
-                               (size_t)part_stride, n, width)
+                               (size_t)part_stride, n, width, per)
     if (x_dtype == WLLM_BF16 && g_dtype == WLLM_BF16) return GO(bf16, bf16);
     if (x_dtype == WLLM_BF16 && g_dtype == WLLM_F32) return GO(bf16, float);
     if (x_dtype == WLLM_F32 && g_dtype == WLLM_F32) return GO(float, float);

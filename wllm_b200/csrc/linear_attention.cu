@@ -14,7 +14,9 @@
 //                           scaled, v copied, and the decay of every key channel worked out from a low-rank map:
 //                               z = W2 (x W1^T) + b,   a = sigmoid(z)^(1/tau) = exp(log_sigmoid(z) / tau)
 //                           or (decay form 1)  z = W2 tanh(x W1^T) + b,   a = exp(-exp(z)), handed on as a - 1; the decay alone
-//                           where q, k and v are read from the projections as they are
+//                           where q, k and v are read from the projections as they are; or (form 2)  z = W2 (x W1^T) + b,
+//                               a - 1 = expm1(-exp(A_log_h) softplus(z))
+//                           or (form 3) z = W2 (x W1^T) itself (a low-rank gate, which its reader passes through a sigmoid)
 //   wllm_linattn_scan       the recurrence.  Grid (tiles of 64 value columns, heads, requests); a lane owns two
 //                           columns of S, a warp a run of at most 16 key channels of them, in registers.  Tokens
 //                           arrive in tiles of 8 through a two-stage cp.async ring; the warps' partial dot products of a
@@ -25,8 +27,10 @@
 //                           key and value counted u times: o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t (time mixing).  There
 //                           the decays come as a - 1 (S + ((a - 1) S + k v)): a channel that forgets slowly has a close to one, and
 //                           the rounding of a itself, the same at every token, would grow with its memory.
-//   wllm_head_gate_norm     per head: o / sqrt(mean(o^2) + eps) [* w] * silu(g) [* factor], rounded once to the matrix type
-//                           (the operand of the output projection).  w is shared by the heads or a gain of the whole row.
+//                           With a pair (a - 1, step) per head and token (a state space, state_space.cu) the values are multiplied by
+//                           the step on the way, S + ((a - 1) S + k (step v)), and several heads may share a row of q and k.
+//   wllm_head_gate_norm     per head: o / sqrt(mean(o^2) + eps) [* w] * act(g) [* factor], act = silu or sigmoid, rounded once to the matrix
+//                           type (the operand of the output projection).  w is shared by the heads or a gain of the whole row.
 #include "common.cuh"
 
 __device__ __forceinline__ float la_any(const void* p, int dtype, size_t i) {
@@ -56,6 +60,16 @@ __device__ __forceinline__ float la_in(const void* p, int dtype, int parts, size
 // ---------------------------------------------------------------------------------------------------
 constexpr int PREP_RK = 32;      // columns of the low-rank map taken at a time
 
+// What a row z of the low-rank map becomes, by form (see the head of this file); rate = exp(A_log_h) of form 2
+__device__ __forceinline__ float lowrank_out(int form, float z, float inv_tau, float rate) {
+    if (form == 1) return expm1f(-expf(z));
+    if (form == 2) return expm1f(-rate * (z > 20.f ? z : log1pf(expf(z))));
+    if (form == 3) return z;
+    // log(sigmoid(z)) = min(z, 0) - log(1 + e^-|z|), exact at both ends
+    const float log_sig = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+    return expf(log_sig * inv_tau);
+}
+
 // TT tokens a CTA: the head's slab of the low-rank matrix is read once for all of them (prompts: 8); a step of few
 // tokens takes one token a CTA, so that tokens x heads CTAs share the work.
 template <int TT, bool MULTI>
@@ -65,7 +79,7 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
                        const int* __restrict__ positions, const float* __restrict__ inv_freq, int rot_dim,
                        float q_scale, float k_scale, const void* __restrict__ w2, const void* __restrict__ b2,
                        int w_dtype, float inv_tau, float* __restrict__ q, float* __restrict__ k,
-                       float* __restrict__ v, float* __restrict__ decay, int form) {
+                       float* __restrict__ v, float* __restrict__ decay, int form, const void* __restrict__ a_log) {
     __shared__ __align__(16) float low_s[PREP_RK][TT];      // the tokens' low-rank vectors, a run of PREP_RK columns at a time
     pdl_begin();
     const int t_lo = blockIdx.x * TT, h = blockIdx.y;
@@ -102,11 +116,12 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
     // thread takes PREP_RK of its channel's weights into registers at a time (16-byte loads where the rows allow), the
     // tokens' low-rank vectors come from shared memory.  The sum over r runs in ascending order whatever the tiling.
     const bool vec = ((uintptr_t)w2 & 15) == 0 && rank % 8 == 0;
+    const float rate = form == 2 ? expf(la_any(a_log, w_dtype, h)) : 0.f;
     for (int c0 = 0; c0 < D; c0 += 128) {
         const int c = c0 + threadIdx.x;
         const size_t ch = (size_t)h * D + min(c, D - 1);
         float z[TT];
-        const float bias = la_any(b2, w_dtype, ch);
+        const float bias = b2 ? la_any(b2, w_dtype, ch) : 0.f;
 #pragma unroll
         for (int tt = 0; tt < TT; ++tt) z[tt] = bias;
         for (int r0 = 0; r0 < rank; r0 += PREP_RK) {
@@ -159,16 +174,14 @@ linattn_prepare_kernel(const void* __restrict__ fused, int in_dtype, int row_str
 #pragma unroll
             for (int tt = 0; tt < TT; ++tt) {
                 if (tt >= count) break;
-                // log(sigmoid(z)) = min(z, 0) - log(1 + e^-|z|), exact at both ends
-                const float log_sig = fminf(z[tt], 0.f) - log1pf(expf(-fabsf(z[tt])));
-                decay[((size_t)(t_lo + tt) * H + h) * D + c] = form == 1 ? expm1f(-expf(z[tt])) : expf(log_sig * inv_tau);
+                decay[((size_t)(t_lo + tt) * H + h) * D + c] = lowrank_out(form, z[tt], inv_tau, rate);
             }
         }
     }
 }
 
-// The decay of time mixing for many tokens, bfloat16 maps, on the tensor cores (mma.sync): a CTA takes 64 tokens, whose tanh'd low-rank
-// rows it holds in shared memory as a high and a low bfloat16 piece each (together some sixteen bits), and walks tiles of 128
+// The low-rank maps of forms 1 to 3 for many tokens, bfloat16 maps, on the tensor cores (mma.sync): a CTA takes 64 tokens, whose low-rank
+// rows (form 1: through tanh) it holds in shared memory as a high and a low bfloat16 piece each (together some sixteen bits), and walks tiles of 128
 // channels; 2 x 4 warps, 32 tokens by 32 channels each.  grid (CTAs that share the channels' tiles, tiles of tokens), 256 threads.
 constexpr int DEC_TM = 64, DEC_TN = 128, DEC_MAX_RANK = 256;
 
@@ -182,10 +195,11 @@ __device__ __forceinline__ void dec_ldsm4(const bf16* p, uint32_t (&r)[4]) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 
-template <bool MULTI>
+template <bool MULTI, int FORM>
 __global__ void __launch_bounds__(256)
 linattn_decay_mma_kernel(const void* __restrict__ low, int in_dtype, int row_stride, int parts, size_t part_stride, int a_off, int n, int HD,
-                         int rank, const bf16* __restrict__ w2, const bf16* __restrict__ b2, float* __restrict__ decay) {
+                         int rank, const bf16* __restrict__ w2, const bf16* __restrict__ b2, float* __restrict__ decay,
+                         const bf16* __restrict__ a_log, int D) {
     extern __shared__ __align__(16) unsigned char dec_smem[];
     const int kp = (rank + 15) & ~15, pitch = kp + 8;
     bf16* hi = reinterpret_cast<bf16*>(dec_smem);        // [64][pitch]
@@ -196,7 +210,8 @@ linattn_decay_mma_kernel(const void* __restrict__ low, int in_dtype, int row_str
     for (int idx = threadIdx.x; idx < DEC_TM * kp; idx += 256) {
         const int tt = idx / kp, r = idx - tt * kp;
         float v = 0.f;
-        if (t0 + tt < n && r < rank) v = tanhf(la_in<MULTI>(low, in_dtype, parts, part_stride, (size_t)(t0 + tt) * row_stride + a_off + r));
+        if (t0 + tt < n && r < rank) v = la_in<MULTI>(low, in_dtype, parts, part_stride, (size_t)(t0 + tt) * row_stride + a_off + r);
+        if (FORM == 1) v = tanhf(v);
         const bf16 h = __float2bfloat16_rn(v);
         hi[tt * pitch + r] = h;
         lo[tt * pitch + r] = __float2bfloat16_rn(v - __bfloat162float(h));
@@ -236,6 +251,15 @@ linattn_decay_mma_kernel(const void* __restrict__ low, int in_dtype, int row_str
                     dec_mma(acc[mi][2 * nj + 1], ah[mi], bw[nj][2], bw[nj][3]);
                 }
         }
+        float bias[4][2], rate[4][2];                    // of the lane's eight channels
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int ch = min(tile * DEC_TN + wn * 32 + j * 8 + (lane & 3) * 2 + e, HD - 1);
+                bias[j][e] = b2 ? __bfloat162float(b2[ch]) : 0.f;
+                rate[j][e] = FORM == 2 ? expf(__bfloat162float(a_log[ch / D])) : 0.f;
+            }
 #pragma unroll
         for (int mi = 0; mi < 2; ++mi)
 #pragma unroll
@@ -243,48 +267,57 @@ linattn_decay_mma_kernel(const void* __restrict__ low, int in_dtype, int row_str
                 const int t = t0 + wm * 32 + mi * 16 + (lane >> 2) + half * 8;
                 if (t >= n) continue;
 #pragma unroll
-                for (int j = 0; j < 4; ++j)
-#pragma unroll
-                    for (int e = 0; e < 2; ++e) {
-                        const int ch = tile * DEC_TN + wn * 32 + j * 8 + (lane & 3) * 2 + e;
-                        if (ch < HD) decay[(size_t)t * HD + ch] = expm1f(-expf(acc[mi][j][half * 2 + e] + __bfloat162float(b2[ch])));
+                for (int j = 0; j < 4; ++j) {
+                    const int ch = tile * DEC_TN + wn * 32 + j * 8 + (lane & 3) * 2;
+                    float* dst = decay + (size_t)t * HD + ch;
+                    const float y0 = lowrank_out(FORM, acc[mi][j][half * 2] + bias[j][0], 0.f, rate[j][0]);
+                    const float y1 = lowrank_out(FORM, acc[mi][j][half * 2 + 1] + bias[j][1], 0.f, rate[j][1]);
+                    if (ch + 1 < HD && (HD & 1) == 0) *reinterpret_cast<float2*>(dst) = make_float2(y0, y1);
+                    else {
+                        if (ch < HD) dst[0] = y0;
+                        if (ch + 1 < HD) dst[1] = y1;
                     }
+                }
             }
     }
 }
 
-// q null: q, k and v stay where they are and only the decay is worked out.  form 0: sigmoid(z)^(1/tau); 1: exp(-exp(z)) - 1 over tanh
-// of the low-rank columns (tau is not used).
+// q null: q, k and v stay where they are and only the map is worked out.  form 0: sigmoid(z)^(1/tau); 1: exp(-exp(z)) - 1 over tanh
+// of the low-rank columns; 2: exp(-exp(a_log[h]) softplus(z)) - 1; 3: z (tau is not used by 1 to 3; b2 may be null; a_log is of form 2).
 WLLM_API int wllm_linattn_prepare_form(const void* fused, int in_dtype, int row_stride, int parts, long long part_stride, int q_off,
                                        int k_off, int v_off, int a_off, int n, int H, int D, int V, int rank, const int* positions,
                                        const float* inv_freq, int rot_dim, float q_scale, float k_scale, const void* w2,
                                        const void* b2, int w_dtype, float tau, float* q, float* k, float* v, float* decay, int form,
-                                       cudaStream_t stream) {
+                                       const void* a_log, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
-    if (H <= 0 || H > 65535 || D <= 0 || V <= 0 || parts < 1 || rot_dim < 0 || rot_dim > D || (rot_dim & 1) || form < 0 || form > 1) return WLLM_BAD_SIZE;
-    if (a_off >= 0 && (rank <= 0 || !(tau > 0.f) || !w2 || !b2 || !decay)) return WLLM_BAD_SIZE;
+    if (H <= 0 || H > 65535 || D <= 0 || V <= 0 || parts < 1 || rot_dim < 0 || rot_dim > D || (rot_dim & 1) || form < 0 || form > 3) return WLLM_BAD_SIZE;
+    if (a_off >= 0 && (rank <= 0 || !(tau > 0.f) || !w2 || !decay || (form == 2 && !a_log))) return WLLM_BAD_SIZE;
     if ((in_dtype != WLLM_BF16 && in_dtype != WLLM_F32) || (a_off >= 0 && w_dtype != WLLM_BF16 && w_dtype != WLLM_F32))
         return WLLM_BAD_DTYPE;
-    if (q == nullptr && form == 1 && a_off >= 0 && n >= 64 && w_dtype == WLLM_BF16 && rank % 8 == 0 && rank <= DEC_MAX_RANK && ((uintptr_t)w2 & 15) == 0) {
+    if (q == nullptr && form >= 1 && a_off >= 0 && n >= 64 && w_dtype == WLLM_BF16 && rank % 8 == 0 && rank <= DEC_MAX_RANK && ((uintptr_t)w2 & 15) == 0) {
         const int HD = H * D, row_tiles = (n + DEC_TM - 1) / DEC_TM, col_tiles = (HD + DEC_TN - 1) / DEC_TN;
         int share = (2 * 148 + row_tiles - 1) / row_tiles;           // CTAs that share a tile of tokens: some two CTAs an SM in all
         if (share > col_tiles) share = col_tiles;
         const size_t smem = (size_t)(2 * DEC_TM + DEC_TN) * (((rank + 15) & ~15) + 8) * sizeof(bf16);
         static bool raised = false;
         if (!raised) {
-            cudaError_t e = cudaFuncSetAttribute(linattn_decay_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
-            if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_decay_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+            cudaError_t e = cudaSuccess;
+#define RAISE(M, F) if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_decay_mma_kernel<M, F>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)
+            RAISE(true, 1); RAISE(false, 1); RAISE(true, 2); RAISE(false, 2); RAISE(true, 3); RAISE(false, 3);
+#undef RAISE
             if (e != cudaSuccess) return 1000 + (int)e;
             raised = true;
         }
-#define DEC(M) wllm_launch(linattn_decay_mma_kernel<M>, dim3(share, row_tiles), 256, smem, stream, fused, in_dtype, row_stride, parts, \
-        (size_t)part_stride, a_off, n, HD, rank, (const bf16*)w2, (const bf16*)b2, decay)
+#define DEC2(M, F) wllm_launch(linattn_decay_mma_kernel<M, F>, dim3(share, row_tiles), 256, smem, stream, fused, in_dtype, row_stride, parts, \
+        (size_t)part_stride, a_off, n, HD, rank, (const bf16*)w2, (const bf16*)b2, decay, (const bf16*)a_log, D)
+#define DEC(M) (form == 1 ? DEC2(M, 1) : form == 2 ? DEC2(M, 2) : DEC2(M, 3))
         return parts > 1 ? DEC(true) : DEC(false);
 #undef DEC
+#undef DEC2
     }
 #define PREP2(TT, M) wllm_launch(linattn_prepare_kernel<TT, M>, dim3((n + TT - 1) / TT, H), 128, 0, stream, fused, \
         in_dtype, row_stride, parts, (size_t)part_stride, q_off, k_off, v_off, a_off, n, H, D, V, rank, positions, \
-        inv_freq, rot_dim, q_scale, k_scale, w2, b2, w_dtype, a_off >= 0 ? 1.0f / tau : 0.f, q, k, v, decay, form)
+        inv_freq, rot_dim, q_scale, k_scale, w2, b2, w_dtype, a_off >= 0 ? 1.0f / tau : 0.f, q, k, v, decay, form, a_log)
 #define PREP(TT) (parts > 1 ? PREP2(TT, true) : PREP2(TT, false))
     if ((long long)n * H >= 2048) return PREP(8);
     return PREP(1);
@@ -299,7 +332,7 @@ WLLM_API int wllm_linattn_prepare(const void* fused, int in_dtype, int row_strid
                                   cudaStream_t stream) {
     if (q == nullptr) return WLLM_BAD_SIZE;
     return wllm_linattn_prepare_form(fused, in_dtype, row_stride, parts, part_stride, q_off, k_off, v_off, a_off, n, H, D, V, rank, positions,
-                                     inv_freq, rot_dim, q_scale, k_scale, w2, b2, w_dtype, tau, q, k, v, decay, 0, stream);
+                                     inv_freq, rot_dim, q_scale, k_scale, w2, b2, w_dtype, tau, q, k, v, decay, 0, nullptr, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------
@@ -333,15 +366,17 @@ __device__ __forceinline__ void la_cp16(float* smem_dst, const float* src) {    
 // a read left the kernel waiting for shared memory (a read a multiply-add).
 // FULL: every warp holds LA_CPT channels (the head's key size is a multiple of 16): the loops carry no guards.
 // BONUS: the output is S_(t-1)^T q + (q . (u k)) v, taken channel by channel in front of the update, and the decays are a - 1.
-// q, k and v are rows `q_stride`, `k_stride`, `v_stride` elements apart.
-template <bool PER_CHANNEL, int MODE, bool FULL, bool BONUS>
+// q, k and v are rows `q_stride`, `k_stride`, `v_stride` elements apart; `share` neighbouring heads read the same head of q and k.
+// DECAY: 0 one constant per head (`head_decay`), 1 per key channel and token, 2 a pair (a - 1, step) per head and token in `decay`.
+template <int DECAY, int MODE, bool FULL, bool BONUS>
 __global__ void __launch_bounds__(512)
 linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v,
                     const float* __restrict__ decay, const float* __restrict__ head_decay, float* __restrict__ state,
                     float* __restrict__ out, const int* __restrict__ req_q_start, const int* __restrict__ req_q_len,
                     const int* __restrict__ req_slot, int H, int D, int V, int cpt, int seg_len, int max_seg,
                     float* __restrict__ seg_state, float* __restrict__ seg_decay, size_t q_stride, size_t k_stride, size_t v_stride,
-                    const float* __restrict__ bonus) {
+                    const float* __restrict__ bonus, int share) {
+    constexpr bool PER_CHANNEL = DECAY == 1, STEP = DECAY == 2, MINUS_ONE = BONUS || STEP;
     extern __shared__ __align__(16) float la_smem[];
     pdl_begin();
     const int r = MODE == 0 ? blockIdx.z : blockIdx.z / max_seg, seg = MODE == 0 ? 0 : blockIdx.z % max_seg, h = blockIdx.y;
@@ -359,7 +394,8 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
     // shared memory: two stages of [q | k | (a) | v] for LA_TT tokens (each run of D padded to a multiple of 4), then
     // two rounds of the warps' partial sums
     const int Dp = (D + 3) & ~3, NA = PER_CHANNEL ? 3 : 2;
-    const int per_token = NA * Dp + LA_COLS;
+    const int per_token = NA * Dp + LA_COLS + (STEP ? 4 : 0);      // STEP: the pair behind the value columns
+    const int hk = h / share;                                 // the head's row of q and k
     float* stage0 = la_smem;
     float* red = la_smem + 2 * LA_TT * per_token;             // [2][warps][LA_TT][64]
 
@@ -373,10 +409,10 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
         const bool ch = MODE != 1 && (FULL || c_lo + i < c_hi);
         S0[i] = (ch && col0) ? St[(size_t)(c_lo + i) * V + j0] : 0.f;
         S1[i] = (ch && col1) ? St[(size_t)(c_lo + i) * V + j1] : 0.f;
-        P[i] = BONUS ? 0.f : 1.f;
+        P[i] = MINUS_ONE ? 0.f : 1.f;
         U[i] = BONUS && (FULL || c_lo + i < c_hi) ? bonus[h * D + c_lo + i] : 0.f;
     }
-    const float fixed = PER_CHANNEL ? 0.f : head_decay[h];
+    const float fixed = DECAY == 0 ? head_decay[h] : 0.f;
 
     // rows of whole 16-byte pieces (key sizes in steps of 16, value sizes in steps of 4, aligned buffers): a warp a token,
     // a lane a piece of q, k and the decay, sixteen lanes a piece of v; no division, a quarter of the copies
@@ -389,8 +425,8 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
         if (pieces) {
             for (int tt = warp; tt < count; tt += warps) {
                 const size_t at = ((size_t)(first + tt) * H + h) * D;
-                const float* qrow = q + (size_t)(first + tt) * q_stride + (size_t)h * D;
-                const float* krow = k + (size_t)(first + tt) * k_stride + (size_t)h * D;
+                const float* qrow = q + (size_t)(first + tt) * q_stride + (size_t)hk * D;
+                const float* krow = k + (size_t)(first + tt) * k_stride + (size_t)hk * D;
                 float* d = dst + tt * per_token;
                 for (int c = 4 * lane; c < D; c += 128) {
                     la_cp16(d + c, qrow + c);
@@ -403,6 +439,9 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
                     if (cc + 3 < V) la_cp16(d + NA * Dp + 4 * lane, vrow + cc);
                     else
                         for (int e = 0; e < 4; ++e) la_cp4(d + NA * Dp + 4 * lane + e, vrow + min(cc + e, V - 1));
+                } else if (STEP && lane < LA_COLS / 4 + 2) {
+                    const int e = lane - LA_COLS / 4;
+                    la_cp4(d + NA * Dp + LA_COLS + e, decay + ((size_t)(first + tt) * H + h) * 2 + e);
                 }
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
@@ -412,8 +451,8 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
             const int tt = idx / D, c = idx - tt * D;
             const size_t at = ((size_t)(first + tt) * H + h) * D + c;
             float* d = dst + tt * per_token + c;
-            la_cp4(d, q + (size_t)(first + tt) * q_stride + (size_t)h * D + c);
-            la_cp4(d + Dp, k + (size_t)(first + tt) * k_stride + (size_t)h * D + c);
+            la_cp4(d, q + (size_t)(first + tt) * q_stride + (size_t)hk * D + c);
+            la_cp4(d + Dp, k + (size_t)(first + tt) * k_stride + (size_t)hk * D + c);
             if (PER_CHANNEL) la_cp4(d + 2 * Dp, decay + at);
         }
         for (int idx = threadIdx.x; idx < count * LA_COLS; idx += blockDim.x) {
@@ -421,6 +460,9 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
             la_cp4(dst + tt * per_token + NA * Dp + cc,
                    v + (size_t)(first + tt) * v_stride + (size_t)h * V + min(blockIdx.x * LA_COLS + cc, V - 1));
         }
+        if (STEP)
+            for (int idx = threadIdx.x; idx < 2 * count; idx += blockDim.x)
+                la_cp4(dst + (idx >> 1) * per_token + NA * Dp + LA_COLS + (idx & 1), decay + ((size_t)(first + (idx >> 1)) * H + h) * 2 + (idx & 1));
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
 
@@ -444,13 +486,15 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
             p0[tt] = p1[tt] = 0.f;
             if (tt < count) {
                 const float* qs = base + tt * per_token;
-                const float v0 = qs[NA * Dp + lane], v1 = qs[NA * Dp + 32 + lane];
+                const float less = STEP ? qs[NA * Dp + LA_COLS] : fixed, step = STEP ? qs[NA * Dp + LA_COLS + 1] : 1.f;
+                const float v0 = STEP ? qs[NA * Dp + lane] * step : qs[NA * Dp + lane];
+                const float v1 = STEP ? qs[NA * Dp + 32 + lane] * step : qs[NA * Dp + 32 + lane];
 #pragma unroll
                 for (int i4 = 0; i4 < LA_CPT; i4 += 4) {
                     if (FULL || c_lo + i4 < c_hi) {
                         const float4 q4 = *reinterpret_cast<const float4*>(qs + c_lo + i4);
                         const float4 k4 = *reinterpret_cast<const float4*>(qs + Dp + c_lo + i4);
-                        float4 a4 = make_float4(fixed, fixed, fixed, fixed);
+                        float4 a4 = make_float4(less, less, less, less);
                         if (PER_CHANNEL) a4 = *reinterpret_cast<const float4*>(qs + 2 * Dp + c_lo + i4);
                         const float qe[4] = {q4.x, q4.y, q4.z, q4.w}, ke[4] = {k4.x, k4.y, k4.z, k4.w}, ae[4] = {a4.x, a4.y, a4.z, a4.w};
 #pragma unroll
@@ -461,14 +505,14 @@ linattn_scan_kernel(const float* __restrict__ q, const float* __restrict__ k, co
                                     p0[tt] = fmaf(fmaf(uk, v0, S0[i4 + e]), qe[e], p0[tt]);
                                     p1[tt] = fmaf(fmaf(uk, v1, S1[i4 + e]), qe[e], p1[tt]);
                                 }
-                                if (BONUS) {
+                                if (MINUS_ONE) {
                                     S0[i4 + e] += fmaf(ae[e], S0[i4 + e], ke[e] * v0);
                                     S1[i4 + e] += fmaf(ae[e], S1[i4 + e], ke[e] * v1);
                                 } else {
                                     S0[i4 + e] = fmaf(ae[e], S0[i4 + e], ke[e] * v0);
                                     S1[i4 + e] = fmaf(ae[e], S1[i4 + e], ke[e] * v1);
                                 }
-                                if (MODE == 1) P[i4 + e] = BONUS ? P[i4 + e] + fmaf(ae[e], P[i4 + e], ae[e]) : P[i4 + e] * ae[e];
+                                if (MODE == 1) P[i4 + e] = MINUS_ONE ? P[i4 + e] + fmaf(ae[e], P[i4 + e], ae[e]) : P[i4 + e] * ae[e];
                                 else if (!BONUS) {
                                     p0[tt] = fmaf(S0[i4 + e], qe[e], p0[tt]);
                                     p1[tt] = fmaf(S1[i4 + e], qe[e], p1[tt]);
@@ -555,39 +599,43 @@ __global__ void linattn_combine_kernel(const float* __restrict__ state, const in
 // must cover the longest portion); seg_state holds requests * max_seg * H * D * V floats, seg_decay requests * max_seg * H * D.
 // q_stride, k_stride, v_stride: elements between two tokens' rows (H * D, H * D and H * V where the rows lie one behind the other).
 // bonus [H, D] (null: none): time mixing, see above; with a decay per key channel, given as a - 1.
-WLLM_API int wllm_linattn_scan_rows(const float* q, const float* k, const float* v, long long q_stride, long long k_stride,
-                                    long long v_stride, const float* decay, const float* head_decay, const float* bonus, float* state,
-                                    float* out, const int* req_q_start, const int* req_q_len, const int* req_slot, int requests, int H,
-                                    int D, int V, int seg_len, int max_seg, float* seg_state, float* seg_decay, cudaStream_t stream) {
+// pairs: decay holds [n, H, 2] = (a - 1, step) instead; share: neighbouring heads that read the same head of q and k (rows of H / share heads).
+WLLM_API int wllm_linattn_scan_shared(const float* q, const float* k, const float* v, long long q_stride, long long k_stride,
+                                      long long v_stride, const float* decay, int pairs, const float* head_decay, const float* bonus,
+                                      float* state, float* out, const int* req_q_start, const int* req_q_len, const int* req_slot,
+                                      int requests, int H, int share, int D, int V, int seg_len, int max_seg, float* seg_state,
+                                      float* seg_decay, cudaStream_t stream) {
     if (requests <= 0) return WLLM_OK;
     if (H <= 0 || H > 65535 || requests > 65535 || D <= 0 || D > 16 * LA_CPT || V <= 0) return WLLM_BAD_SIZE;
     if (!decay && !head_decay) return WLLM_BAD_SIZE;
-    if (bonus && !decay) return WLLM_BAD_SIZE;
-    if (q_stride < (long long)H * D || k_stride < (long long)H * D || v_stride < (long long)H * V) return WLLM_BAD_SIZE;
+    if ((bonus && (!decay || pairs)) || (pairs && !decay) || share < 1 || H % share != 0) return WLLM_BAD_SIZE;
+    if (q_stride < (long long)(H / share) * D || k_stride < (long long)(H / share) * D || v_stride < (long long)H * V) return WLLM_BAD_SIZE;
     const bool cut = seg_len > 0 && max_seg > 1;
     if (cut && (!seg_state || !seg_decay || (long long)requests * max_seg > 65535)) return WLLM_BAD_SIZE;
     const int most = (D + LA_CPT - 1) / LA_CPT;
     const int cpt = (((D + most - 1) / most) + 3) & ~3;          // a multiple of 4, at most LA_CPT
     const int warps = (D + cpt - 1) / cpt;
     const int vtiles = (V + LA_COLS - 1) / LA_COLS;
-    const size_t smem = ((size_t)2 * LA_TT * ((decay ? 3 : 2) * ((D + 3) & ~3) + LA_COLS) + 2 * warps * LA_TT * 64) * sizeof(float);
+    const size_t smem = ((size_t)2 * LA_TT * ((decay && !pairs ? 3 : 2) * ((D + 3) & ~3) + LA_COLS + (pairs ? 4 : 0)) +
+                         2 * warps * LA_TT * 64) * sizeof(float);
     const bool full = cpt == LA_CPT && D % LA_CPT == 0;
     static bool raised = false;
     if (!raised) {
         cudaError_t e = cudaSuccess;
 #define RAISE(PC, M, B) if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_scan_kernel<PC, M, true, B>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024); \
         if (e == cudaSuccess) e = cudaFuncSetAttribute(linattn_scan_kernel<PC, M, false, B>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024)
-        RAISE(true, 0, false); RAISE(true, 1, false); RAISE(true, 2, false); RAISE(false, 0, false); RAISE(false, 1, false); RAISE(false, 2, false);
-        RAISE(true, 0, true); RAISE(true, 1, true); RAISE(true, 2, true);
+        RAISE(1, 0, false); RAISE(1, 1, false); RAISE(1, 2, false); RAISE(0, 0, false); RAISE(0, 1, false); RAISE(0, 2, false);
+        RAISE(1, 0, true); RAISE(1, 1, true); RAISE(1, 2, true); RAISE(2, 0, false); RAISE(2, 1, false); RAISE(2, 2, false);
 #undef RAISE
         if (e != cudaSuccess) return 1000 + (int)e;
         raised = true;
     }
 #define SCAN2(PC, MODE, F, B, GRID) wllm_launch(linattn_scan_kernel<PC, MODE, F, B>, GRID, warps * 32, smem, stream, q, k, v, decay, head_decay, \
         state, out, req_q_start, req_q_len, req_slot, H, D, V, cpt, seg_len, max_seg, seg_state, seg_decay, (size_t)q_stride, (size_t)k_stride, \
-        (size_t)v_stride, bonus)
+        (size_t)v_stride, bonus, share)
 #define SCAN1(PC, MODE, B, GRID) (full ? SCAN2(PC, MODE, true, B, GRID) : SCAN2(PC, MODE, false, B, GRID))
-#define SCAN(MODE, GRID) (bonus ? SCAN1(true, MODE, true, GRID) : decay ? SCAN1(true, MODE, false, GRID) : SCAN1(false, MODE, false, GRID))
+#define SCAN(MODE, GRID) (bonus ? SCAN1(1, MODE, true, GRID) : pairs ? SCAN1(2, MODE, false, GRID) : decay ? SCAN1(1, MODE, false, GRID) \
+                                                                                               : SCAN1(0, MODE, false, GRID))
     if (!cut) {
         const dim3 grid(vtiles, H, requests);
         return SCAN(0, grid);
@@ -596,12 +644,20 @@ WLLM_API int wllm_linattn_scan_rows(const float* q, const float* k, const float*
     int st = SCAN(1, grid);
     if (st != WLLM_OK) return st;
     st = wllm_launch(linattn_combine_kernel, dim3((D * V + 255) / 256, H, requests), 256, 0, stream, (const float*)state,
-                     req_q_len, req_slot, H, D, V, seg_len, max_seg, seg_state, (const float*)seg_decay, bonus != nullptr ? 1 : 0);
+                     req_q_len, req_slot, H, D, V, seg_len, max_seg, seg_state, (const float*)seg_decay, (bonus != nullptr || pairs) ? 1 : 0);
     if (st != WLLM_OK) return st;
     return SCAN(2, grid);
 #undef SCAN
 #undef SCAN1
 #undef SCAN2
+}
+
+WLLM_API int wllm_linattn_scan_rows(const float* q, const float* k, const float* v, long long q_stride, long long k_stride,
+                                    long long v_stride, const float* decay, const float* head_decay, const float* bonus, float* state,
+                                    float* out, const int* req_q_start, const int* req_q_len, const int* req_slot, int requests, int H,
+                                    int D, int V, int seg_len, int max_seg, float* seg_state, float* seg_decay, cudaStream_t stream) {
+    return wllm_linattn_scan_shared(q, k, v, q_stride, k_stride, v_stride, decay, 0, head_decay, bonus, state, out, req_q_start, req_q_len,
+                                    req_slot, requests, H, 1, D, V, seg_len, max_seg, seg_state, seg_decay, stream);
 }
 
 WLLM_API int wllm_linattn_scan(const float* q, const float* k, const float* v, const float* decay, const float* head_decay,
@@ -618,7 +674,8 @@ WLLM_API int wllm_linattn_scan(const float* q, const float* k, const float* v, c
 template <typename TO, bool MULTI>
 __global__ void head_gate_norm_kernel(const float* __restrict__ o, const void* __restrict__ fused, int in_dtype, int row_stride,
                                       int parts, size_t part_stride, int g_off, const void* __restrict__ w, int w_dtype,
-                                      float eps, TO* __restrict__ out, int H, int V, int w_head_stride, size_t out_stride, float factor) {
+                                      float eps, TO* __restrict__ out, int H, int V, int w_head_stride, size_t out_stride, float factor,
+                                      int sigmoid) {
     pdl_begin();
     const int t = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (h >= H) return;
@@ -632,20 +689,20 @@ __global__ void head_gate_norm_kernel(const float* __restrict__ o, const void* _
         const float g = la_in<MULTI>(fused, in_dtype, parts, part_stride, grow + c);
         float y = orow[c] * inv;
         if (w) y *= la_any(w, w_dtype, (size_t)h * w_head_stride + c);
-        out[(size_t)t * out_stride + (size_t)h * V + c] = from_f32<TO>(y * (g / (1.0f + expf(-g))) * factor);
+        out[(size_t)t * out_stride + (size_t)h * V + c] = from_f32<TO>(y * ((sigmoid ? 1.0f : g) / (1.0f + expf(-g))) * factor);
     }
 }
 
 // out[n, H*V] = o / sqrt(mean_V(o^2) + eps) * w[V] (w may be null) * silu(g) * factor, g = fused[:, g_off + h*V + c]; per_head: w is
-// [H*V], a gain of the whole row; out's rows are out_stride elements apart
+// [H*V], a gain of the whole row; sigmoid: sigmoid(g) in place of silu(g); out's rows are out_stride elements apart
 WLLM_API int wllm_head_gate_norm_rows(const float* o, const void* fused, int in_dtype, int row_stride, int parts,
                                       long long part_stride, int g_off, const void* w, int w_dtype, int per_head, float eps, void* out,
-                                      int out_dtype, int out_stride, float factor, int n, int H, int V, cudaStream_t stream) {
+                                      int out_dtype, int out_stride, float factor, int sigmoid, int n, int H, int V, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
     if (H <= 0 || H > 65535 || V <= 0 || parts < 1 || out_stride < H * V) return WLLM_BAD_SIZE;
     if ((in_dtype != WLLM_BF16 && in_dtype != WLLM_F32) || (w && w_dtype != WLLM_BF16 && w_dtype != WLLM_F32)) return WLLM_BAD_DTYPE;
 #define GATE(TO, M) wllm_launch(head_gate_norm_kernel<TO, M>, dim3(n, (H + 3) / 4), 128, 0, stream, o, fused, in_dtype, row_stride, parts, \
-        (size_t)part_stride, g_off, w, w_dtype, eps, (TO*)out, H, V, per_head ? V : 0, (size_t)out_stride, factor)
+        (size_t)part_stride, g_off, w, w_dtype, eps, (TO*)out, H, V, per_head ? V : 0, (size_t)out_stride, factor, sigmoid)
     if (out_dtype == WLLM_BF16) return parts > 1 ? GATE(bf16, true) : GATE(bf16, false);
     if (out_dtype == WLLM_F32) return parts > 1 ? GATE(float, true) : GATE(float, false);
 #undef GATE
@@ -655,6 +712,6 @@ WLLM_API int wllm_head_gate_norm_rows(const float* o, const void* fused, int in_
 WLLM_API int wllm_head_gate_norm(const float* o, const void* fused, int in_dtype, int row_stride, int parts,
                                  long long part_stride, int g_off, const void* w, int w_dtype, float eps, void* out,
                                  int out_dtype, int n, int H, int V, cudaStream_t stream) {
-    return wllm_head_gate_norm_rows(o, fused, in_dtype, row_stride, parts, part_stride, g_off, w, w_dtype, 0, eps, out, out_dtype, H * V, 1.0f,
+    return wllm_head_gate_norm_rows(o, fused, in_dtype, row_stride, parts, part_stride, g_off, w, w_dtype, 0, eps, out, out_dtype, H * V, 1.0f, 0,
                                     n, H, V, stream);
 }

@@ -21,12 +21,16 @@
 // (plus a small number), and end with identity experts: the last ones of its list, without matrices, whose output is the
 // token's row itself.  Their pairs are sorted behind all others, no product touches them, and the combine reads the row.
 //
-// Two more forms.  Scores: softmax over all experts, or (score_mode 1) sigmoid(z) expert by expert, not normalised (without
-// groups the experts are then chosen by z itself: the same order, and no ties where large logits all round to a score of 1).  Unit
+// The router's logits may carry a bias per expert (it counts for the choice and for the weights).
+//
+// More forms.  Scores: softmax over all experts, or (score_mode 1) sigmoid(z) expert by expert, not normalised (without
+// groups the experts are then chosen by z itself: the same order, and no ties where large logits all round to a score of 1), or
+// (score_mode 2) the experts are chosen by z and weighted by the softmax over the chosen z alone.  Unit
 // (MODE 2): an expert without a gate, down(relu(up (s a))^2), whose input is multiplied by the pair's score s: the up product
 // is linear, so s multiplies its 32-bit sums in front of the activation; the combine then adds the experts' outputs as they are.
 //
-// The gated unit is the clamped one: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(slope g) (u + 1).
+// The gated unit is the clamped one, g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(slope g) (u + shift) with
+// shift = 1; the plain SiLU unit is that with limit = infinity, slope = 1 and shift = 0.
 #include "common.cuh"
 
 constexpr int MOE_MAX_EXPERTS = 1024;
@@ -37,7 +41,8 @@ template <typename T>
 __global__ void __launch_bounds__(1024)
 moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ w_gate,
                  int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ gate_out, int n, int H, int E, int top,
-                 int groups, int groups_kept, int tpb, int score_mode, const float* __restrict__ correction, float renorm_eps) {
+                 int groups, int groups_kept, int tpb, int score_mode, const float* __restrict__ correction, float renorm_eps,
+                 const float* __restrict__ bias) {
     extern __shared__ float route_smem[];          // [tpb][H] the tokens' rows, [tpb][E] scores, [tpb][groups] group scores, [tpb][E] corrected scores
     float* hs_all = route_smem;
     float* sc_all = hs_all + (size_t)tpb * H;
@@ -80,7 +85,7 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
             for (int j = 0; j < TB; ++j) {
                 const float acc = warp_sum((a4[j][0] + a4[j][1]) + (a4[j][2] + a4[j][3]));
                 if (lane == 0 && j0 + j < here) {
-                    if (e < E) sc_all[(size_t)(j0 + j) * E + e] = acc; else gate_out[t0 + j0 + j] = 1.0f / (1.0f + expf(-acc));
+                    if (e < E) sc_all[(size_t)(j0 + j) * E + e] = bias ? acc + bias[e] : acc; else gate_out[t0 + j0 + j] = 1.0f / (1.0f + expf(-acc));
                 }
             }
         }
@@ -107,6 +112,30 @@ moe_route_kernel(const T* __restrict__ h, const float* __restrict__ w_router, co
                 }
                 __syncwarp();
             }
+            continue;
+        }
+        if (score_mode == 2) {                     // the best `top` logits, then their softmax (the first one is the largest)
+            float first = 0.f, total = 0.f;
+            for (int k = 0; k < top; ++k) {
+                float best = -INFINITY; int at = 0x7fffffff;
+                for (int e = lane; e < E; e += 32) { const float v = sc[e]; if (v > best) { best = v; at = e; } }
+                for (int o = 16; o > 0; o >>= 1) {
+                    const float ob = __shfl_xor_sync(0xffffffffu, best, o); const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+                    if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+                }
+                at = min(at, E - 1);                // (logits that are no numbers choose nothing; the index stays inside)
+                if (k == 0) first = best;
+                const float p = expf(best - first);
+                total += p;
+                if (lane == 0) {
+                    chosen[(size_t)t * top + k] = at;
+                    weights[(size_t)t * top + k] = p;
+                    sc[at] = -INFINITY;
+                }
+                __syncwarp();
+            }
+            if (lane == 0)
+                for (int k = 0; k < top; ++k) weights[(size_t)t * top + k] = weights[(size_t)t * top + k] / total;
             continue;
         }
         if (score_mode == 1) {
@@ -266,7 +295,7 @@ template <typename T, typename TO, int MODE>
 __global__ void __launch_bounds__(256)
 moe_grouped_kernel(const T* __restrict__ a, int a_stride, const T* __restrict__ w, TO* __restrict__ out, int N, int K,
                    const int* __restrict__ offset, const int* __restrict__ sorted, int E, int top, float limit, float slope,
-                   const float* __restrict__ row_w) {
+                   const float* __restrict__ row_w, float shift) {
     constexpr bool GATED = MODE == 1, GATHER = MODE != 0;
     __shared__ float As[GK][GM + 1];
     __shared__ float Ws[GATED ? 2 : 1][GK][GN + 1];
@@ -341,7 +370,7 @@ moe_grouped_kernel(const T* __restrict__ a, int a_stride, const T* __restrict__ 
             float v = acc[0][i][j];
             if (GATED) {
                 const float g = fminf(v, limit), u = fminf(fmaxf(acc[GATED ? 1 : 0][i][j], -limit), limit);
-                v = (g / (1.0f + expf(-slope * g))) * (u + 1.0f);
+                v = (g / (1.0f + expf(-slope * g))) * (u + shift);
             }
             if (MODE == 2) {
                 v = fmaxf(row_w ? v * row_w[sorted[row0 + r]] : v, 0.f);
@@ -404,7 +433,7 @@ template <typename TO, int MODE>
 __global__ void __launch_bounds__(256)
 moe_grouped_mma_kernel(const bf16* __restrict__ a, int a_stride, const bf16* __restrict__ w, TO* __restrict__ out, int N, int K,
                        const int* __restrict__ offset, const int* __restrict__ sorted, int E, int top, float limit, float slope,
-                       const float* __restrict__ row_w) {
+                       const float* __restrict__ row_w, float shift) {
     constexpr bool GATED = MODE == 1, GATHER = MODE != 0;
     extern __shared__ __align__(16) unsigned char moe_smem[];
     bf16 (*As)[TM][TPITCH] = reinterpret_cast<bf16 (*)[TM][TPITCH]>(moe_smem);
@@ -502,7 +531,7 @@ moe_grouped_mma_kernel(const bf16* __restrict__ a, int a_stride, const bf16* __r
                     float v = acc[mi][ni][half * 2 + c];
                     if (GATED) {
                         const float g = fminf(v, limit), u = fminf(fmaxf(acc[mi][ni + 2][half * 2 + c], -limit), limit);
-                        v = (g / (1.0f + expf(-slope * g))) * (u + 1.0f);
+                        v = (g / (1.0f + expf(-slope * g))) * (u + shift);
                     }
                     if (MODE == 2) { v = fmaxf(v * rw, 0.f); v *= v; }
                     orow[col] = from_f32<TO>(v);
@@ -599,12 +628,13 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ place, c
     }
 }
 
-// correction [E] (null: none): added to the scores for the choice; renorm_eps >= 0: the chosen scores over (their sum + renorm_eps)
+// correction [E] (null: none): added to the scores for the choice; renorm_eps >= 0: the chosen scores over (their sum + renorm_eps);
+// bias [E] (null: none): added to the logits
 WLLM_API int wllm_moe_route_corrected(const void* h, int dtype, const float* w_router, const float* w_gate, int* chosen, float* weights,
                                       float* gate_out, int n, int H, int E, int top, int groups, int groups_kept, int score_mode,
-                                      const float* correction, float renorm_eps, cudaStream_t stream) {
+                                      const float* correction, float renorm_eps, const float* bias, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
-    if (score_mode != 0 && score_mode != 1) return WLLM_BAD_SIZE;
+    if (score_mode < 0 || score_mode > 2 || (score_mode == 2 && (groups != 1 || correction != nullptr || renorm_eps >= 0.f))) return WLLM_BAD_SIZE;
     if (H <= 0 || E <= 0 || E > MOE_MAX_EXPERTS || top < 1 || groups < 1 || E % groups != 0 || groups_kept < 1 ||
         groups_kept > groups || top > groups_kept * (E / groups) || (w_gate != nullptr && gate_out == nullptr))
         return WLLM_BAD_SIZE;
@@ -622,7 +652,7 @@ WLLM_API int wllm_moe_route_corrected(const void* h, int dtype, const float* w_r
             if (er != cudaSuccess) return 1000 + (int)er; \
         } \
         return wllm_launch(moe_route_kernel<T>, (n + tpb - 1) / tpb, threads, smem, stream, (const T*)h, w_router, w_gate, chosen, weights, \
-                           gate_out, n, H, E, top, groups, groups_kept, tpb, score_mode, correction, renorm_eps); \
+                           gate_out, n, H, E, top, groups, groups_kept, tpb, score_mode, correction, renorm_eps, bias); \
     } while (0)
     if (dtype == WLLM_BF16) GO(bf16);
     if (dtype == WLLM_F32) GO(float);
@@ -634,7 +664,7 @@ WLLM_API int wllm_moe_route(const void* h, int dtype, const float* w_router, con
                             float* gate_out, int n, int H, int E, int top, int groups, int groups_kept, int score_mode,
                             cudaStream_t stream) {
     return wllm_moe_route_corrected(h, dtype, w_router, w_gate, chosen, weights, gate_out, n, H, E, top, groups, groups_kept, score_mode,
-                                    nullptr, -1.0f, stream);
+                                    nullptr, -1.0f, nullptr, stream);
 }
 
 // count [E], offset [E + 1], sorted [pairs], place [pairs]
@@ -702,18 +732,18 @@ WLLM_API int wllm_moe_gather(const void* x, int x_stride, const int* sorted, int
     return wllm_moe_gather_scaled(x, x_stride, sorted, top, out, pairs, K, nullptr, stream);
 }
 
-// unit = 1: a [n][K] rows of tokens (stride a_stride), w [E][2 N][K], out [pairs][N] of the operands' type (the clamped gated unit);
+// unit = 1: a [n][K] rows of tokens (stride a_stride), w [E][2 N][K], out [pairs][N] of the operands' type (the clamped gated unit with `shift`);
 // unit = 0: a [pairs][K] sorted rows, w [E][N][K], out [pairs][N] 32-bit;
 // unit = 2: a [n][K] rows of tokens, w [E][N][K], out [pairs][N] of the operands' type = relu(row_w[pair] * (w a))^2 (row_w null: 1).
 WLLM_API int wllm_moe_grouped_unit(const void* a, int a_stride, const void* w, void* out, int dtype, int unit, int pairs, int N, int K,
-                                   const int* offset, const int* sorted, int E, int top, float limit, float slope, const float* row_w,
-                                   cudaStream_t stream) {
+                                   const int* offset, const int* sorted, int E, int top, float limit, float slope, float shift,
+                                   const float* row_w, cudaStream_t stream) {
     if (pairs <= 0) return WLLM_OK;
     if (N <= 0 || K <= 0 || E <= 0 || E > MOE_MAX_EXPERTS || top < 1 || unit < 0 || unit > 2) return WLLM_BAD_SIZE;
     const dim3 grid((N + GN - 1) / GN, (pairs + GM - 1) / GM + E);
     if (grid.y > 65535) return WLLM_BAD_SIZE;
 #define GO(T, TO, M) wllm_launch(moe_grouped_kernel<T, TO, M>, grid, 256, 0, stream, (const T*)a, a_stride, (const T*)w, (TO*)out, N, K, \
-                                 offset, sorted, E, top, limit, slope, row_w)
+                                 offset, sorted, E, top, limit, slope, row_w, shift)
     if (dtype == WLLM_BF16 && K % 8 == 0 && a_stride % 8 == 0 && !((uintptr_t)a & 15) && !((uintptr_t)w & 15)) {
         const int cols = unit == 1 ? TN / 2 : TN;
         const dim3 tgrid((N + cols - 1) / cols, (pairs + TM - 1) / TM + E);
@@ -727,7 +757,7 @@ WLLM_API int wllm_moe_grouped_unit(const void* a, int a_stride, const void* w, v
             raised = true;
         }
 #define TGO(TO, M) wllm_launch(moe_grouped_mma_kernel<TO, M>, tgrid, 256, T_SMEM, stream, (const bf16*)a, a_stride, (const bf16*)w, \
-                               (TO*)out, N, K, offset, sorted, E, top, limit, slope, row_w)
+                               (TO*)out, N, K, offset, sorted, E, top, limit, slope, row_w, shift)
         return unit == 1 ? TGO(bf16, 1) : unit == 2 ? TGO(bf16, 2) : TGO(float, 0);
 #undef TGO
     }
@@ -739,7 +769,7 @@ WLLM_API int wllm_moe_grouped_unit(const void* a, int a_stride, const void* w, v
 
 WLLM_API int wllm_moe_grouped(const void* a, int a_stride, const void* w, void* out, int dtype, int gated, int pairs, int N, int K,
                               const int* offset, const int* sorted, int E, int top, float limit, float slope, cudaStream_t stream) {
-    return wllm_moe_grouped_unit(a, a_stride, w, out, dtype, gated ? 1 : 0, pairs, N, K, offset, sorted, E, top, limit, slope, nullptr, stream);
+    return wllm_moe_grouped_unit(a, a_stride, w, out, dtype, gated ? 1 : 0, pairs, N, K, offset, sorted, E, top, limit, slope, 1.0f, nullptr, stream);
 }
 
 // gate null: the shared unit joins as it is.  chosen (null: no identity experts) [n, top], real_experts, x [n, H]: see above.

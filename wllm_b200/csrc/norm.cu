@@ -324,9 +324,27 @@ WLLM_API int wllm_branch_norm(const void* a, int a_dtype, int a_parts, long long
                                    factor, 0.f, out, n, H, stream);
 }
 
+// out[n, H] (32-bit) = a + bias: a branch output (a tensor or `parts` 32-bit slabs, added in order) with the bias row of its projection
+template <bool MULTI>
+__global__ void branch_bias_kernel(const void* __restrict__ a, int a_dtype, int a_parts, size_t a_stride, const float* __restrict__ bias,
+                                   float* __restrict__ out, int H) {
+    pdl_begin();
+    const size_t row0 = (size_t)blockIdx.x * H;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) out[row0 + c] = parts_at<MULTI>(a, a_dtype, a_parts, a_stride, row0 + c) + bias[c];
+}
+
+WLLM_API int wllm_branch_bias(const void* a, int a_dtype, int a_parts, long long a_stride, const float* bias, float* out, int n, int H,
+                              cudaStream_t stream) {
+    if (n <= 0) return WLLM_OK;
+    if (H <= 0 || a_parts < 1 || bias == nullptr) return WLLM_BAD_SIZE;
+    if (a_dtype != WLLM_BF16 && a_dtype != WLLM_F32) return WLLM_BAD_DTYPE;
+    return a_parts > 1 ? wllm_launch(branch_bias_kernel<true>, n, 256, 0, stream, a, a_dtype, a_parts, (size_t)a_stride, bias, out, H)
+                       : wllm_launch(branch_bias_kernel<false>, n, 256, 0, stream, a, a_dtype, a_parts, (size_t)a_stride, bias, out, H);
+}
+
 // ---------------------------------------------------------------------------------------------------
 // A block that norms behind its sublayers as well as in front, in one kernel a row:
-//     u   = a                                             (one branch), or
+//     u   = a [+ bias]                                    (one branch; bias: one 32-bit row, joins the branch's finished sum), or
 //           factor * (rms(a) * wa + rms(b) * wb)          (two mixers side by side, each normed over the width)
 //     r  += norm_p(u) * (offset_p + wp)                   (the norm behind the sublayer; center_p: layer norm)
 //     out = norm(r) * (offset + w)                        (the norm in front of the next sublayer, or the model's last;
@@ -340,7 +358,7 @@ __global__ void sandwich_norm_kernel(float* __restrict__ resid, const void* __re
                                      size_t b_stride, const void* __restrict__ wb, float inner_eps, float factor,
                                      const void* __restrict__ wp, int center_p, float eps_p, const void* __restrict__ w,
                                      float offset, int center, float eps, int w_dtype, TO* __restrict__ out,
-                                     const int* __restrict__ rows, int H, float offset_p) {
+                                     const int* __restrict__ rows, int H, float offset_p, const float* __restrict__ bias) {
     extern __shared__ float row_s[];          // [H] the row between the passes; with two branches [H] more for the second
     __shared__ float scratch[32];
     pdl_begin();
@@ -351,7 +369,8 @@ __global__ void sandwich_norm_kernel(float* __restrict__ resid, const void* __re
     // the branches' parts are added once and kept: every later pass reads shared memory
     float ssa = 0.f, ssb = 0.f;
     for (int c = threadIdx.x; c < H; c += blockDim.x) {
-        const float x = parts_at<MULTI>(a, a_dtype, a_parts, a_stride, row0 + c);
+        float x = parts_at<MULTI>(a, a_dtype, a_parts, a_stride, row0 + c);
+        if (bias) x += bias[c];
         row_s[c] = x;
         ssa += x * x;
         if (b) { const float y = parts_at<MULTI>(b, b_dtype, b_parts, b_stride, row0 + c); row_b[c] = y; ssb += y * y; }
@@ -397,12 +416,13 @@ __global__ void sandwich_norm_kernel(float* __restrict__ resid, const void* __re
 
 // a, b: branch outputs [n, H] of either element type, or `parts` 32-bit slabs `stride` elements apart; wa null: a is taken as
 // it is (b, wb unused); all gains (wa, wb, wp, w) share one element type.
-// offset_p: the gain of the norm behind the sublayer is offset_p + wp; w null: the second norm is left out (out = r).
+// offset_p: the gain of the norm behind the sublayer is offset_p + wp; w null: the second norm is left out (out = r); bias (null: none)
+// [H]: added to a.
 WLLM_API int wllm_sandwich_norm_offset(float* resid, const void* a, int a_dtype, int a_parts, long long a_stride, const void* wa,
                                        const void* b, int b_dtype, int b_parts, long long b_stride, const void* wb, float inner_eps,
                                        float factor, const void* wp, float offset_p, int center_p, float eps_p, const void* w,
                                        float offset, int center, float eps, int w_dtype, void* out, int out_dtype,
-                                       const int* rows, int n, int H, cudaStream_t stream) {
+                                       const int* rows, int n, int H, const float* bias, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
     if (H <= 0 || H > 24 * 1024 || a_parts < 1 || (b && b_parts < 1) || (b && !wa)) return WLLM_BAD_SIZE;
     if ((a_dtype != WLLM_BF16 && a_dtype != WLLM_F32) || (w_dtype != WLLM_BF16 && w_dtype != WLLM_F32) ||
@@ -423,7 +443,7 @@ WLLM_API int wllm_sandwich_norm_offset(float* resid, const void* a, int a_dtype,
     const bool multi = a_parts > 1 || (b && b_parts > 1);
 #define GO2(TO, M) wllm_launch(sandwich_norm_kernel<TO, M>, n, threads, smem, stream, resid, a, a_dtype, a_parts, (size_t)a_stride, wa, b, \
         b_dtype, b_parts, (size_t)b_stride, wb, inner_eps, factor, wp, center_p ? 1 : 0, eps_p, w, offset, center ? 1 : 0, eps, \
-        w_dtype, (TO*)out, rows, H, offset_p)
+        w_dtype, (TO*)out, rows, H, offset_p, bias)
 #define GO(TO) (multi ? GO2(TO, true) : GO2(TO, false))
     if (out_dtype == WLLM_BF16) return GO(bf16);
     if (out_dtype == WLLM_F32) return GO(float);
@@ -439,7 +459,7 @@ WLLM_API int wllm_sandwich_norm(float* resid, const void* a, int a_dtype, int a_
                                 cudaStream_t stream) {
     if (w == nullptr) return WLLM_BAD_SIZE;
     return wllm_sandwich_norm_offset(resid, a, a_dtype, a_parts, a_stride, wa, b, b_dtype, b_parts, b_stride, wb, inner_eps, factor,
-                                     wp, 0.f, center_p, eps_p, w, offset, center, eps, w_dtype, out, out_dtype, rows, n, H, stream);
+                                     wp, 0.f, center_p, eps_p, w, offset, center, eps, w_dtype, out, out_dtype, rows, n, H, nullptr, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------

@@ -20,7 +20,8 @@
 // With row gains (`wllm_rope_row_norm_kv_write`) the query row and the key row of a token are normed as wholes, all heads at
 // once, in front of the turn: q <- q / sqrt(mean(q^2) + eps) * wq over the token's nq * hd query elements, the same for k.
 // There the projections may have a bias (one 32-bit row for q | k | v, added to the finished sums, in front of the norms), and
-// the values may be blended with an earlier layer's values of the same token before they are cached.
+// the values may be blended with an earlier layer's values of the same token before they are cached.  `turn_scale` (here and in
+// `wllm_rope_kv_write_general`): sines and cosines are multiplied by it, so the turned part of a head is scaled and the rest is not.
 //
 // Page layout: [page][kv_head][slot_in_page][head_dim] (values: [..][vd]); `slots[n]` is page * page_size + slot_in_page.
 #include "common.cuh"
@@ -36,7 +37,7 @@ __global__ void rope_kv_write_kernel(const TI* __restrict__ qkv, int row_stride,
                                      TO* __restrict__ q_out, int q_stride, const int* __restrict__ positions,
                                      const int* __restrict__ slots, const float* __restrict__ inv_freq,
                                      TO* __restrict__ k_pages, TO* __restrict__ v_pages, int nq, int nkv, int hd,
-                                     int rot_dim, int page_size, int interleaved, int vd) {
+                                     int rot_dim, int page_size, int interleaved, int vd, float turn_scale) {
     pdl_launch_dependents();
     const int t = blockIdx.x;
     const int slot = slots ? slots[t] : -1;
@@ -45,6 +46,8 @@ __global__ void rope_kv_write_kernel(const TI* __restrict__ qkv, int row_stride,
     // the angle of this thread's first pair (all of them when the block is as wide as half the rotary size)
     float s0 = 0.f, c0 = 1.f;
     if ((int)threadIdx.x < half) sincosf(pos * inv_freq[threadIdx.x], &s0, &c0);
+    s0 *= turn_scale;
+    c0 *= turn_scale;
     pdl_wait();
     const int h_lo = ALL_HEADS ? 0 : blockIdx.y, h_hi = ALL_HEADS ? nq + 2 * nkv : blockIdx.y + 1;
     for (int h = h_lo; h < h_hi; ++h) {
@@ -78,7 +81,7 @@ __global__ void rope_kv_write_kernel(const TI* __restrict__ qkv, int row_stride,
         }
         for (int j = threadIdx.x; j < half; j += blockDim.x) {
             float sn = s0, cs = c0;
-            if (j != (int)threadIdx.x) sincosf(pos * inv_freq[j], &sn, &cs);
+            if (j != (int)threadIdx.x) { sincosf(pos * inv_freq[j], &sn, &cs); sn *= turn_scale; cs *= turn_scale; }
             const int ia = interleaved ? 2 * j : j, ib = interleaved ? 2 * j + 1 : j + half;
             const float x1 = in(ia), x2 = in(ib);
             float y1, y2;
@@ -353,14 +356,18 @@ __global__ void rope_kv_write_rows_kernel(const bf16* __restrict__ qkv, int row_
                                           const int* __restrict__ positions, const int* __restrict__ slots,
                                           const float* __restrict__ inv_freq, bf16* __restrict__ k_pages,
                                           bf16* __restrict__ v_pages, int nq, int nkv, int hd, int rot_dim, int page_size,
-                                          int interleaved) {
+                                          int interleaved, float turn_scale) {
     extern __shared__ float sc[];            // [half] sines, [half] cosines
     pdl_launch_dependents();
     const int t = blockIdx.x;
     const int slot = slots ? slots[t] : -1;
     const float pos = (float)positions[t];
     const int half = rot_dim >> 1;
-    for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf(pos * inv_freq[j], &sc[j], &sc[half + j]);
+    for (int j = threadIdx.x; j < half; j += blockDim.x) {
+        sincosf(pos * inv_freq[j], &sc[j], &sc[half + j]);
+        sc[j] *= turn_scale;
+        sc[half + j] *= turn_scale;
+    }
     __syncthreads();
     pdl_wait();
     const bf16* row = qkv + (size_t)t * row_stride;
@@ -439,7 +446,8 @@ rope_row_norm_kernel(const TI* __restrict__ qkv, int row_stride, int in_splits, 
                      TO* __restrict__ k_pages, TO* __restrict__ v_pages, int nq, int nkv, int hd,
                      int rot_dim, int page_size, int interleaved, int vd, const void* __restrict__ wq,
                      const void* __restrict__ wk, int w_dtype, int q_count, int k_count, float eps,
-                     const float* __restrict__ bias, float* __restrict__ v_first, const float* __restrict__ lam, int mix_mode) {
+                     const float* __restrict__ bias, float* __restrict__ v_first, const float* __restrict__ lam, int mix_mode,
+                     float turn_scale) {
     extern __shared__ float row[];            // [(nq + nkv) * hd] the token's q and k parts, [half] sines, [half] cosines
     __shared__ float scratch[32];
     pdl_launch_dependents();
@@ -449,7 +457,10 @@ rope_row_norm_kernel(const TI* __restrict__ qkv, int row_stride, int in_splits, 
     const int half = rot_dim >> 1, qw = nq * hd, kw = nkv * hd;
     float* sn = row + qw + kw;
     float* cs = sn + half;
-    for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf(pos * inv_freq[j], &sn[j], &cs[j]);
+    for (int j = threadIdx.x; j < half; j += blockDim.x) {
+        sincosf(pos * inv_freq[j], &sn[j], &cs[j]);
+        if (turn_scale != 1.0f) { sn[j] *= turn_scale; cs[j] *= turn_scale; }
+    }
     pdl_wait();
     const TI* x = qkv + (size_t)t * row_stride;
     auto sum_in = [&](int c) {     // part 0 + part 1 + ... in order; sixteen loads are in flight at a time
@@ -522,7 +533,7 @@ rope_row_norm_vec_kernel(const bf16* __restrict__ qkv, int row_stride, bf16* __r
                          bf16* __restrict__ k_pages, bf16* __restrict__ v_pages, int nq, int nkv, int hd, int rot_dim,
                          int page_size, int interleaved, int vd, const bf16* __restrict__ wq, const bf16* __restrict__ wk,
                          int q_count, int k_count, float eps, const float* __restrict__ bias, float* __restrict__ v_first,
-                         const float* __restrict__ lam, int mix_mode) {
+                         const float* __restrict__ lam, int mix_mode, float turn_scale) {
     extern __shared__ float row[];            // [(nq + nkv) * hd] the token's q and k parts, [half] sines, [half] cosines
     __shared__ float scratch[32];
     pdl_launch_dependents();
@@ -532,7 +543,10 @@ rope_row_norm_vec_kernel(const bf16* __restrict__ qkv, int row_stride, bf16* __r
     const int half = rot_dim >> 1, qw = nq * hd, kw = nkv * hd;
     float* sn = row + qw + kw;
     float* cs = sn + half;
-    for (int j = threadIdx.x; j < half; j += blockDim.x) sincosf(pos * inv_freq[j], &sn[j], &cs[j]);
+    for (int j = threadIdx.x; j < half; j += blockDim.x) {
+        sincosf(pos * inv_freq[j], &sn[j], &cs[j]);
+        if (turn_scale != 1.0f) { sn[j] *= turn_scale; cs[j] *= turn_scale; }
+    }
     pdl_wait();
     const bf16* x = qkv + (size_t)t * row_stride;
     float ssq = 0.f, ssk = 0.f;
@@ -615,7 +629,7 @@ WLLM_API int wllm_rope_row_norm_kv_write(const void* qkv, int in_dtype, int row_
                                          const float* inv_freq, void* k_pages, void* v_pages, int n, int nq, int nkv, int hd,
                                          int rot_dim, int page_size, int interleaved, int vd, const void* wq, const void* wk,
                                          int w_dtype, int q_count, int k_count, float eps, const float* bias, float* v_first,
-                                         const float* lam, int mix_mode, cudaStream_t stream) {
+                                         const float* lam, int mix_mode, float turn_scale, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
     if (mix_mode < 0 || mix_mode > 2 || (mix_mode > 0 && (v_first == nullptr || slots == nullptr)) || (mix_mode == 2 && lam == nullptr))
         return WLLM_BAD_SIZE;
@@ -635,7 +649,7 @@ WLLM_API int wllm_rope_row_norm_kv_write(const void* qkv, int in_dtype, int row_
         } \
         return wllm_launch(rope_row_norm_kernel<TI, TO>, n, 256, smem, stream, (const TI*)qkv, row_stride, in_splits, \
             (size_t)in_split_stride, (TO*)q_out, q_stride, positions, slots, inv_freq, (TO*)k_pages, (TO*)v_pages, nq, nkv, hd, \
-            rot_dim, page_size, interleaved, vd, wq, wk, w_dtype, q_count, k_count, eps, bias, v_first, lam, mix_mode); \
+            rot_dim, page_size, interleaved, vd, wq, wk, w_dtype, q_count, k_count, eps, bias, v_first, lam, mix_mode, turn_scale); \
     } while (0)
     const bool aligned = !(((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)wq | (uintptr_t)wk) & 15);
     if (in_dtype == WLLM_BF16 && out_dtype == WLLM_BF16 && w_dtype == WLLM_BF16 && in_splits == 1 && aligned && hd % 8 == 0 &&
@@ -648,7 +662,7 @@ WLLM_API int wllm_rope_row_norm_kv_write(const void* qkv, int in_dtype, int row_
         }
         return wllm_launch(rope_row_norm_vec_kernel, n, 256, smem, stream, (const bf16*)qkv, row_stride, (bf16*)q_out, q_stride,
                            positions, slots, inv_freq, (bf16*)k_pages, (bf16*)v_pages, nq, nkv, hd, rot_dim, page_size, interleaved,
-                           vd, (const bf16*)wq, (const bf16*)wk, q_count, k_count, eps, bias, v_first, lam, mix_mode);
+                           vd, (const bf16*)wq, (const bf16*)wk, q_count, k_count, eps, bias, v_first, lam, mix_mode, turn_scale);
     }
     if (in_dtype == WLLM_BF16 && out_dtype == WLLM_BF16) RN(bf16, bf16);
     if (in_dtype == WLLM_F32 && out_dtype == WLLM_BF16) RN(float, bf16);
@@ -706,7 +720,7 @@ WLLM_API int wllm_rope_kv_write_general(const void* qkv, int in_dtype, int row_s
                                         void* q_out, int out_dtype, int q_stride, const int* positions, const int* slots,
                                         const float* inv_freq, void* k_pages, void* v_pages, int n, int nq, int nkv, int hd,
                                         int rot_dim, int page_size, int interleaved, int vd, int unit_norm, float norm_eps,
-                                        cudaStream_t stream) {
+                                        float turn_scale, cudaStream_t stream) {
     if (n <= 0) return WLLM_OK;
     if (hd <= 0 || vd <= 0 || rot_dim < 0 || rot_dim > hd || (rot_dim & 1) || page_size <= 0 || nq <= 0 || nkv < 0 || (nkv == 0 && slots != nullptr) || in_splits < 1)
         return WLLM_BAD_SIZE;
@@ -715,7 +729,8 @@ WLLM_API int wllm_rope_kv_write_general(const void* qkv, int in_dtype, int row_s
         !((uintptr_t)k_pages & 15) && !((uintptr_t)v_pages & 15))
         return wllm_launch(rope_kv_write_rows_kernel, n, 128, (size_t)rot_dim * sizeof(float), stream, (const bf16*)qkv, row_stride,
                            (bf16*)q_out, q_stride, positions, slots, inv_freq, (bf16*)k_pages, (bf16*)v_pages, nq, nkv, hd,
-                           rot_dim, page_size, interleaved);
+                           rot_dim, page_size, interleaved, turn_scale);
+    if (unit_norm && turn_scale != 1.0f) return WLLM_BAD_SIZE;      // the head norms are built without a factor on the turn
     if (unit_norm)
         return launch_head_norm(qkv, in_dtype, row_stride, in_splits, in_split_stride, q_out, out_dtype, q_stride, positions, slots, inv_freq,
                                 k_pages, v_pages, n, nq, nkv, hd, rot_dim, page_size, interleaved, vd, norm_eps,
@@ -728,7 +743,7 @@ WLLM_API int wllm_rope_kv_write_general(const void* qkv, int in_dtype, int row_s
     const dim3 grid(n, all_heads ? 1 : nq + 2 * nkv);
 #define GO2(TI, TO, A) wllm_launch(rope_kv_write_kernel<TI, TO, A>, grid, threads, 0, stream, (const TI*)qkv, row_stride, in_splits, \
         (size_t)in_split_stride, (TO*)q_out, q_stride, positions, slots, inv_freq, (TO*)k_pages, (TO*)v_pages, nq, nkv, hd, \
-        rot_dim, page_size, interleaved, vd)
+        rot_dim, page_size, interleaved, vd, turn_scale)
 #define GO(TI, TO) (all_heads ? GO2(TI, TO, true) : GO2(TI, TO, false))
     if (in_dtype == WLLM_BF16 && out_dtype == WLLM_BF16) return GO(bf16, bf16);
     if (in_dtype == WLLM_F32 && out_dtype == WLLM_BF16) return GO(float, bf16);
@@ -744,5 +759,5 @@ WLLM_API int wllm_rope_kv_write(const void* qkv, int in_dtype, int row_stride, i
                                 int rot_dim, int page_size, int interleaved, cudaStream_t stream) {
     return wllm_rope_kv_write_general(qkv, in_dtype, row_stride, in_splits, in_split_stride, q_out, out_dtype, q_stride,
                                       positions, slots, inv_freq, k_pages, v_pages, n, nq, nkv, hd, rot_dim, page_size,
-                                      interleaved, hd, 0, 0.f, stream);
+                                      interleaved, hd, 0, 0.f, 1.0f, stream);
 }

@@ -278,7 +278,7 @@ class ModelRunner:
             all(len(e.tokens) == 1 and list(e.want) == [0] for e in entries)
 
     def _forward_graph(self, entries: list, device_tokens=None) -> torch.Tensor:
-        widest = max(1, max(len(t) for e in entries for t in e.cache.tables))
+        widest = max(1, max((len(t) for e in entries for t in e.cache.tables), default=1))
         width = 8
         while width < widest:
             width *= 2

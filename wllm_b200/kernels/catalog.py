@@ -14,6 +14,7 @@ FAMILIES = {
     "activation": [{}],
     "linear_attention": [{}],
     "delta_rule": [{}],
+    "state_space": [{}],
     "rg_lru": [{}],
     "token_blend": [{}],
     "latent_attention": [{}],

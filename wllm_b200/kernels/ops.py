@@ -177,9 +177,9 @@ def branch_norm(a, weight_a: torch.Tensor, out: torch.Tensor, eps: float, center
 
 def sandwich_norm(resid: torch.Tensor, a, out: torch.Tensor, post_weight: torch.Tensor, post_center: bool, post_eps: float,
                   weight, offset: float, center: bool, eps: float, rows=None, gain_a=None, b=None, gain_b=None,
-                  inner_eps: float = 0.0, factor: float = 1.0, post_offset: float = 0.0) -> torch.Tensor:
+                  inner_eps: float = 0.0, factor: float = 1.0, post_offset: float = 0.0, bias=None) -> torch.Tensor:
     """One kernel for a block that norms behind its sublayers too (csrc/norm.cu):
-        u = a, or factor * (rms(a) * gain_a + rms(b) * gain_b) when gain_a is given;
+        u = a [+ bias], or factor * (rms(a) * gain_a + rms(b) * gain_b) when gain_a is given;
         resid += norm(u) * (post_offset + post_weight)  (post_center: with the mean taken off);
         out = norm(resid) * (offset + weight), or, with `weight` None, resid as it is (rounded to out's type).
     `a`, `b`: (tensor [n, H] or float32 partial sums [S, n, H], S or 0).  With `rows` the residual is read at those rows
@@ -190,6 +190,7 @@ def sandwich_norm(resid: torch.Tensor, a, out: torch.Tensor, post_weight: torch.
     assert resid.dtype == torch.float32 and resid.is_contiguous() and out.is_contiguous() and out.shape == (n, H)
     gains = [g for g in (post_weight, weight, gain_a, gain_b) if g is not None]
     assert all(g.shape == (H,) and g.is_contiguous() and g.dtype == post_weight.dtype for g in gains)
+    assert bias is None or (bias.dtype == torch.float32 and bias.shape == (H,) and bias.is_contiguous())
     pa = _branch_args(a, N, H)
     pb = _branch_args(b, N, H) if b is not None else (_ptr(None), _F32, 1, ctypes.c_longlong(0))
     lib = load_family("norm")
@@ -197,7 +198,17 @@ def sandwich_norm(resid: torch.Tensor, a, out: torch.Tensor, post_weight: torch.
                                          _ptr(post_weight), c_float(post_offset), 1 if post_center else 0, c_float(post_eps),
                                          _ptr(weight), c_float(offset), 1 if center else 0, c_float(eps), _dt(post_weight),
                                          _ptr(out), _dt(out), _ptr(_int32(rows, "rows") if rows is not None else None), n, H,
-                                         _stream()), "sandwich_norm")
+                                         _ptr(bias), _stream()), "sandwich_norm")
+    return out
+
+
+def branch_bias(a, bias: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out[n, H] (float32) = a + bias[H] (float32), a being a branch output: (tensor [n, H] or float32 partial sums [S, n, H], S or 0)."""
+    n, H = out.shape
+    _need_cuda(a[0], bias, out)
+    assert out.dtype == torch.float32 and out.is_contiguous() and bias.dtype == torch.float32 and bias.shape == (H,) and bias.is_contiguous()
+    lib = load_family("norm")
+    _check(lib.wllm_branch_bias(*_branch_args(a, n, H), _ptr(bias), _ptr(out), n, H, _stream()), "branch_bias")
     return out
 
 
@@ -255,13 +266,14 @@ def hyper_norm(src: torch.Tensor, dst: torch.Tensor, S: int, branch, prev_mix, p
 
 def rope_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, positions: torch.Tensor, slots, inv_freq: torch.Tensor,
                   k_pages, v_pages, nq: int, nkv: int, hd: int, rot_dim: int, page_size: int, in_splits: int = 0,
-                  pairing: str = "half", vd: int | None = None, unit_norm_eps: float | None = None) -> None:
+                  pairing: str = "half", vd: int | None = None, unit_norm_eps: float | None = None,
+                  turn_scale: float = 1.0) -> None:
     """Rotate the q and k heads of the fused rows `qkv` [n, (nq+2nkv)*hd] (or [S, n, ...] float32 partial sums
     when in_splits = S > 0); rotated q goes to `q_out` [n, nq*hd], rotated k and v to the pages.
     pairing 'half': element j turns with j + rot_dim/2; 'interleaved': 2j with 2j + 1.
     `vd`: size of a value head when it is not hd (the row is then nq*hd | nkv*hd | nkv*vd, and may be the first
     columns of a wider fused row).  `unit_norm_eps`: every rotated q and k head is divided by its root mean
-    square, y / sqrt(mean(y^2) + eps)."""
+    square, y / sqrt(mean(y^2) + eps).  `turn_scale` multiplies the sines and cosines (not with unit_norm_eps)."""
     if pairing not in ("half", "interleaved"):
         raise KernelError(f"rotary pairing {pairing!r} not supported (half, interleaved)")
     _need_cuda(qkv, q_out, positions, slots, inv_freq, k_pages, v_pages)
@@ -284,21 +296,23 @@ def rope_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, positions: torch.Tenso
                                           _ptr(_int32(slots, "slots") if slots is not None else None), _ptr(inv_freq),
                                           _ptr(k_pages), _ptr(v_pages), n, nq, nkv, hd, rot_dim, page_size,
                                           1 if pairing == "interleaved" else 0, vd, 0 if unit_norm_eps is None else 1,
-                                          c_float(unit_norm_eps or 0.0), _stream()),
+                                          c_float(unit_norm_eps or 0.0), c_float(turn_scale), _stream()),
            "rope_kv_write")
 
 
 def rope_row_norm_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, positions: torch.Tensor, slots, inv_freq: torch.Tensor,
                            k_pages, v_pages, nq: int, nkv: int, hd: int, rot_dim: int, page_size: int, q_gain: torch.Tensor,
-                           k_gain: torch.Tensor, eps: float, q_count: int, k_count: int, in_splits: int = 0,
+                           k_gain: torch.Tensor | None, eps: float, q_count: int, k_count: int, in_splits: int = 0,
                            pairing: str = "half", vd: int | None = None, bias: torch.Tensor | None = None,
-                           v_first: torch.Tensor | None = None, blend: torch.Tensor | None = None, mix: str | None = None) -> None:
+                           v_first: torch.Tensor | None = None, blend: torch.Tensor | None = None, mix: str | None = None,
+                           turn_scale: float = 1.0) -> None:
     """As rope_kv_write, with the token's query row and key row normed as wholes (all heads at once) in front of the
     turn: q <- q / sqrt(mean(q^2) + eps) * q_gain over the nq * hd query elements, the same for k with k_gain
     (csrc/rope_cache.cu).  `q_count`, `k_count`: the elements that count for the means (heads held in steps of 8
     elements carry zeros behind them).  `bias`: one float32 row [(nq + nkv) * hd + nkv * vd] added to the projections' sums
     in front of the norms.  `mix` 'first': the token's values are also left in `v_first` [n, nkv * vd] float32; 'later': the
-    values that are cached are (1 - blend[0]) v + blend[0] v_first."""
+    values that are cached are (1 - blend[0]) v + blend[0] v_first.  nkv = 0 (k_gain None, no slots): a row of query heads
+    alone.  `turn_scale` multiplies the sines and cosines."""
     if pairing not in ("half", "interleaved"):
         raise KernelError(f"rotary pairing {pairing!r} not supported (half, interleaved)")
     _need_cuda(qkv, q_out, positions, slots, inv_freq, k_pages, v_pages, q_gain, k_gain)
@@ -307,8 +321,8 @@ def rope_row_norm_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, positions: to
     ptr, dt, row_stride, nparts, part_stride, n = _fused_args(qkv, in_splits)
     assert qkv.shape[-1] >= width and q_out.shape == (n, nq * hd) and q_out.stride(1) == 1
     assert inv_freq.dtype == torch.float32 and inv_freq.numel() == rot_dim // 2 and inv_freq.is_contiguous()
-    assert q_gain.shape == (nq * hd,) and k_gain.shape == (nkv * hd,) and q_gain.dtype == k_gain.dtype
-    assert q_gain.is_contiguous() and k_gain.is_contiguous()
+    assert q_gain.shape == (nq * hd,) and q_gain.is_contiguous() and (nkv > 0 or slots is None)
+    assert (nkv == 0 and k_gain is None) or (k_gain.shape == (nkv * hd,) and k_gain.dtype == q_gain.dtype and k_gain.is_contiguous())
     if slots is not None:
         assert k_pages.is_contiguous() and v_pages.is_contiguous() and k_pages.dtype == q_out.dtype == v_pages.dtype
     if mix not in (None, "first", "later"):
@@ -326,7 +340,7 @@ def rope_row_norm_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, positions: to
                                            1 if pairing == "interleaved" else 0, vd, _ptr(q_gain), _ptr(k_gain), _dt(q_gain),
                                            q_count, k_count, c_float(eps), _ptr(bias), _ptr(v_first if mix is not None else None),
                                            _ptr(blend if mix == "later" else None), {None: 0, "first": 1, "later": 2}[mix],
-                                           _stream()), "rope_row_norm_kv_write")
+                                           c_float(turn_scale), _stream()), "rope_row_norm_kv_write")
 
 
 def rope_head_norm_kv_write(qkv: torch.Tensor, q_out: torch.Tensor, positions: torch.Tensor, slots, inv_freq: torch.Tensor,
@@ -757,17 +771,17 @@ def unit_act(x: torch.Tensor, out: torch.Tensor, act: str) -> torch.Tensor:
     return out
 
 
-def sigmoid_gate(x: torch.Tensor, fused: torch.Tensor, parts: int, col0: int) -> torch.Tensor:
-    """x[n, c] *= sigmoid(gate[n, c]) in place, the gate being columns col0 .. col0 + x.shape[1] of the fused projection
-    `fused` [n, W] (or float32 partial sums [parts, n, W], added in order)."""
+def sigmoid_gate(x: torch.Tensor, fused: torch.Tensor, parts: int, col0: int, per: int = 1) -> torch.Tensor:
+    """x[n, c] *= sigmoid(gate[n, c // per]) in place, the gate being columns col0 .. col0 + x.shape[1] // per of the fused
+    projection `fused` [n, W] (or float32 partial sums [parts, n, W], added in order); per = the head size: one number per head."""
     _need_cuda(x, fused)
     n, width = x.shape
     ptr, dt, row_stride, nparts, part_stride, rows = _fused_args(fused, parts)
-    assert rows == n and x.stride(1) == 1 and col0 + width <= fused.shape[-1]
+    assert rows == n and x.stride(1) == 1 and width % per == 0 and col0 + width // per <= fused.shape[-1]
     lib = load_family("activation")
     item = 4 if fused.dtype == torch.float32 else 2
     _check(lib.wllm_sigmoid_gate(_ptr(x), _dt(x), x.stride(0), c_void_p(fused.data_ptr() + col0 * item), dt, row_stride, nparts,
-                                 part_stride, n, width, _stream()), "sigmoid_gate")
+                                 part_stride, n, width, per, _stream()), "sigmoid_gate")
     return x
 
 
@@ -1069,6 +1083,25 @@ def linattn_prepare(fused, parts: int, q_off: int, k_off: int, v_off: int, heads
                                     c_float(tau), _ptr(q), _ptr(k), _ptr(v), _ptr(decay), _stream()), "linattn_prepare")
 
 
+def lowrank_map(low: torch.Tensor, parts: int, low_off: int, w2: torch.Tensor, heads: int, dim: int, out: torch.Tensor,
+                bias: torch.Tensor | None = None, decay_log: torch.Tensor | None = None) -> torch.Tensor:
+    """z = w2 @ low [+ bias] (csrc/linear_attention.cu, forms 2 and 3), out [n, heads*dim] float32, where `low` are the rank =
+    w2.shape[1] columns of the projection `low` [n, W] (or partial sums [parts, n, W]) from `low_off`; with `decay_log` [heads] the
+    map becomes a decay per key channel, minus one: expm1(-exp(decay_log_h) softplus(z))."""
+    _need_cuda(low, w2, bias, decay_log, out)
+    ptr, dt, row_stride, nparts, part_stride, n = _fused_args(low, parts)
+    assert w2.shape[0] == heads * dim and w2.is_contiguous() and low_off + w2.shape[1] <= low.shape[-1]
+    assert bias is None or (bias.shape == (heads * dim,) and bias.dtype == w2.dtype and bias.is_contiguous())
+    assert decay_log is None or (decay_log.shape == (heads,) and decay_log.dtype == w2.dtype and decay_log.is_contiguous())
+    assert out.dtype == torch.float32 and out.is_contiguous() and out.shape == (n, heads * dim)
+    lib = load_family("linear_attention")
+    null = _ptr(None)
+    _check(lib.wllm_linattn_prepare_form(ptr, dt, row_stride, nparts, part_stride, 0, 0, 0, low_off, n, heads, dim, dim, w2.shape[1], null,
+                                         null, 0, c_float(1.0), c_float(1.0), _ptr(w2), _ptr(bias), _dt(w2), c_float(1.0), null, null, null,
+                                         _ptr(out), 3 if decay_log is None else 2, _ptr(decay_log), _stream()), "lowrank_map")
+    return out
+
+
 def linattn_decay(low: torch.Tensor, parts: int, low_off: int, w2: torch.Tensor, b2: torch.Tensor, heads: int, dim: int,
                   decay: torch.Tensor) -> torch.Tensor:
     """The decay per key channel of time mixing, minus one: decay [n, heads*dim] = expm1(-exp(w2 @ tanh(low) + b2)), where `low` are the
@@ -1082,7 +1115,7 @@ def linattn_decay(low: torch.Tensor, parts: int, low_off: int, w2: torch.Tensor,
     null = _ptr(None)
     _check(lib.wllm_linattn_prepare_form(ptr, dt, row_stride, nparts, part_stride, 0, 0, 0, low_off, n, heads, dim, dim, w2.shape[1], null,
                                          null, 0, c_float(1.0), c_float(1.0), _ptr(w2), _ptr(b2), _dt(w2), c_float(1.0), null, null, null,
-                                         _ptr(decay), 1, _stream()), "linattn_decay")
+                                         _ptr(decay), 1, null, _stream()), "linattn_decay")
     return decay
 
 
@@ -1110,14 +1143,17 @@ def linattn_segment_plan(max_q_len: int, requests_multi: int, heads: int, vdim: 
 def linattn_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay, head_decay, state: torch.Tensor,
                  out: torch.Tensor, req_q_start: torch.Tensor, req_q_len: torch.Tensor, req_slot: torch.Tensor, heads: int,
                  dim: int, vdim: int, seg_len: int = 0, max_seg: int = 1, seg_state: torch.Tensor | None = None,
-                 seg_decay: torch.Tensor | None = None, bonus: torch.Tensor | None = None) -> torch.Tensor:
+                 seg_decay: torch.Tensor | None = None, bonus: torch.Tensor | None = None, pairs: torch.Tensor | None = None,
+                 share: int = 1) -> torch.Tensor:
     """S <- diag(a_t) S + k_t v_t^T, o_t = S^T q_t over every request's tokens of the step, from and to the
     request's row of `state` [slots, heads, dim, vdim] (float32).  `decay` [n, heads*dim] per key channel, or None
     with `head_decay` [heads].  With seg_len > 0 and max_seg > 1 (linattn_segment_plan) portions are cut into segments
     of seg_len tokens that run side by side; seg_state (requests * max_seg * heads * dim * vdim floats) and seg_decay
     (requests * max_seg * heads * dim) are their scratch.  q, k and v may be columns of wider rows.  `bonus` [heads*dim]
-    (time mixing): o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t, the output in front of the update; `decay` then holds a - 1."""
-    _need_cuda(bonus, q, k, v, decay, head_decay, state, out, req_q_start, req_q_len, req_slot, seg_state, seg_decay)
+    (time mixing): o_t = (S_(t-1) + diag(bonus) k_t v_t^T)^T q_t, the output in front of the update; `decay` then holds a - 1.
+    `pairs` [n, heads, 2] (a state space; decay and head_decay None): (a - 1, step) per head and token, S <- a S + k (step v)^T.
+    `share`: neighbouring heads that read the same head of q and k, whose rows then hold heads / share heads."""
+    _need_cuda(pairs, bonus, q, k, v, decay, head_decay, state, out, req_q_start, req_q_len, req_slot, seg_state, seg_decay)
     R = req_q_len.shape[0]
     if seg_len > 0 and max_seg > 1:
         assert seg_state.dtype == seg_decay.dtype == torch.float32 and seg_state.is_contiguous() and seg_decay.is_contiguous()
@@ -1127,68 +1163,80 @@ def linattn_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay, head_
     n = q.shape[0]
     assert all(t.dtype == torch.float32 for t in (q, k, v, state, out)) and all(t.stride(1) == 1 for t in (q, k, v))
     assert state.is_contiguous() and out.is_contiguous()
-    assert q.shape == k.shape == (n, heads * dim) and v.shape == out.shape == (n, heads * vdim)
+    assert heads % share == 0 and q.shape == k.shape == (n, heads // share * dim) and v.shape == out.shape == (n, heads * vdim)
     assert state.shape[1:] == (heads, dim, vdim)
     assert bonus is None or (decay is not None and bonus.dtype == torch.float32 and bonus.shape == (heads * dim,) and bonus.is_contiguous())
-    if decay is not None:
-        assert decay.dtype == torch.float32 and decay.is_contiguous() and decay.shape == q.shape
+    if pairs is not None:
+        assert decay is None and head_decay is None and bonus is None
+        assert pairs.dtype == torch.float32 and pairs.is_contiguous() and pairs.shape == (n, heads, 2)
+    elif decay is not None:
+        assert decay.dtype == torch.float32 and decay.is_contiguous() and decay.shape == (n, heads * dim)
     else:
         assert head_decay.dtype == torch.float32 and head_decay.shape == (heads,) and head_decay.is_contiguous()
     lib = load_family("linear_attention")
     def stride(t, width):
         return ctypes.c_longlong(t.stride(0) if n > 1 else max(t.stride(0), width))
-    _check(lib.wllm_linattn_scan_rows(_ptr(q), _ptr(k), _ptr(v), stride(q, heads * dim), stride(k, heads * dim), stride(v, heads * vdim),
-                                 _ptr(decay), _ptr(head_decay), _ptr(bonus), _ptr(state), _ptr(out),
-                                 _ptr(_int32(req_q_start, "req_q_start")), _ptr(_int32(req_q_len, "req_q_len")),
-                                 _ptr(_int32(req_slot, "req_slot")), R, heads, dim, vdim, seg_len, max_seg,
-                                 _ptr(seg_state), _ptr(seg_decay), _stream()),
+    qk = heads // share * dim
+    _check(lib.wllm_linattn_scan_shared(_ptr(q), _ptr(k), _ptr(v), stride(q, qk), stride(k, qk), stride(v, heads * vdim),
+                                        _ptr(decay if pairs is None else pairs), 0 if pairs is None else 1, _ptr(head_decay), _ptr(bonus),
+                                        _ptr(state), _ptr(out), _ptr(_int32(req_q_start, "req_q_start")),
+                                        _ptr(_int32(req_q_len, "req_q_len")), _ptr(_int32(req_slot, "req_slot")), R, heads, share, dim,
+                                        vdim, seg_len, max_seg, _ptr(seg_state), _ptr(seg_decay), _stream()),
            f"linattn_scan(heads={heads}, dim={dim}, vdim={vdim})")
     return out
 
 
 def head_gate_norm(o: torch.Tensor, fused, parts: int, gate_off: int, weight, eps: float, out: torch.Tensor, heads: int,
-                   vdim: int, factor: float = 1.0) -> torch.Tensor:
-    """out[n, heads*vdim] = o / sqrt(mean over a head of o^2 + eps) [* weight] * silu(gate) * factor, the gate being the
-    columns of the fused projection row from `gate_off`; 32-bit inside, rounded once to out's element type.  weight [vdim] is
+                   vdim: int, factor: float = 1.0, gate_act: str = "silu") -> torch.Tensor:
+    """out[n, heads*vdim] = o / sqrt(mean over a head of o^2 + eps) [* weight] * act(gate) * factor (`gate_act` 'silu' or 'sigmoid'), the gate
+    being the columns of the fused projection row from `gate_off`; 32-bit inside, rounded once to out's element type.  weight [vdim] is
     shared by the heads, weight [heads*vdim] a gain of the whole row; `out` may be columns of wider rows."""
     _need_cuda(o, fused, weight, out)
     ptr, dt, row_stride, nparts, part_stride, n = _fused_args(fused, parts)
     assert o.dtype == torch.float32 and o.is_contiguous() and o.shape == (n, heads * vdim) == out.shape and out.stride(1) == 1
     assert weight is None or (weight.shape in ((vdim,), (heads * vdim,)) and weight.is_contiguous())
+    if gate_act not in ("silu", "sigmoid"):
+        raise KernelError(f"head gate {gate_act!r}: 'silu' or 'sigmoid'")
     whole_row = weight is not None and weight.shape[0] == heads * vdim
     lib = load_family("linear_attention")
     _check(lib.wllm_head_gate_norm_rows(_ptr(o), ptr, dt, row_stride, nparts, part_stride, gate_off, _ptr(weight),
                                         _dt(weight) if weight is not None else _F32, 1 if whole_row else 0, c_float(eps), _ptr(out),
-                                        _dt(out), max(out.stride(0), heads * vdim), c_float(factor), n, heads, vdim, _stream()),
+                                        _dt(out), max(out.stride(0), heads * vdim), c_float(factor), 1 if gate_act == "sigmoid" else 0,
+                                        n, heads, vdim, _stream()),
            "head_gate_norm")
     return out
 
 
 def delta_prepare(fused, parts: int, offsets: dict, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, conv_q, conv_k,
                   conv_v, a_log, dt_bias, token_req, req_q_start, req_slot, conv_state, unit_eps: float, q_scale: float, q, k, v,
-                  beta, decay) -> None:
+                  beta, decay, shift: torch.Tensor | None = None) -> None:
     """What enters the gated delta rule, from the fused projection [n, W] (or float32 partial sums [parts, n, W]) whose columns
     `offsets` names (q, k, v, b, a): q, k [n, kv_heads, dim] and v [n, heads, vdim] through their short convolutions (taps
     [channels, taps], the last tap the token's own; the inputs before a portion's start come from `conv_state`
     [slots, taps - 1, channels]) and SiLU, q and k divided by sqrt(sum(x^2) + unit_eps) per head (q also times q_scale),
-    beta = sigmoid(b) and decay = exp(-exp(a_log) softplus(a + dt_bias)) [n, heads]; all 32-bit (csrc/delta_rule.cu)."""
-    _need_cuda(fused, conv_q, conv_k, conv_v, a_log, dt_bias, token_req, req_q_start, req_slot, conv_state, q, k, v, beta, decay)
+    beta = sigmoid(b) and decay = exp(-exp(a_log) softplus(a + dt_bias)) [n, heads]; all 32-bit (csrc/delta_rule.cu).  Without
+    offsets["a"] (a_log, dt_bias, decay None) the decays come from elsewhere.  `shift` (the requests' lengths; every request of the
+    step brings at most one token): conv_state is brought up to date too, delta_conv_update has nothing left to do."""
+    _need_cuda(shift,fused, conv_q, conv_k, conv_v, a_log, dt_bias, token_req, req_q_start, req_slot, conv_state, q, k, v, beta, decay)
     ptr, dt, row_stride, nparts, part_stride, n = _fused_args(fused, parts)
     C = 2 * kv_heads * dim + heads * vdim
     assert conv_q.shape == conv_k.shape == (kv_heads * dim, taps) and conv_v.shape == (heads * vdim, taps)
-    assert conv_q.dtype == conv_k.dtype == conv_v.dtype == a_log.dtype == dt_bias.dtype
-    assert all(t.is_contiguous() for t in (conv_q, conv_k, conv_v, a_log, dt_bias, q, k, v, beta, decay))
-    assert a_log.shape == dt_bias.shape == (heads,)
-    assert q.shape == k.shape == (n, kv_heads * dim) and v.shape == (n, heads * vdim) and beta.shape == decay.shape == (n, heads)
-    assert all(t.dtype == torch.float32 for t in (q, k, v, beta, decay))
+    per_head = "a" in offsets
+    own = (a_log, dt_bias, decay) if per_head else ()
+    assert conv_q.dtype == conv_k.dtype == conv_v.dtype and (not per_head or a_log.dtype == dt_bias.dtype == conv_q.dtype)
+    assert all(t.is_contiguous() for t in (conv_q, conv_k, conv_v, q, k, v, beta) + own)
+    assert not per_head or (a_log.shape == dt_bias.shape == (heads,) and decay.shape == (n, heads) and decay.dtype == torch.float32)
+    assert q.shape == k.shape == (n, kv_heads * dim) and v.shape == (n, heads * vdim) and beta.shape == (n, heads)
+    assert all(t.dtype == torch.float32 for t in (q, k, v, beta))
     assert taps == 1 or (conv_state.dtype == torch.float32 and conv_state.is_contiguous() and conv_state.shape[1:] == (taps - 1, C))
     lib = load_family("delta_rule")
     _check(lib.wllm_delta_prepare(ptr, dt, row_stride, nparts, part_stride, offsets["q"], offsets["k"], offsets["v"], offsets["b"],
-                                  offsets["a"], n, heads, kv_heads, dim, vdim, taps, _ptr(conv_q), _ptr(conv_k), _ptr(conv_v),
+                                  offsets.get("a", -1), n, heads, kv_heads, dim, vdim, taps, _ptr(conv_q), _ptr(conv_k), _ptr(conv_v),
                                   _ptr(a_log), _ptr(dt_bias), _dt(conv_q), _ptr(_int32(token_req, "token_req")),
-                                  _ptr(_int32(req_q_start, "req_q_start")), _ptr(_int32(req_slot, "req_slot")),
-                                  _ptr(conv_state if taps > 1 else None), c_float(unit_eps), c_float(q_scale), _ptr(q), _ptr(k), _ptr(v),
-                                  _ptr(beta), _ptr(decay), _stream()), "delta_prepare")
+                                  _ptr(_int32(req_q_start, "req_q_start")), _ptr(_int32(shift, "lengths") if shift is not None else None),
+                                  _ptr(_int32(req_slot, "req_slot")), _ptr(conv_state if taps > 1 else None), c_float(unit_eps),
+                                  c_float(q_scale), _ptr(q), _ptr(k), _ptr(v), _ptr(beta), _ptr(decay),
+                                  1 if shift is not None and taps > 1 else 0, _stream()), "delta_prepare")
 
 
 def delta_conv_update(fused, parts: int, offsets: dict, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, req_q_start,
@@ -1206,27 +1254,89 @@ def delta_conv_update(fused, parts: int, offsets: dict, heads: int, kv_heads: in
                                       _ptr(conv_state), _stream()), "delta_conv_update")
 
 
-def delta_scan(q, k, v, beta, decay, state, out, req_q_start, req_q_len, req_slot, heads: int, kv_heads: int, dim: int, vdim: int):
+def delta_scan(q, k, v, beta, decay, state, out, req_q_start, req_q_len, req_slot, heads: int, kv_heads: int, dim: int, vdim: int,
+               channel: bool = False):
     """The gated delta rule over every request's tokens of the step, in order, from and to its state slot:
     S <- decay S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q.  q, k [n, kv_heads * dim], v, out [n, heads * vdim],
-    beta, decay [n, heads], state [slots, heads, dim, vdim], all float32 (csrc/delta_rule.cu)."""
+    beta, decay [n, heads], state [slots, heads, dim, vdim], all float32 (csrc/delta_rule.cu).  `channel`: decay
+    [n, heads * dim], one per key channel, given as decay - 1 (lowrank_map)."""
     _need_cuda(q, k, v, beta, decay, state, out, req_q_start, req_q_len, req_slot)
     n = q.shape[0]
     assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (q, k, v, beta, decay, state, out))
-    assert q.shape == k.shape == (n, kv_heads * dim) and v.shape == out.shape == (n, heads * vdim) and beta.shape == decay.shape == (n, heads)
+    assert q.shape == k.shape == (n, kv_heads * dim) and v.shape == out.shape == (n, heads * vdim) and beta.shape == (n, heads)
+    assert decay.shape == (n, heads * dim if channel else heads)
     assert state.shape[1:] == (heads, dim, vdim)
     lib = load_family("delta_rule")
-    _check(lib.wllm_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(beta), _ptr(decay), _ptr(state), _ptr(out),
+    _check(lib.wllm_delta_scan(_ptr(q), _ptr(k), _ptr(v), _ptr(beta), _ptr(decay), 1 if channel else 0, _ptr(state), _ptr(out),
                                _ptr(_int32(req_q_start, "req_q_start")), _ptr(_int32(req_q_len, "req_q_len")),
                                _ptr(_int32(req_slot, "req_slot")), req_q_len.shape[0], heads, kv_heads, dim, vdim, _stream()),
            f"delta_scan(heads={heads}/{kv_heads}, dim={dim}/{vdim})")
     return out
 
 
+def ssd_prepare(fused, parts: int, x_off: int, dt_off: int, taps: int, conv: torch.Tensor, conv_bias, a_log: torch.Tensor,
+                dt_bias: torch.Tensor, ctx, conv_state, out: torch.Tensor, pairs: torch.Tensor, shift: bool = False) -> None:
+    """What enters a state space (csrc/state_space.cu) from the fused projection [n, W] (or float32 partial sums [parts, n, W]): the
+    columns from `x_off` through their causal convolution (conv [C, taps], the last tap the token's own; conv_bias [C] or None; the inputs in
+    front of a portion come from `conv_state` [slots, taps - 1, C]) and SiLU into out [n, C]; the columns dt_off .. + heads become
+    pairs [n, heads, 2] = (a - 1, dt), dt = softplus(. + dt_bias), a = exp(-exp(a_log) dt).  `shift` (every request of the step brings at
+    most one token): conv_state is brought up to date too."""
+    _need_cuda(fused, conv, conv_bias, a_log, dt_bias, conv_state, out, pairs)
+    ptr, dt, row_stride, nparts, part_stride, n = _fused_args(fused, parts)
+    C, H = conv.shape[0], a_log.shape[0]
+    assert conv.shape == (C, taps) and a_log.shape == dt_bias.shape == (H,) and conv.dtype == a_log.dtype == dt_bias.dtype
+    assert conv_bias is None or (conv_bias.shape == (C,) and conv_bias.dtype == conv.dtype and conv_bias.is_contiguous())
+    assert out.shape == (n, C) and pairs.shape == (n, H, 2) and out.dtype == pairs.dtype == torch.float32
+    assert all(t.is_contiguous() for t in (conv, a_log, dt_bias, out, pairs))
+    assert x_off + C <= fused.shape[-1] and dt_off + H <= fused.shape[-1]
+    assert taps == 1 or (conv_state.dtype == torch.float32 and conv_state.is_contiguous() and conv_state.shape[1:] == (taps - 1, C))
+    lib = load_family("state_space")
+    _check(lib.wllm_ssd_prepare(ptr, dt, row_stride, nparts, part_stride, x_off, dt_off, n, C, H, taps, _ptr(conv), _ptr(conv_bias),
+                                _ptr(a_log), _ptr(dt_bias), _dt(conv), _ptr(_int32(ctx.token_req, "token_req")),
+                                _ptr(_int32(ctx.req_q_start, "req_q_start")), _ptr(_int32(ctx.req_q_len, "req_q_len")),
+                                _ptr(_int32(ctx.req_slot, "req_slot")), _ptr(conv_state if taps > 1 else None), _ptr(out), _ptr(pairs),
+                                1 if shift and taps > 1 else 0, _stream()), "ssd_prepare")
+
+
+def ssd_conv_update(fused, parts: int, x_off: int, taps: int, ctx, conv_state: torch.Tensor) -> None:
+    """The newest taps - 1 inputs of the convolution, per request, after a step with portions (see ssd_prepare)."""
+    _need_cuda(fused, conv_state)
+    ptr, dt, row_stride, nparts, part_stride, _ = _fused_args(fused, parts)
+    lib = load_family("state_space")
+    _check(lib.wllm_ssd_conv_update(ptr, dt, row_stride, nparts, part_stride, x_off, conv_state.shape[2], taps,
+                                    _ptr(_int32(ctx.req_q_start, "req_q_start")), _ptr(_int32(ctx.req_q_len, "req_q_len")),
+                                    _ptr(_int32(ctx.req_slot, "req_slot")), ctx.req_q_len.shape[0], _ptr(conv_state), _stream()),
+           "ssd_conv_update")
+
+
+def ssd_gate_norm(o: torch.Tensor, x: torch.Tensor, skip: torch.Tensor, fused, parts: int, z_off: int, weight: torch.Tensor, eps: float,
+                  out: torch.Tensor, groups: int) -> torch.Tensor:
+    """out [n, inner] = y / sqrt(mean over a part of y^2 + eps) * weight, the row being `groups` equal parts, y = (o + skip_h x) silu(z): o, x
+    [n, inner] float32 (x may be columns of wider rows), skip [heads], z the columns of `fused` from z_off; 32-bit inside, rounded once."""
+    _need_cuda(o, x, skip, fused, weight, out)
+    ptr, dt, row_stride, nparts, part_stride, n = _fused_args(fused, parts)
+    inner, H = o.shape[1], skip.shape[0]
+    assert o.dtype == x.dtype == torch.float32 and o.is_contiguous() and x.shape == o.shape == out.shape == (n, inner) and x.stride(1) == 1
+    assert skip.dtype == weight.dtype and weight.shape == (inner,) and weight.is_contiguous() and skip.is_contiguous() and inner % H == 0
+    assert out.is_contiguous() and z_off + inner <= fused.shape[-1]
+    lib = load_family("state_space")
+    _check(lib.wllm_ssd_gate_norm(_ptr(o), _ptr(x), ctypes.c_longlong(max(x.stride(0), inner)), _ptr(skip), ptr, dt, row_stride, nparts,
+                                  part_stride, z_off, _ptr(weight), _dt(weight), c_float(eps), _ptr(out), _dt(out), n, inner, inner // H,
+                                  groups, _stream()), "ssd_gate_norm")
+    return out
+
+
+ROUTER_SCORES = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
+# the experts' gated units: 'capped_swish' (with its limit and slope) and 'silu', its plain form: g sigmoid(g) u
+EXPERT_GATED_UNITS = ("capped_swish", "silu")
+
+
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, w_gate, chosen: torch.Tensor, weights: torch.Tensor, gate_out,
               groups: int = 1, groups_kept: int = 1, scores: str = "softmax", correction: torch.Tensor | None = None,
-              renorm_eps: float | None = None) -> None:
-    """The router of routed experts (csrc/moe.cu): scores = softmax(w_router x) in 32-bit over all E experts (`scores`
+              renorm_eps: float | None = None, bias: torch.Tensor | None = None) -> None:
+    """The router of routed experts (csrc/moe.cu): scores = softmax(w_router x + bias) in 32-bit over all E experts (`bias` [E]
+    float32, None: none; `scores` 'softmax_chosen': the `top` largest logits are chosen, their weights are the softmax over the
+    chosen logits alone, without groups and corrections; `scores`
     'sigmoid': sigmoid(w_router x) expert by expert, not normalised; without groups the choice is made on the logits, whose order
     the sigmoid keeps, so that large logits that all round to a score of 1 do not tie), the choice
     limited to the `groups_kept` best of `groups` groups of neighbouring experts; chosen [n, top] (descending score) and
@@ -1242,12 +1352,14 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, w_gate, chosen: torch.Ten
         assert w_gate.dtype == torch.float32 and w_gate.shape == (H,) and w_gate.is_contiguous()
         assert gate_out.dtype == torch.float32 and gate_out.shape == (n,) and gate_out.is_contiguous()
     assert correction is None or (correction.dtype == torch.float32 and correction.shape == (E,) and correction.is_contiguous())
-    if scores not in ("softmax", "sigmoid"):
-        raise KernelError(f"router scores {scores!r}: 'softmax' or 'sigmoid'")
+    if scores not in ROUTER_SCORES:
+        raise KernelError(f"router scores {scores!r}: one of {', '.join(ROUTER_SCORES)}")
+    _need_cuda(bias)
+    assert bias is None or (bias.dtype == torch.float32 and bias.shape == (E,) and bias.is_contiguous())
     lib = load_family("moe")
     _check(lib.wllm_moe_route_corrected(_ptr(x), _dt(x), _ptr(w_router), _ptr(w_gate), _ptr(chosen), _ptr(weights), _ptr(gate_out), n, H, E,
-                                        top, groups, groups_kept, 1 if scores == "sigmoid" else 0, _ptr(correction),
-                                        c_float(-1.0 if renorm_eps is None else renorm_eps), _stream()), f"moe_route(experts={E}, top={top}, groups={groups}/{groups_kept})")
+                                        top, groups, groups_kept, ROUTER_SCORES[scores], _ptr(correction),
+                                        c_float(-1.0 if renorm_eps is None else renorm_eps), _ptr(bias), _stream()), f"moe_route(experts={E}, top={top}, groups={groups}/{groups_kept})")
 
 
 MOE_TILE_ROWS = 128      # rows of a row tile of the experts' products on the tensor-memory kernel
@@ -1282,28 +1394,36 @@ def moe_plan(chosen: torch.Tensor, count: torch.Tensor, offset: torch.Tensor, or
     launches += 1
 
 
+def _check_unit(unit, gated: bool) -> None:
+    if unit not in ((None,) + EXPERT_GATED_UNITS if gated else (None, "relu_squared")):
+        raise KernelError(f"expert unit {unit!r}: None or 'relu_squared' without a gate, {' or '.join(EXPERT_GATED_UNITS)} with one")
+
+
 def moe_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, offset: torch.Tensor, order: torch.Tensor, top: int,
                 gated: bool, limit: float = 0.0, slope: float = 0.0, unit: str | None = None,
                 row_weights: torch.Tensor | None = None) -> torch.Tensor:
     """The experts' products over rows sorted by expert.  gated: a [n, K] holds the tokens' rows (sorted row r reads row
-    order[r] // top), w [E, 2N, K] = [gate; up] per expert, out [pairs, N] = the clamped gated unit, in the operands' type.
+    order[r] // top), w [E, 2N, K] = [gate; up] per expert, out [pairs, N] = the clamped gated unit (`unit` 'silu': silu(gate) up,
+    without limit and slope), in the operands' type.
     `unit` 'relu_squared' (not gated): a [n, K] holds the tokens' rows too, w [E, N, K], out [pairs, N] = relu(s (w a))^2 in the
     operands' type, s = row_weights[pair] (float32 [pairs] in pair order; None: 1).
     Otherwise a [pairs, K] holds sorted rows, w [E, N, K], out [pairs, N] float32.  32-bit accumulation."""
     _need_cuda(a, w, out, offset, order, row_weights)
-    if unit not in (None, "relu_squared") or (unit is not None and gated):
-        raise KernelError(f"expert unit {unit!r}: None or 'relu_squared', and not gated")
+    _check_unit(unit, gated)
+    shift = 1.0
+    if gated and unit == "silu":
+        limit, slope, shift = float("inf"), 1.0, 0.0
     E, pairs, K = w.shape[0], order.shape[0], a.shape[1]
     N = w.shape[1] // 2 if gated else w.shape[1]
-    gathers = gated or unit is not None
+    gathers = gated or unit is not None          # (without a unit: the down product, which reads sorted rows)
     assert a.dtype == w.dtype and a.stride(1) == 1 and w.is_contiguous() and w.shape[2] == K and out.is_contiguous()
     assert out.shape == (pairs, N) and out.dtype == (a.dtype if gathers else torch.float32) and offset.shape == (E + 1,)
     assert gathers or a.shape[0] == pairs
-    assert row_weights is None or (unit is not None and row_weights.dtype == torch.float32 and row_weights.numel() == pairs and row_weights.is_contiguous())
+    assert row_weights is None or (unit == "relu_squared" and row_weights.dtype == torch.float32 and row_weights.numel() == pairs and row_weights.is_contiguous())
     lib = load_family("moe")
     _check(lib.wllm_moe_grouped_unit(_ptr(a), a.stride(0), _ptr(w), _ptr(out), _dt(a), 1 if gated else (2 if unit else 0), pairs, N, K,
                                      _ptr(_int32(offset, "offset")), _ptr(_int32(order, "order")), E, top, c_float(limit), c_float(slope),
-                                     _ptr(row_weights), _stream()), f"moe_grouped({pairs}x{N}x{K}, {E} experts)")
+                                     c_float(shift), _ptr(row_weights), _stream()), f"moe_grouped({pairs}x{N}x{K}, {E} experts)")
     return out
 
 
@@ -1329,7 +1449,7 @@ def tc_grouped_ok(a: torch.Tensor, w: torch.Tensor) -> bool:
 def gemm_bf16_tc_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, tiles: torch.Tensor, gated: bool, limit: float = 0.0,
                          slope: float = 0.0, unit: str | None = None) -> torch.Tensor:
     """The experts' products on tcgen05 tensor cores (csrc/gemm_bf16_tc.cu, grouped): a [rows, K] bfloat16 rows sorted by
-    expert, w [E, N, K] (or, gated, [E, 2N, K] = [gate; up]: out = the clamped gated unit, bfloat16 [rows, N]; else out float32
+    expert, w [E, N, K] (or, gated, [E, 2N, K] = [gate; up]: out = the clamped gated unit, `unit` 'silu': silu(gate) up, bfloat16 [rows, N]; else out float32
     [rows, N]; `unit` 'relu_squared': out = relu(a w^T)^2, bfloat16), `tiles` the table of row tiles that moe_plan left on the device."""
     _need_cuda(a, w, out, tiles)
     if not tc_grouped_ok(a, w):
@@ -1337,12 +1457,12 @@ def gemm_bf16_tc_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, ti
     rows, K = a.shape
     E = w.shape[0]
     N = w.shape[1] // 2 if gated else w.shape[1]
-    if unit not in (None, "relu_squared") or (unit is not None and gated):
-        raise KernelError(f"expert unit {unit!r}: None or 'relu_squared', and not gated")
+    _check_unit(unit, gated)
+    epilogue = (3 if unit == "silu" else 5) if gated else (6 if unit else 1)
     assert out.shape == (rows, N) and out.is_contiguous() and out.dtype == (torch.bfloat16 if gated or unit else torch.float32)
     assert tiles.dtype == torch.int32 and tiles.numel() >= 1 + 3 * moe_row_tiles(rows, E)
     lib = load_family("gemm_bf16_tc")
-    _check(lib.wllm_gemm_bf16_tc_grouped(_ptr(a), K, _ptr(w), K, _ptr(out), N, rows, N, K, E, 5 if gated else (6 if unit else 1), _ptr(tiles),
+    _check(lib.wllm_gemm_bf16_tc_grouped(_ptr(a), K, _ptr(w), K, _ptr(out), N, rows, N, K, E, epilogue, _ptr(tiles),
                                          moe_row_tiles(rows, E), _ptr(_status_word(a.device)), sm_count(), c_float(limit),
                                          c_float(slope), _stream()), f"gemm_bf16_tc_grouped({rows}x{N}x{K}, {E} experts)")
     return out

@@ -1,2 +1,2 @@
 """Built-in architectures: importing this package registers them."""
-from . import fusanex, gemma, gudarax, pesanex, taritar, zafilix  # noqa: F401
+from . import fusanex, gemma, gudarax, pesanex, taritar, vifirax, zafilix  # noqa: F401

@@ -31,7 +31,12 @@ first layer leaves its values in a buffer of the step; its own `weight` tensor i
 any of "q": name, "k": name, "values": True}: every query and key head is divided by its root mean square and multiplied by the
 gain [head_dim] of that name, shared by the heads, in front of the turn; with `values` every value head is divided by its root mean
 square before it is cached), query_temperature ({"coef": c, "every": m}: queries are multiplied by
-1 + c * ln(floor((p + 1) / m) + 1) at position p; with head_norm).
+1 + c * ln(floor((p + 1) / m) + 1) at position p; with head_norm), sink_score (a number: every query head's softmax
+denominator has e^that as one more term, a sink without a tensor; not with `sink`), head_gate (checkpoint name of a matrix
+[num_heads, hidden]: a head's output is multiplied by the sigmoid of its one number, computed by the same product as q, k and
+v; not with gate_proj).  `bias` may also name "o", the bias row of the output projection; it is handed on as a
+`BiasedBranch` and added in 32-bit.  A mixer that reads another run's cache may norm its query row ("q" alone in row_norm and
+in bias).
 
 A mixer may be one of several that read the same input (a block that runs two mixers side
 by side): `input_weights()` lists the matrices that read the input, `mix(fused, parts,
@@ -51,7 +56,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import MIXERS, POSITIONS, CacheRef, KVNeed, ParamSpec, as_branch
+from .base import MIXERS, POSITIONS, BiasedBranch, CacheRef, KVNeed, ParamSpec, as_branch
 
 
 @MIXERS.register("attention")
@@ -84,8 +89,10 @@ class PagedAttention:
         self.value_mix = spec.options.get("value_mix")
         if self.value_mix is not None and self.value_mix["role"] not in ("first", "later"):
             raise ValueError(f"value_mix role {self.value_mix['role']!r}: 'first' or 'later'")
-        if (self.bias_names is not None or self.value_mix is not None) and (self.row_norm is None or self.borrows):
+        if (self.bias_names is not None or self.value_mix is not None) and self.row_norm is None:
             raise ValueError("projection biases and blended values are built into the kernel that norms q and k as whole rows (row_norm)")
+        if self.value_mix is not None and self.borrows:
+            raise ValueError("blended values need the mixer's own value projection")
         if self.slope_values is not None and len(self.slope_values) != self.nq:
             raise ValueError(f"{len(self.slope_values)} distance slopes for {self.nq} query heads")
         self.head_norm = spec.options.get("head_norm")
@@ -96,9 +103,13 @@ class PagedAttention:
             raise ValueError("head norms carry gains for q and k, or for neither")
         if self.temperature is not None and self.head_norm is None:
             raise ValueError("a query temperature is built into the kernel that norms heads (head_norm)")
-        if self.row_norm is not None and self.borrows:
-            raise ValueError("row norms of q and k need the mixer's own key projection")
+        self.head_gate_name = spec.options.get("head_gate")
+        if self.head_gate_name is not None and self.gate_name is not None:
+            raise ValueError("the heads' outputs are gated element by element (gate_proj) or head by head (head_gate), not both")
         self.position = POSITIONS.build(spec.position)
+        self.turn_scale = float(getattr(self.position, "turn_scale", 1.0))
+        if self.turn_scale != 1.0 and (self.head_norm is not None or spec.options.get("qk_unit_norm_eps") is not None):
+            raise ValueError("a factor on the turn is not built into the kernels that norm head by head")
         self.vd = int(spec.options.get("value_dim") or self.hd)
         scale = spec.options.get("scale")
         self.scale = float(self.hd) ** -0.5 if scale is None else float(scale)
@@ -109,16 +120,20 @@ class PagedAttention:
         self.hd, self.vd = -(-self.hd // 8) * 8, -(-self.vd // 8) * 8
         if spec.options.get("qk_unit_norm_eps") is not None and self.hd != self.hd_file:
             raise ValueError(f"head size {self.hd_file}: heads that are divided by their root mean square come in steps of 8 elements")
-        self.sink_name = spec.options.get("sink")
+        self.sink_name, self.sink_score = spec.options.get("sink"), spec.options.get("sink_score")
+        if self.sink_name is not None and self.sink_score is not None:
+            raise ValueError("a sink has its scores from a tensor (sink) or one fixed score (sink_score), not both")
         self.unit_norm_eps = spec.options.get("qk_unit_norm_eps")
         # the tensor-core kernels take keys and values of one size; other cases run on the general kernels
         self.general = self.vd != self.hd
         # columns of the fused q|k|v row (q alone in a mixer that reads another's keys and values), the gate's behind them
         self.qkv_width = self.nq * self.hd if self.borrows else (self.nq + self.nkv) * self.hd + self.nkv * self.vd
         self.width = self.qkv_width + (self.nq * self.vd if self.gate_name is not None else 0)
+        if self.head_gate_name is not None:      # the product's rows in steps of 8 columns (16 bytes of the matrix type)
+            self.width += -(-self.nq // 8) * 8
         self.q_gain = self.k_gain = None
         self.tag = ""                    # set by a mixer that runs this one beside another: keeps their buffers apart
-        self.wqkv = self.wo = self.sinks = self.bias = self.slopes = self.blend = None
+        self.wqkv = self.wo = self.sinks = self.bias = self.out_bias = self.slopes = self.blend = None
 
     def cache_need(self):
         return KVNeed(self.nkv, self.hd, self.window, self.vd if self.vd != self.hd else None, self.keep_first, blocks=self.blocks)
@@ -132,18 +147,27 @@ class PagedAttention:
             out.append(ParamSpec(self.sink_name, (self.nq,), "vector"))
         if self.gate_name is not None:
             out.append(ParamSpec(self.gate_name, (self.nq * self.vd_file, H)))
+        if self.head_gate_name is not None:
+            out.append(ParamSpec(self.head_gate_name, (self.nq, H)))
         if self.row_norm is not None:
-            out += [ParamSpec(self.row_norm["q"], (self.nq * self.hd_file,), "vector"),
-                    ParamSpec(self.row_norm["k"], (self.nkv * self.hd_file,), "vector")]
+            out += [ParamSpec(self.row_norm[k], (heads * self.hd_file,), "vector") for k, heads in self._query_key()]
         if self.head_norm is not None and "q" in self.head_norm:
             out += [ParamSpec(self.head_norm[k], (self.hd_file,), "vector") for k in ("q", "k")]
         if self.bias_names is not None:
-            out += [ParamSpec(self.bias_names["q"], (self.nq * self.hd_file,), "vector"),
-                    ParamSpec(self.bias_names["k"], (self.nkv * self.hd_file,), "vector"),
-                    ParamSpec(self.bias_names["v"], (self.nkv * self.vd_file,), "vector")]
+            out += [ParamSpec(self.bias_names[k], (heads * size,), "vector") for k, heads, size, _ in self._projections()]
+            if "o" in self.bias_names:
+                out.append(ParamSpec(self.bias_names["o"], (H,), "vector"))
         if self.value_mix is not None:
             out.append(ParamSpec(self.value_mix["weight"], (), "vector"))
         return out
+
+    def _query_key(self) -> list:
+        return [("q", self.nq)] + ([] if self.borrows else [("k", self.nkv)])
+
+    def _projections(self) -> list:
+        """(name, heads, a head's size in the checkpoint, the size it is held in) of the mixer's own projections."""
+        own = [] if self.borrows else [("k", self.nkv, self.hd_file, self.hd), ("v", self.nkv, self.vd_file, self.vd)]
+        return [("q", self.nq, self.hd_file, self.hd)] + own
 
     def load(self, fetch):
         n = self.names
@@ -161,24 +185,31 @@ class PagedAttention:
                                    heads_padded(fetch(n["v_proj"]), self.nkv, self.vd_file, self.vd)], dim=0).contiguous()
         if self.gate_name is not None:
             self.wqkv = torch.cat([self.wqkv, heads_padded(fetch(self.gate_name), self.nq, self.vd_file, self.vd)], dim=0).contiguous()
+        if self.head_gate_name is not None:
+            rows = fetch(self.head_gate_name)
+            pad = rows.new_zeros((self.width - self.qkv_width - self.nq, self.hidden_size))
+            self.wqkv = torch.cat([self.wqkv, rows, pad], dim=0).contiguous()
         if self.row_norm is not None:
             gains = [heads_padded(fetch(self.row_norm[k])[:, None], heads, self.hd_file, self.hd)[:, 0].contiguous()
-                     for k, heads in (("q", self.nq), ("k", self.nkv))]
-            self.q_gain, self.k_gain = gains
+                     for k, heads in self._query_key()]
+            self.q_gain, self.k_gain = gains if len(gains) == 2 else (gains[0], None)
         if self.head_norm is not None and "q" in self.head_norm:
             self.q_gain, self.k_gain = (heads_padded(fetch(self.head_norm[k])[:, None], 1, self.hd_file, self.hd)[:, 0].contiguous()
                                         for k in ("q", "k"))
         if self.bias_names is not None:
             rows = [heads_padded(fetch(self.bias_names[k]).to(torch.float32)[:, None], heads, size, to)[:, 0]
-                    for k, heads, size, to in (("q", self.nq, self.hd_file, self.hd), ("k", self.nkv, self.hd_file, self.hd),
-                                               ("v", self.nkv, self.vd_file, self.vd))]
+                    for k, heads, size, to in self._projections()]
             self.bias = torch.cat(rows).contiguous()
+            if "o" in self.bias_names:
+                self.out_bias = fetch(self.bias_names["o"]).to(torch.float32).contiguous()
         if self.value_mix is not None:
             self.blend = fetch(self.value_mix["weight"]).to(torch.float32).reshape(1).contiguous()
         wo = fetch(n["o_proj"])
         self.wo = heads_padded(wo.t().contiguous(), self.nq, self.vd_file, self.vd).t().contiguous()
         if self.sink_name is not None:
             self.sinks = fetch(self.sink_name).to(torch.float32).contiguous()
+        if self.sink_score is not None:
+            self.sinks = torch.full((self.nq,), float(self.sink_score), dtype=torch.float32, device=self.wo.device)
         if self.slope_values is not None:
             self.slopes = torch.tensor(self.slope_values, dtype=torch.float64).to(torch.float32).to(self.wo.device)
         self.position.to(self.wo.device)
@@ -194,7 +225,8 @@ class PagedAttention:
         """The mixer on columns col0 .. col0 + width of a fused product [n, W] (or partial sums [parts, n, W])."""
         attn = ctx.buffer(self.tag + "attn", (fused.shape[-2], self.nq * self.vd), self.model_dtype)
         self.heads(fused, parts, col0, ctx, cache, attn)
-        return as_branch(ops.project(attn, self.wo, lambda name, shape, dt: ctx.buffer(self.tag + "branch_" + name, shape, dt)))
+        branch = as_branch(ops.project(attn, self.wo, lambda name, shape, dt: ctx.buffer(self.tag + "branch_" + name, shape, dt)))
+        return branch if self.out_bias is None else BiasedBranch(branch, self.out_bias)
 
     def heads(self, fused: torch.Tensor, parts: int, col0: int, ctx, cache: CacheRef, attn: torch.Tensor) -> None:
         """The heads' outputs (what the output projection reads) into `attn` [n, num_heads * value size], whose rows may be columns of
@@ -211,15 +243,19 @@ class PagedAttention:
             extra["vd"] = self.vd
         if self.unit_norm_eps is not None:
             extra["unit_norm_eps"] = float(self.unit_norm_eps)
+        if self.turn_scale != 1.0:
+            extra["turn_scale"] = self.turn_scale
         slots = ctx.group_slots[cache.group] if cache.writes else None
         pairing = getattr(self.position, "pairing", "half")
         if self.row_norm is not None:
             if self.unit_norm_eps is not None:
                 raise ValueError("q and k are normed either as whole rows or head by head, not both")
-            ops.rope_row_norm_kv_write(qkv, q, ctx.positions, slots, self.position.inv_freq, k_pages, v_pages, self.nq, self.nkv,
+            nkv = 0 if self.borrows else self.nkv
+            ops.rope_row_norm_kv_write(qkv, q, ctx.positions, slots, self.position.inv_freq, k_pages, v_pages, self.nq, nkv,
                                        self.hd, self.position.rotary_dim, group.page_size, self.q_gain, self.k_gain,
-                                       float(self.row_norm["eps"]), self.nq * self.hd_file, self.nkv * self.hd_file,
-                                       in_splits=parts, pairing=pairing, vd=self.vd, bias=self.bias, **self._blend_args(n, ctx))
+                                       float(self.row_norm["eps"]), self.nq * self.hd_file, nkv * self.hd_file,
+                                       in_splits=parts, pairing=pairing, bias=self.bias, **{**extra, "vd": self.vd},
+                                       **self._blend_args(n, ctx))
         elif self.head_norm is not None:
             t = self.temperature or {"coef": 0.0, "every": 0}
             ops.rope_head_norm_kv_write(qkv, q, ctx.positions, slots, self.position.inv_freq, k_pages, v_pages, self.nq, self.nkv, self.hd,
@@ -233,6 +269,8 @@ class PagedAttention:
         self.attend(q, attn, k_pages, v_pages, ctx, cache.group)
         if self.gate_name is not None:
             ops.sigmoid_gate(attn, qkv, parts, self.qkv_width)
+        if self.head_gate_name is not None:
+            ops.sigmoid_gate(attn, qkv, parts, self.qkv_width, per=self.vd)
 
     def _blend_args(self, n: int, ctx) -> dict:
         """The buffer of the step in which the first layer of a label leaves its values, and this layer's part in it."""

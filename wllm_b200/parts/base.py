@@ -19,7 +19,7 @@ Interfaces (duck-typed; see the built-in parts for examples):
     norm            __call__(residual: Residual, ctx) -> tensor [n, hidden] in the model dtype
                     rows(residual, rows, ctx) -> the same at selected rows only
     position        an object the mixer of its kind understands (rotary: .inv_freq, .rotary_dim, and
-                    optionally .pairing = 'half' | 'interleaved')
+                    optionally .pairing = 'half' | 'interleaved', .turn_scale = a factor on the sines and cosines)
     mixer           cache_need() -> KVNeed | StateNeed | None, or a tuple of them (a mixer that reads pages
                     and keeps state of its own)
                     __call__(x, ctx, cache: CacheRef) -> tensor [n, hidden]
@@ -153,10 +153,23 @@ class BranchSum:
         return out
 
 
+class BiasedBranch:
+    """A branch output whose projection's bias row (float32 [hidden]) is still to be added.  The norm behind the sublayer adds it
+    inside its own kernel; `materialize` does it alone."""
+
+    def __init__(self, branch, bias: torch.Tensor):
+        self.branch, self.bias = branch, bias
+
+    def materialize(self, ctx, name: str = "branch_biased") -> torch.Tensor:
+        from ..kernels import ops
+        pair = branch_pair(self.branch)
+        return ops.branch_bias(pair, self.bias, ctx.buffer(name, tuple(pair[0].shape[-2:]), torch.float32))
+
+
 class NormedBranch:
     """A branch output that is to pass a norm of its own before it joins the residual (a block that norms behind its
-    sublayers): `branch` is a tensor, `Partials` or `MeanOfNormed`, `norm` the norm part.  The next norm of the
-    residual does both in one kernel when it can; `materialize` runs the branch's norm alone."""
+    sublayers): `branch` is a tensor, `Partials`, `BiasedBranch` or `MeanOfNormed`, `norm` the norm part.  The next norm of
+    the residual does both in one kernel when it can; `materialize` runs the branch's norm alone."""
 
     def __init__(self, branch, norm):
         self.branch, self.norm = branch, norm

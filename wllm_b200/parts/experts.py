@@ -11,7 +11,10 @@ the options of a 'gated_dense' unit that every token runs, plus gate_weight: the
 unit's output is multiplied by sigmoid(row . x); without gate_weight it is added as it is), identity (so many further experts behind the
 num_experts, without tensors, whose output is the token's row itself; the router has a row for each), correction (checkpoint
 name of a vector [num_experts + identity] that joins the scores for the choice alone), renorm_eps (the weights are the chosen
-scores over their sum + renorm_eps; absent: the scores as they are).
+scores over their sum + renorm_eps; absent: the scores as they are), router_bias (checkpoint name of a vector [num_experts + identity]
+added to the router's logits).  scores may also be 'softmax_chosen': the `top` largest logits are chosen and weighted by the softmax
+over the chosen logits alone (no groups, correction or renorm_eps).  A gated expert's activation is 'capped_swish' (limit, slope) or
+'silu' (down(silu(gate x) * up x), no limit or slope).
 
 Router logits, the softmax over all experts, the choice and the weights (the chosen experts' scores as they are) are
 32-bit, against a 32-bit copy of the router matrix.  The tokens' (token, rank) pairs are sorted by expert on the device
@@ -44,17 +47,19 @@ class RoutedExperts:
         self.inter, self.activation = int(spec.intermediate_size), spec.activation
         self.gated = bool(spec.options.get("gated", True))
         self.scores, self.weight_on = spec.options.get("scores") or "softmax", spec.options.get("weight_on") or "output"
-        if self.scores not in ("softmax", "sigmoid") or self.weight_on not in ("output", "input"):
-            raise ValueError(f"scores {self.scores!r} ('softmax', 'sigmoid'), weight_on {self.weight_on!r} ('output', 'input')")
-        if self.activation != ("capped_swish" if self.gated else "relu_squared"):
-            raise ValueError("the grouped expert products are built for gated experts with the activation capped_swish and for "
-                             "experts without a gate with relu_squared")
+        if self.scores not in ops.ROUTER_SCORES or self.weight_on not in ("output", "input"):
+            raise ValueError(f"scores {self.scores!r} ({', '.join(ops.ROUTER_SCORES)}), weight_on {self.weight_on!r} ('output', 'input')")
+        if self.scores == "softmax_chosen" and (self.groups > 1 or self.correction_name is not None or self.renorm_eps is not None):
+            raise ValueError("a softmax over the chosen logits knows no groups, no correction and no division by the scores' sum")
+        if self.activation not in (ops.EXPERT_GATED_UNITS if self.gated else ("relu_squared",)):
+            raise ValueError(f"the grouped expert products are built for gated experts with the activation {' or '.join(ops.EXPERT_GATED_UNITS)} "
+                             "and for experts without a gate with relu_squared")
         if self.weight_on == "input" and self.identity:
             raise ValueError("scores on the experts' inputs are built without identity experts")
         if self.weight_on == "input" and self.gated:
             raise ValueError("scores on the experts' inputs are built for experts without a gate")
         self.limit, self.slope = float(spec.options.get("limit") or 0.0), float(spec.options.get("slope") or 0.0)
-        self.router_name, self.prefix = spec.router, spec.expert_prefix
+        self.router_name, self.prefix, self.bias_name = spec.router, spec.expert_prefix, spec.options.get("router_bias")
         self.hidden_size, self.model_dtype = hidden_size, model_dtype
         self.shared = self.gate_name = None
         shared = spec.options.get("shared")
@@ -62,7 +67,7 @@ class RoutedExperts:
             shared = dict(shared)
             self.gate_name = shared.pop("gate_weight", None)
             self.shared = FEED_FORWARDS.build(make_spec("gated_dense", **shared), hidden_size=hidden_size, model_dtype=model_dtype)
-        self.w_router = self.w_gate = self.w_gu = self.w_down = self.correction = None
+        self.w_router = self.w_gate = self.w_gu = self.w_down = self.correction = self.router_bias = None
 
     def parts(self):
         return [] if self.shared is None else [self.shared]
@@ -72,6 +77,8 @@ class RoutedExperts:
         out = [ParamSpec(self.router_name, (self.slots, H))]
         if self.correction_name is not None:
             out.append(ParamSpec(self.correction_name, (self.slots,), "vector"))
+        if self.bias_name is not None:
+            out.append(ParamSpec(self.bias_name, (self.slots,), "vector"))
         for j in range(self.E):
             p = f"{self.prefix}{j}."
             out += ([ParamSpec(p + "gate", (I, H))] if self.gated else []) + [ParamSpec(p + "up", (I, H)), ParamSpec(p + "down", (H, I))]
@@ -83,6 +90,8 @@ class RoutedExperts:
         self.w_router = fetch(self.router_name).to(torch.float32).contiguous()
         if self.correction_name is not None:
             self.correction = fetch(self.correction_name).to(torch.float32).contiguous()
+        if self.bias_name is not None:
+            self.router_bias = fetch(self.bias_name).to(torch.float32).contiguous()
         names = [f"{self.prefix}{j}." for j in range(self.E)]
         if self.gated:
             self.w_gu = torch.stack([torch.cat([fetch(p + "gate"), fetch(p + "up")], dim=0) for p in names]).contiguous()
@@ -101,8 +110,8 @@ class RoutedExperts:
         weights = ctx.buffer("moe_weights", (n, top), torch.float32)
         gate = ctx.buffer("moe_gate", (n,), torch.float32) if self.gate_name is not None else None
         ops.moe_route(x, self.w_router, self.w_gate, chosen, weights, gate, self.groups, self.groups_kept, scores=self.scores,
-                      correction=self.correction, renorm_eps=self.renorm_eps)
-        unit = None if self.gated else self.activation
+                      correction=self.correction, renorm_eps=self.renorm_eps, bias=self.router_bias)
+        unit = None if self.activation == "capped_swish" else self.activation
         on_input = weights.view(-1) if self.weight_on == "input" else None
         slots = self.slots
         index = ctx.buffer("moe_index", (2 * slots + 1 + 2 * pairs,), torch.int32)

@@ -43,6 +43,8 @@ class LatentAttention:
         self.scale, self.eps = float(spec.scale), float(spec.eps)
         self.hidden_size, self.model_dtype = hidden_size, model_dtype
         self.position = POSITIONS.build(spec.position)
+        if getattr(self.position, "turn_scale", 1.0) != 1.0:
+            raise ValueError("a factor on the turn is not built into attention over latent rows")
         if self.position.head_dim != self.rot:
             raise ValueError(f"the rotary encoding covers {self.position.head_dim} elements, the turning part has {self.rot}")
         # a cached row is held in steps of 8 elements (16-byte loads), zeros behind the turned part

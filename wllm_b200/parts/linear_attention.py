@@ -30,6 +30,10 @@ the token itself, inputs in front of the sequence count as zero; the newest taps
 unit_norm_eps), q is also multiplied by q_scale; beta_t = sigmoid(beta_proj x) and g_t = exp(-exp(decay_log) softplus(decay_proj x +
 decay_bias)), one of each per head.  Each head's o is divided by its root mean square over value_dim (eps), times the gain
 head_norm_weight shared by the heads, times silu(g_proj x); then o_proj.
+With decay_maps {"down": name, "up": name} in place of decay_proj there is one decay per head and key channel, g_t = exp(-exp(decay_log_h)
+softplus(up (down x) + decay_bias)) with up [heads * key_dim, rank] and decay_bias [heads * key_dim]; it multiplies the rows of S.
+With gate_maps {"down": name, "up": name} in place of g_proj the gate is sigmoid(up (down x)), up [heads * value_dim, rank].  Both
+ranks are the checkpoint's unless the maps say `rank`.
 spec options: num_heads, num_kv_heads, key_dim, value_dim, conv_taps, eps, unit_norm_eps, q_scale, q_proj/k_proj/v_proj/g_proj/
 o_proj, q_conv/k_conv/v_conv [channels, taps], beta_proj, decay_proj [heads, hidden], decay_log, decay_bias [heads],
 head_norm_weight [value_dim] (checkpoint names).  One product makes q | k | v | g | beta | decay; what enters the
@@ -56,6 +60,8 @@ class LinearAttention:
         self.hidden_size, self.model_dtype = hidden_size, model_dtype
         self.names = {k: spec.options[k] for k in ("q_proj", "k_proj", "v_proj", "g_proj", "o_proj")}
         self.position = POSITIONS.build(spec.position) if spec.options.get("position") is not None else None
+        if getattr(self.position, "turn_scale", 1.0) != 1.0:
+            raise ValueError("a factor on the turn is not built into the recurrence's inputs")
         decay = dict(spec.decay)
         self.decay_kind = decay["kind"]
         if self.decay_kind == "per_head":
@@ -160,6 +166,8 @@ class ParallelMean:
             if not hasattr(m, "mix") or not hasattr(m, "input_weights"):
                 raise TypeError(f"the {side} mixer ({type(m).__name__}) cannot share a fused input product")
             m.tag = side + "_" + getattr(m, "tag", "")
+            if "o" in (getattr(m, "bias_names", None) or {}):
+                raise ValueError(f"the {side} mixer's output has a bias: the norm of two mixers' outputs takes none")
         self.eps = float(spec.eps)
         self.names = {"left": spec.left_out, "right": spec.right_out}
         self.hidden_size, self.model_dtype = hidden_size, model_dtype
@@ -227,14 +235,15 @@ class DeltaRule:
                              f"channels and convolutions of up to 16 taps")
         self.eps, self.unit_eps, self.q_scale = float(spec.eps), float(spec.unit_norm_eps), float(spec.options.get("q_scale", 1.0))
         self.hidden_size, self.model_dtype = hidden_size, model_dtype
-        self.names = {k: spec.options[k] for k in ("q_proj", "k_proj", "v_proj", "g_proj", "o_proj", "q_conv", "k_conv", "v_conv",
-                                                   "beta_proj", "decay_proj", "decay_log", "decay_bias", "head_norm_weight")}
+        self.decay_maps, self.gate_maps = spec.options.get("decay_maps"), spec.options.get("gate_maps")
+        self.names = {k: spec.options[k] for k in ["q_proj", "k_proj", "v_proj", "o_proj", "q_conv", "k_conv", "v_conv", "beta_proj", "decay_log",
+                                                   "decay_bias", "head_norm_weight"] +
+                      (["g_proj"] if self.gate_maps is None else []) + (["decay_proj"] if self.decay_maps is None else [])}
         GD, HV = self.kv_heads * self.dim, self.heads * self.vdim
-        self.offsets = {"q": 0, "k": GD, "v": 2 * GD, "g": 2 * GD + HV, "b": 2 * GD + 2 * HV, "a": 2 * GD + 2 * HV + self.heads}
-        self.width = 2 * GD + 2 * HV + 2 * self.heads
         self.channels = 2 * GD + HV
         self.tag = ""
-        self.w_in = self.wo = self.conv = self.a_log = self.dt_bias = self.norm_weight = None
+        self.offsets = self.width = None         # columns of the fused product; the maps' ranks may be the checkpoint's
+        self.w_in = self.wo = self.conv = self.a_log = self.dt_bias = self.norm_weight = self.decay_up = self.gate_up = None
 
     def cache_need(self):
         need = [("state", (self.heads, self.dim, self.vdim), torch.float32)]
@@ -244,15 +253,45 @@ class DeltaRule:
 
     def param_specs(self):
         H, n, GD, HV = self.hidden_size, self.names, self.kv_heads * self.dim, self.heads * self.vdim
-        return [ParamSpec(n["q_proj"], (GD, H)), ParamSpec(n["k_proj"], (GD, H)), ParamSpec(n["v_proj"], (HV, H)),
-                ParamSpec(n["g_proj"], (HV, H)), ParamSpec(n["beta_proj"], (self.heads, H)), ParamSpec(n["decay_proj"], (self.heads, H)),
-                ParamSpec(n["o_proj"], (H, HV)), ParamSpec(n["q_conv"], (GD, self.taps)), ParamSpec(n["k_conv"], (GD, self.taps)),
-                ParamSpec(n["v_conv"], (HV, self.taps)), ParamSpec(n["decay_log"], (self.heads,), "vector"),
-                ParamSpec(n["decay_bias"], (self.heads,), "vector"), ParamSpec(n["head_norm_weight"], (self.vdim,), "vector")]
+        def maps(m, rows):
+            return [ParamSpec(m["down"], (m.get("rank"), H)), ParamSpec(m["up"], (rows, m.get("rank")))]
+        out = [ParamSpec(n["q_proj"], (GD, H)), ParamSpec(n["k_proj"], (GD, H)), ParamSpec(n["v_proj"], (HV, H))]
+        out += [ParamSpec(n["g_proj"], (HV, H))] if self.gate_maps is None else maps(self.gate_maps, HV)
+        out.append(ParamSpec(n["beta_proj"], (self.heads, H)))
+        out += [ParamSpec(n["decay_proj"], (self.heads, H))] if self.decay_maps is None else maps(self.decay_maps, self.heads * self.dim)
+        return out + [ParamSpec(n["o_proj"], (H, HV)), ParamSpec(n["q_conv"], (GD, self.taps)), ParamSpec(n["k_conv"], (GD, self.taps)),
+                      ParamSpec(n["v_conv"], (HV, self.taps)), ParamSpec(n["decay_log"], (self.heads,), "vector"),
+                      ParamSpec(n["decay_bias"], (self.heads * (1 if self.decay_maps is None else self.dim),), "vector"),
+                      ParamSpec(n["head_norm_weight"], (self.vdim,), "vector")]
+
+    def _maps(self, fetch, m: dict) -> tuple:
+        """(down, up) of a low-rank map, the rank in steps of 8 (with zeros)."""
+        down, up = fetch(m["down"]), fetch(m["up"])
+        if down.shape[0] != up.shape[1]:
+            raise ValueError(f"{m['down']} has {down.shape[0]} rows, {m['up']} reads {up.shape[1]}")
+        pad = -down.shape[0] % 8
+        if pad:
+            down = torch.cat([down, down.new_zeros((pad, down.shape[1]))], dim=0)
+            up = torch.cat([up, up.new_zeros((up.shape[0], pad))], dim=1)
+        return down, up.contiguous()
 
     def load(self, fetch):
         n = self.names
-        mats = [fetch(n[k]) for k in ("q_proj", "k_proj", "v_proj", "g_proj", "beta_proj", "decay_proj")]
+        rows = {"q": fetch(n["q_proj"]), "k": fetch(n["k_proj"]), "v": fetch(n["v_proj"])}
+        if self.gate_maps is None:
+            rows["g"] = fetch(n["g_proj"])
+        else:
+            rows["g_low"], self.gate_up = self._maps(fetch, self.gate_maps)
+        if self.decay_maps is not None:
+            rows["a_low"], self.decay_up = self._maps(fetch, self.decay_maps)
+        rows["b"] = fetch(n["beta_proj"])
+        if self.decay_maps is None:
+            rows["a"] = fetch(n["decay_proj"])
+        self.offsets, self.width = {}, 0
+        for k, w in rows.items():
+            self.offsets[k] = self.width
+            self.width += w.shape[0]
+        mats = list(rows.values())
         pad = -self.width % 8             # the product's rows in steps of 8 columns (16 bytes of the matrix type)
         if pad:
             mats.append(mats[0].new_zeros((pad, self.hidden_size)))
@@ -278,14 +317,25 @@ class DeltaRule:
         k = ctx.buffer(self.tag + "delta_k", (n, G * D), f32)
         v = ctx.buffer(self.tag + "delta_v", (n, H * V), f32)
         beta = ctx.buffer(self.tag + "delta_beta", (n, H), f32)
-        decay = ctx.buffer(self.tag + "delta_decay", (n, H), f32)
+        channel = self.decay_maps is not None
+        decay = ctx.buffer(self.tag + "delta_decay", (n, H * D if channel else H), f32)
         conv_state = ctx.state(cache.state_names["conv"]) if self.taps > 1 else None
-        ops.delta_prepare(fused, parts, off, H, G, D, V, self.taps, *self.conv, self.a_log, self.dt_bias, ctx.token_req,
-                          ctx.req_q_start, ctx.req_slot, conv_state, self.unit_eps, self.q_scale, q, k, v, beta, decay)
-        ops.delta_conv_update(fused, parts, off, H, G, D, V, self.taps, ctx.req_q_start, ctx.req_q_len, ctx.req_slot, conv_state)
+        per_head = (None, None) if channel else (self.a_log, self.dt_bias)
+        single = ctx.num_multi == 0              # no request brings more than one token
+        ops.delta_prepare(fused, parts, off, H, G, D, V, self.taps, *self.conv, *per_head, ctx.token_req, ctx.req_q_start, ctx.req_slot,
+                          conv_state, self.unit_eps, self.q_scale, q, k, v, beta, None if channel else decay,
+                          shift=ctx.req_q_len if single else None)
+        if not single:
+            ops.delta_conv_update(fused, parts, off, H, G, D, V, self.taps, ctx.req_q_start, ctx.req_q_len, ctx.req_slot, conv_state)
+        if channel:
+            ops.lowrank_map(fused, parts, off["a_low"], self.decay_up, H, D, decay, self.dt_bias, self.a_log)
         o = ctx.buffer(self.tag + "delta_o", (n, H * V), f32)
         ops.delta_scan(q, k, v, beta, decay, ctx.state(cache.state_names["state"]), o, ctx.req_q_start, ctx.req_q_len, ctx.req_slot,
-                       H, G, D, V)
+                       H, G, D, V, channel)
         gated = ctx.buffer(self.tag + "delta_gated", (n, H * V), self.model_dtype)
-        ops.head_gate_norm(o, fused, parts, off["g"], self.norm_weight, self.eps, gated, H, V)
+        if self.gate_maps is None:
+            ops.head_gate_norm(o, fused, parts, off["g"], self.norm_weight, self.eps, gated, H, V)
+        else:
+            gate = ops.lowrank_map(fused, parts, off["g_low"], self.gate_up, H, V, ctx.buffer(self.tag + "delta_gate", (n, H * V), f32))
+            ops.head_gate_norm(o, gate, 0, 0, self.norm_weight, self.eps, gated, H, V, gate_act="sigmoid")
         return as_branch(ops.project(gated, self.wo, lambda name, shape, dt: ctx.buffer(self.tag + "delta_out_" + name, shape, dt)))

@@ -18,7 +18,7 @@ from __future__ import annotations
 import torch
 
 from ..kernels import ops
-from .base import NORMS, BranchSum, MeanOfNormed, NormedBranch, ParamSpec, Partials, Residual, branch_pair
+from .base import NORMS, BiasedBranch, BranchSum, MeanOfNormed, NormedBranch, ParamSpec, Partials, Residual, branch_pair
 
 
 @NORMS.register("rmsnorm")
@@ -58,6 +58,8 @@ class RMSNorm:
             post, inner, more = pending.norm, pending.branch, {}
             if isinstance(inner, BranchSum):
                 inner = inner.materialize(ctx)
+            if isinstance(inner, BiasedBranch):
+                inner, more = inner.branch, dict(bias=inner.bias)
             if isinstance(inner, MeanOfNormed):
                 more = dict(gain_a=inner.gain_a, b=branch_pair(inner.b), gain_b=inner.gain_b, inner_eps=inner.eps, factor=inner.factor)
                 inner = inner.a

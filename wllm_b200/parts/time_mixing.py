@@ -125,6 +125,8 @@ class ParallelSum:
             raise TypeError(f"mixers added with factors: an attention mixer and a time mixing, not {type(self.left).__name__} and {type(self.right).__name__}")
         for side, m in (("left", self.left), ("right", self.right)):
             m.tag = side + "_"
+        if "o" in (getattr(self.left, "bias_names", None) or {}):
+            raise ValueError("mixers that share an output product have no bias on it")
         self.left_factor, self.right_factor = float(spec.left_factor), float(spec.right_factor)
         self.hidden_size, self.model_dtype = hidden_size, model_dtype
         self.w_in = self.w_left = self.w_out = self.mu = None
