@@ -1446,6 +1446,242 @@ def fusanex_bench(args) -> int:
     return 0
 
 
+VIFIRAX_SIZES = {
+    # width, dense feed-forward, attention (heads, kv heads, head size, turned part), state space (heads, value size, state rows, groups, taps,
+    # norm groups), delta rule (heads, q/k heads, size, value size, taps, rank of both maps), experts (matrices, chosen, feed-forward)
+    "2k": dict(width=2048, ff=6144, attn=(16, 4, 128, 64), ssm=(64, 64, 128, 8, 4, 8), delta=(16, 16, 128, 128, 4, 128), experts=(16, 2, 2048), vocab=32000),
+    "4k": dict(width=4096, ff=11008, attn=(32, 8, 128, 64), ssm=(128, 64, 128, 8, 4, 8), delta=(32, 32, 128, 128, 4, 128), experts=(16, 2, 3584), vocab=32000),
+}
+
+
+def vifirax_config(size: dict) -> dict:
+    """Four layers: a state space (routed experts), a delta rule (dense), attention (dense), attention on its keys and values (routed experts)."""
+    nq, nkv, hd, dims = size["attn"]
+    sh, sv, sn, sg, taps, parts = size["ssm"]
+    dh, dg, dd, dv, dtaps, rank = size["delta"]
+    E, top, eff = size["experts"]
+    dense, moe = {"kind": "dense", "ff": size["ff"]}, {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}}
+    att = {"heads": nq, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5,
+           "rot": {"dims": dims, "base": 1e6, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    return {"architecture": "Vifirax", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5, "layers": [
+        {"type": "mamba2", "mixer": {"heads": sh, "vdim": sv, "state": sn, "groups": sg, "conv": taps, "norm_groups": parts}, "mlp": moe},
+        {"type": "channel_delta", "mixer": {"heads": dh, "kv_heads": dg, "dim": dd, "vdim": dv, "conv": dtaps, "decay_rank": rank, "gate_rank": rank}, "mlp": dense},
+        {"type": "attention", "mixer": att, "mlp": dense}, {"type": "attention", "mixer": {**att, "kv_from": 2}, "mlp": moe}]}
+
+
+def vifirax_like_config(size: dict) -> dict:
+    """The closest of the other designs at equal sizes, a Gudarax of four layers: two delta rules and two attention layers (whole-row norms,
+    biases on q, k and v), the same feed-forwards."""
+    nq, nkv, hd, _ = size["attn"]
+    dh, dg, dd, dv, dtaps, _ = size["delta"]
+    E, top, eff = size["experts"]
+    dense, moe = {"kind": "dense", "ff": size["ff"]}, {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}}
+    att = {"heads": nq, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5}
+    dlt = {"heads": dh, "kv_heads": dg, "dim": dd, "vdim": dv, "conv": dtaps}
+    return {"architecture": "Gudarax", "vocab": size["vocab"], "width": size["width"], "max_positions": 16384, "embedding": {"scale": 1.0},
+            "norm": {"eps": 1e-6}, "layers": [{"type": "delta", "mixer": dlt, "mlp": moe}, {"type": "delta", "mixer": dlt, "mlp": dense},
+                                              {"type": "attention", "mixer": att, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe}]}
+
+
+def vifirax_kernel_table(size: dict, pk: dict, T: int, batch: int, context: int) -> dict:
+    """Vifirax's kernels alone at one size's shapes, each with its like kernel of the framework's other designs; columns as in
+    fusanex_kernel_table."""
+    import torch
+    from types import SimpleNamespace
+    from wllm_b200.kernels import ops
+    dev, bf, f32, i32 = "cuda:0", torch.bfloat16, torch.float32, torch.int32
+    flush = torch.zeros(160 << 20, dtype=f32, device=dev)
+    W = size["width"]
+    nq, nkv, hd, dims = size["attn"]
+    sh, sv, sn, sg, taps, parts = size["ssm"]
+    dh, dg, dd, dv, dtaps, rank = size["delta"]
+    E, top, eff = size["experts"]
+    ps, out = 64, {}
+
+    def row(name, fn, bytes_moved, flops=0.0, like=None):
+        us = timed_us(fn, flush)
+        floor = max(bytes_moved / (pk["hbm_gbs"] * 1e3), flops / (pk["bf16_tflops"] * 1e6))
+        out[name] = {"us": round(us, 1), "floor_us": round(floor, 2), "x_floor": round(us / max(floor, 1e-9), 1)}
+        if like is not None:
+            out[name].update(like=like, ratio=round((us / floor) / (out[like]["us"] / out[like]["floor"]), 2))
+        out[name]["floor"] = floor
+    g = torch.Generator(device=dev).manual_seed(1)
+
+    def rnd(*shape, dtype=f32, scale=1.0):
+        return (torch.randn(*shape, generator=g, device=dev, dtype=f32) * scale).to(dtype)
+    ints = lambda v: torch.tensor(v, dtype=i32, device=dev)
+    per_req = -(-(context + 1) // ps)
+    pages = batch * per_req + -(-T // ps) + 1
+    kp, vp = rnd(pages, nkv, ps, hd, dtype=bf), rnd(pages, nkv, ps, hd, dtype=bf)
+    for n, tag in ((T, "prefill"), (batch, "decode")):
+        R = 1 if tag == "prefill" else batch
+        one = R == 1
+        ctx = SimpleNamespace(positions=torch.arange(n, dtype=i32, device=dev) if one else ints([context] * n), token_req=ints([0] * n if one else list(range(n))),
+                              req_q_start=ints([0] if one else list(range(n))), req_q_len=ints([n] if one else [1] * n), req_slot=ints(list(range(R))))
+        reqs = (ctx.req_q_start, ctx.req_q_len, ctx.req_slot)
+        # ---- the norm behind a sublayer, the add and the rounded copy
+        resid, delta, gain, bias = rnd(n, W), rnd(n, W, dtype=bf), rnd(W, dtype=bf), rnd(W)
+        o = torch.empty(n, W, dtype=bf, device=dev)
+        sand = lambda **kw: ops.sandwich_norm(resid, (delta, 0), o, gain, False, 1e-6, None, 0.0, False, 0.0, post_offset=1.0, **kw)
+        row(f"{tag}/norm behind the sublayer+add+rounded copy", sand, n * W * (2 + 8 + 2))
+        row(f"{tag}/norm behind the sublayer+add+rounded copy, the projection's bias", lambda: sand(bias=bias), n * W * (2 + 8 + 2),
+            like=f"{tag}/norm behind the sublayer+add+rounded copy")
+        # ---- q | k | v into the pages
+        width = (nq + 2 * nkv) * hd
+        qkv, qo = rnd(n, width + 16, dtype=bf), torch.empty(n, nq * hd, dtype=bf, device=dev)
+        slots = torch.arange(n, dtype=i32, device=dev)
+        freq, qg, kg, brow = torch.rand(dims // 2, device=dev), rnd(nq * hd, dtype=bf), rnd(nkv * hd, dtype=bf), rnd(width)
+        rope = lambda **kw: ops.rope_row_norm_kv_write(qkv, qo, ctx.positions, slots, freq, kp, vp, nq, nkv, hd, dims, ps, qg, kg, 1e-6, nq * hd, nkv * hd, bias=brow, **kw)
+        row(f"{tag}/biases, row norms, turn, cache write", rope, n * width * 4)
+        row(f"{tag}/biases, row norms, scaled turn, cache write", lambda: rope(turn_scale=1.14), n * width * 4, like=f"{tag}/biases, row norms, turn, cache write")
+        row(f"{tag}/bias, row norm, scaled turn of q alone",
+            lambda: ops.rope_row_norm_kv_write(qkv, qo, ctx.positions, None, freq, None, None, nq, 0, hd, dims, ps, qg, None, 1e-6, nq * hd, 0, bias=brow[:nq * hd],
+                                               turn_scale=1.14), n * nq * hd * 4, like=f"{tag}/biases, row norms, turn, cache write")
+        # ---- attention
+        q, heads = rnd(n, nq * hd, dtype=bf), torch.empty(n, nq * hd, dtype=bf, device=dev)
+        sinks = torch.zeros(nq, device=dev)
+        if one:
+            table, ctx_len = torch.arange(-(-T // ps), dtype=i32, device=dev)[None].contiguous(), ints([T])
+            att = lambda **kw: ops.attention_mma_prefill(q, heads, kp, vp, ctx.req_q_start, ctx.req_q_len, ctx_len, table, n, nq, nkv, hd, ps, 0, hd ** -0.5,
+                                                         skip_single=False, **kw)
+            work = dict(bytes_moved=n * (2 * nq + 2 * nkv) * hd * 2, flops=2.0 * n * n * nq * hd)
+        else:
+            table = torch.arange(R * per_req, dtype=i32, device=dev).view(R, per_req)
+            split, most = ops.decode_split_plan(R * nkv, -(-(context + 1) // 512) * 512, 32)
+            scratch = torch.empty(ops.attention_mma_scratch_floats(R, nq, hd, most), device=dev)
+            ctx_len = ints([context + 1] * R)
+            att = lambda **kw: ops.attention_mma_decode(q, heads, kp, vp, ctx.req_q_start, ctx.req_q_len, ctx_len, table, nq, nkv, hd, ps, 0, hd ** -0.5, split, most,
+                                                        scratch, **kw)
+            work = dict(bytes_moved=R * (context + 1) * nkv * hd * 4, flops=4.0 * R * context * nq * hd)
+        row(f"{tag}/attention", att, **work)
+        row(f"{tag}/attention with a one in the denominator", lambda: att(sinks=sinks), **work, like=f"{tag}/attention")
+        gates = rnd(n, nq * hd, dtype=bf)
+        row(f"{tag}/sigmoid gate, an element each", lambda: ops.sigmoid_gate(heads, gates, 0, 0), n * nq * hd * 2 * 3)
+        row(f"{tag}/sigmoid gate, a head each", lambda: ops.sigmoid_gate(heads, gates, 0, 0, per=hd), n * nq * hd * 2 * 2, like=f"{tag}/sigmoid gate, an element each")
+        # ---- the delta rule: one decay per head, and per key channel
+        GD, HV = dg * dd, dh * dv
+        off = {"q": 0, "k": GD, "v": 2 * GD, "g": 2 * GD + HV, "b": 2 * GD + 2 * HV, "a": 2 * GD + 2 * HV + dh}
+        fused = rnd(n, 2 * GD + 2 * HV + 2 * dh, dtype=bf)
+        conv = [rnd(c, dtaps, dtype=bf) for c in (GD, GD, HV)]
+        a_log, dt_bias = rnd(dh, dtype=bf), rnd(dh, dtype=bf)
+        dq, dk, dvv, beta = torch.empty(n, GD, device=dev), torch.empty(n, GD, device=dev), torch.empty(n, HV, device=dev), torch.empty(n, dh, device=dev)
+        decay = torch.empty(n, dh, device=dev)
+        cstate = torch.zeros(batch + 1, dtaps - 1, 2 * GD + HV, device=dev)
+        shift = None if one else ctx.req_q_len
+        prep = lambda o_, a_, b_, d_, s_: ops.delta_prepare(fused, 0, o_, dh, dg, dd, dv, dtaps, *conv, a_, b_, ctx.token_req, ctx.req_q_start, ctx.req_slot, cstate, 1e-6,
+                                                            dd ** -0.5, dq, dk, dvv, beta, d_, shift=s_)
+        moved = n * (2 * GD + HV) * (2 + 4)
+        row(f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)", lambda: prep(off, a_log, dt_bias, decay, None), moved)
+        row(f"{tag}/delta rule: inputs without decays", lambda: prep({k: v for k, v in off.items() if k != "a"}, None, None, None, shift), moved,
+            like=f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)")
+        low, up, ub, ulog = rnd(n, 2 * rank, dtype=bf), rnd(dh * dd, rank, dtype=bf, scale=0.1), rnd(dh * dd, dtype=bf), rnd(dh, dtype=bf)
+        chan = torch.empty(n, dh * dd, device=dev)
+        moved = n * (rank * 2 + dh * dd * 4) + dh * dd * rank * 2
+        row(f"{tag}/time mixing: the decay", lambda: ops.linattn_decay(low, 0, 0, up, ub, dh, dd, chan), moved)
+        row(f"{tag}/delta rule: decays per key channel", lambda: ops.lowrank_map(low, 0, 0, up, dh, dd, chan, ub, ulog), moved, like=f"{tag}/time mixing: the decay")
+        gup, gate = rnd(HV, rank, dtype=bf, scale=0.1), torch.empty(n, HV, device=dev)
+        row(f"{tag}/delta rule: the low-rank gate", lambda: ops.lowrank_map(low, 0, rank, gup, dh, dv, gate), n * (rank * 2 + HV * 4) + HV * rank * 2,
+            like=f"{tag}/time mixing: the decay")
+        state, do = torch.zeros(batch + 1, dh, dd, dv, device=dev), torch.empty(n, HV, device=dev)
+        decay.uniform_(0.9, 1.0)
+        chan.uniform_(-0.1, 0.0)
+        sb, sf = R * 2 * dh * dd * dv * 4, 6.0 * n * dh * dd * dv
+        row(f"{tag}/delta rule: recurrence", lambda: ops.delta_scan(dq, dk, dvv, beta, decay, state, do, *reqs, dh, dg, dd, dv), n * (2 * GD + 2 * HV + 2 * dh) * 4 + sb, sf)
+        row(f"{tag}/delta rule: recurrence, decays per key channel", lambda: ops.delta_scan(dq, dk, dvv, beta, chan, state, do, *reqs, dh, dg, dd, dv, True),
+            n * (2 * GD + 2 * HV + dh + dh * dd) * 4 + sb, sf, like=f"{tag}/delta rule: recurrence")
+        hw, gated = rnd(dv, dtype=bf), torch.empty(n, HV, dtype=bf, device=dev)
+        row(f"{tag}/head norm and SiLU gate", lambda: ops.head_gate_norm(do, gate, 0, 0, hw, 1e-6, gated, dh, dv), n * HV * (4 + 4 + 2))
+        row(f"{tag}/head norm and sigmoid gate", lambda: ops.head_gate_norm(do, gate, 0, 0, hw, 1e-6, gated, dh, dv, gate_act="sigmoid"), n * HV * (4 + 4 + 2),
+            like=f"{tag}/head norm and SiLU gate")
+        # ---- the state space, beside the delta rule's inputs and the decayed state of linear attention with as many heads and elements
+        inner, C = sh * sv, sh * sv + 2 * sg * sn
+        sfused = rnd(n, inner + C + sh, dtype=bf)
+        sconv, scb, slog, sdt = rnd(C, taps), rnd(C), rnd(sh), rnd(sh)
+        xbc, pairs_ = torch.empty(n, C, device=dev), torch.empty(n, sh, 2, device=dev)
+        sc = torch.zeros(batch + 1, taps - 1, C, device=dev)
+        row(f"{tag}/state space: inputs (convolution, SiLU, steps, decays)",
+            lambda: ops.ssd_prepare(sfused, 0, inner, inner + C, taps, sconv, scb, slog, sdt, ctx, sc, xbc, pairs_, shift=not one), n * C * (2 + 4),
+            like=f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)")
+        xbc.normal_(generator=g)
+        pairs_.uniform_(-0.1, 0.0)
+        seg_len, max_seg = ops.linattn_segment_plan(n, 1, sh, sv) if one else (0, 1)
+        ss, sd = torch.empty(R * max_seg * sh * sn * sv, device=dev), torch.empty(R * max_seg * sh * sn, device=dev)
+        sstate, so = torch.zeros(batch + 1, sh, sn, sv, device=dev), torch.empty(n, inner, device=dev)
+        lq, lk, ldec = rnd(n, sh * sn), rnd(n, sh * sn), torch.rand(n, sh * sn, device=dev) * 0.1 + 0.9
+        lv = rnd(n, inner)
+        seg = (sh, sn, sv, seg_len, max_seg, ss, sd)
+        sb, sf = R * 2 * sh * sn * sv * 4, 4.0 * n * sh * sn * sv
+        row(f"{tag}/decayed state: recurrence (decay per key channel)", lambda: ops.linattn_scan(lq, lk, lv, ldec, None, sstate, so, *reqs, *seg),
+            n * (3 * sh * sn + 2 * inner) * 4 + sb, sf)
+        hdec = torch.rand(sh, device=dev) * 0.1 + 0.9
+        row(f"{tag}/decayed state: recurrence (one decay per head)", lambda: ops.linattn_scan(lq, lk, lv, None, hdec, sstate, so, *reqs, *seg),
+            n * (2 * sh * sn + 2 * inner) * 4 + sb, sf)
+        xs, bs, cs = xbc[:, :inner], xbc[:, inner:inner + sg * sn], xbc[:, inner + sg * sn:]
+        row(f"{tag}/state space: recurrence", lambda: ops.linattn_scan(cs, bs, xs, None, None, sstate, so, *reqs, *seg, pairs=pairs_, share=sh // sg),
+            n * (C + inner + 2 * sh) * 4 + sb, sf, like=f"{tag}/decayed state: recurrence (one decay per head)")
+        skip, nw, sgated = rnd(sh, dtype=bf), rnd(inner, dtype=bf), torch.empty(n, inner, dtype=bf, device=dev)
+        row(f"{tag}/state space: skip, gate, norm in parts", lambda: ops.ssd_gate_norm(so, xs, skip, sfused, 0, 0, nw, 1e-6, sgated, parts), n * inner * (4 + 4 + 2 + 2),
+            like=f"{tag}/head norm and SiLU gate")
+        # ---- experts
+        x, wr, rb = rnd(n, W, dtype=bf), rnd(E, W, scale=0.05), rnd(E)
+        chosen, weights = torch.empty(n, top, dtype=i32, device=dev), torch.empty(n, top, device=dev)
+        row(f"{tag}/router (softmax scores, choice)", lambda: ops.moe_route(x, wr, None, chosen, weights, None), n * W * 2 + E * W * 4)
+        row(f"{tag}/router with a bias, softmax over the chosen", lambda: ops.moe_route(x, wr, None, chosen, weights, None, scores="softmax_chosen", bias=rb),
+            n * W * 2 + E * W * 4, like=f"{tag}/router (softmax scores, choice)")
+        pairs = n * top
+        count, offset = torch.empty(E, dtype=i32, device=dev), torch.empty(E + 1, dtype=i32, device=dev)
+        order, place = torch.empty(pairs, dtype=i32, device=dev), torch.empty(pairs, dtype=i32, device=dev)
+        tiles = torch.empty(1 + 3 * ops.moe_row_tiles(pairs, E), dtype=i32, device=dev)
+        ops.moe_plan(chosen, count, offset, order, place, tiles, torch.empty(ops.MOE_PLAN_SEGMENTS * E, dtype=i32, device=dev))
+        w_gu, act = rnd(E, 2 * eff, W, dtype=bf, scale=0.02), torch.empty(pairs, eff, dtype=bf, device=dev)
+        used = int((count > 0).sum())
+        xr = rnd(pairs, W, dtype=bf)
+        unit = (lambda **kw: ops.gemm_bf16_tc_grouped(xr, w_gu, act, tiles, True, 7.0, 1.702, **kw)) if pairs >= 1024 else \
+            (lambda **kw: ops.moe_grouped(x, w_gu, act, offset, order, top, True, 7.0, 1.702, **kw))
+        work = dict(bytes_moved=used * 2 * eff * W * 2 + pairs * (W + eff) * 2, flops=4.0 * pairs * eff * W)
+        row(f"{tag}/experts: gate|up with the clamped unit", unit, **work)
+        row(f"{tag}/experts: gate|up with the SiLU unit", lambda: unit(unit="silu"), **work, like=f"{tag}/experts: gate|up with the clamped unit")
+    for r in out.values():
+        del r["floor"]
+    return out
+
+
+def vifirax_bench(args) -> int:
+    import torch
+    from wllm_b200.config import EngineConfig, GudaraxConfig, VifiraxConfig
+    from wllm_b200.engine import build_model
+    pk = peaks()
+    ps, T = args.page_size, 2048
+    context = args.context or 2048
+    engine_cfg = EngineConfig(dtype="bfloat16", block_size=ps, max_num_seqs=max(64, args.batch), cuda_graphs=not args.no_graphs)
+    sizes = {}
+    for name in (args.sizes if args.sizes != "2b,7b" else "2k,4k").split(","):
+        size = VIFIRAX_SIZES[name]
+        models = {"gudarax": GudaraxConfig.from_dict(vifirax_like_config(size)), "vifirax": VifiraxConfig.from_dict(vifirax_config(size))}
+        res = {}
+        for label, cfg in models.items():
+            model = build_model(None, engine_cfg.dtype, engine_cfg.device, config=cfg, random_seed=1)
+            pre_ms = prefill_run(model, engine_cfg, T, ps)
+            ms, launches, _, clocks, _ = decode_run(model, engine_cfg, args.batch, context, min(args.steps, 32), args.warmup, ps, 3)
+            res[label] = {"weights_gb": round(model.weight_bytes() / 1e9, 3), "prefill_tok_s": round(T / (pre_ms / 1e3), 1),
+                          "prefill_ms": round(pre_ms, 3), "decode_tok_s": round(args.batch / (ms / 1e3), 1),
+                          "decode_ms_per_step": round(ms, 4), "decode_launches": launches,
+                          "decode_weights_hbm_frac": round(model.weight_bytes() / (ms / 1e3) / 1e9 / pk["hbm_gbs"], 3), "clocks": clocks}
+            del model
+            torch.cuda.empty_cache()
+        sizes[name] = {"shape": size, "models": res}
+        if not args.no_points:
+            sizes[name]["kernels"] = vifirax_kernel_table(size, pk, T, args.batch, context)
+    print(json.dumps({"metric": "Vifirax beside Gudarax at equal layer sizes: prefill tok/s @ 2048 tokens, decode tok/s",
+                      "design": "vifirax", "unit": "tokens/s", "n_gpus": 1, "steps": min(args.steps, 32), "warmup": args.warmup,
+                      "dtype": "bf16", "data": "synthetic (random weights, random token ids, random cached keys/values)",
+                      "config": {"global_batch": args.batch, "seq_len": context, "prefill_tokens": T, "page_size": ps,
+                                 "cuda_graphs": not args.no_graphs, "peaks": pk["source"],
+                                 "l2": "kernel table: a 640 MB buffer is written before every timed launch"},
+                      "peaks": pk, "sizes": sizes}))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1460,7 +1696,7 @@ def main() -> int:
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-points", action="store_true")
     ap.add_argument("--regions", type=int, default=5, help="timed regions of --steps steps each; the median is reported")
-    ap.add_argument("--design", default="gemma", choices=["gemma", "pesanex", "taritar", "zafilix", "gudarax", "fusanex"],
+    ap.add_argument("--design", default="gemma", choices=["gemma", "pesanex", "taritar", "zafilix", "gudarax", "fusanex", "vifirax"],
                     help="gemma: the default workload; the others: models of that design beside a model of an earlier design of equal layer sizes (another line)")
     ap.add_argument("--sizes", default="2b,7b", help="which of the layer sizes to run (--design pesanex: 2b, 7b; the others: 2k, 4k)")
     args = ap.parse_args()
@@ -1480,6 +1716,8 @@ def main() -> int:
         return gudarax_bench(args)
     if args.design == "fusanex":
         return fusanex_bench(args)
+    if args.design == "vifirax":
+        return vifirax_bench(args)
     import torch
     from wllm_b200.config import EngineConfig, GemmaConfig
     from wllm_b200.engine import build_model
