@@ -1598,9 +1598,10 @@ def vifirax_kernel_table(size: dict, pk: dict, T: int, batch: int, context: int)
         sfused = rnd(n, inner + C + sh, dtype=bf)
         sconv, scb, slog, sdt = rnd(C, taps), rnd(C), rnd(sh), rnd(sh)
         xbc, pairs_ = torch.empty(n, C, device=dev), torch.empty(n, sh, 2, device=dev)
+        made = torch.empty(n, C, dtype=bf if one else f32, device=dev)
         sc = torch.zeros(batch + 1, taps - 1, C, device=dev)
         row(f"{tag}/state space: inputs (convolution, SiLU, steps, decays)",
-            lambda: ops.ssd_prepare(sfused, 0, inner, inner + C, taps, sconv, scb, slog, sdt, ctx, sc, xbc, pairs_, shift=not one), n * C * (2 + 4),
+            lambda: ops.ssd_prepare(sfused, 0, inner, inner + C, taps, sconv, scb, slog, sdt, ctx, sc, made, pairs_, shift=not one), n * C * (4 if one else 6),
             like=f"{tag}/delta rule: inputs (convolutions, SiLU, unit norms, step sizes, decays)")
         xbc.normal_(generator=g)
         pairs_.uniform_(-0.1, 0.0)
@@ -1617,10 +1618,17 @@ def vifirax_kernel_table(size: dict, pk: dict, T: int, batch: int, context: int)
         row(f"{tag}/decayed state: recurrence (one decay per head)", lambda: ops.linattn_scan(lq, lk, lv, None, hdec, sstate, so, *reqs, *seg),
             n * (2 * sh * sn + 2 * inner) * 4 + sb, sf)
         xs, bs, cs = xbc[:, :inner], xbc[:, inner:inner + sg * sn], xbc[:, inner + sg * sn:]
-        row(f"{tag}/state space: recurrence", lambda: ops.linattn_scan(cs, bs, xs, None, None, sstate, so, *reqs, *seg, pairs=pairs_, share=sh // sg),
-            n * (C + inner + 2 * sh) * 4 + sb, sf, like=f"{tag}/decayed state: recurrence (one decay per head)")
+        if one:
+            xbc16 = xbc.to(bf)
+            xs = xbc16[:, :inner]
+            row(f"{tag}/state space: recurrence in chunks", lambda: ops.ssd_chunks(xbc16, pairs_, sstate, so, *reqs, sh, sh // sg, sn, sv),
+                n * (C * 2 + inner * 4 + sh * 8) + sb, sf, like=f"{tag}/decayed state: recurrence (one decay per head)")
+        else:
+            row(f"{tag}/state space: recurrence", lambda: ops.linattn_scan(cs, bs, xs, None, None, sstate, so, *reqs, *seg, pairs=pairs_, share=sh // sg),
+                n * (C + inner + 2 * sh) * 4 + sb, sf, like=f"{tag}/decayed state: recurrence (one decay per head)")
         skip, nw, sgated = rnd(sh, dtype=bf), rnd(inner, dtype=bf), torch.empty(n, inner, dtype=bf, device=dev)
-        row(f"{tag}/state space: skip, gate, norm in parts", lambda: ops.ssd_gate_norm(so, xs, skip, sfused, 0, 0, nw, 1e-6, sgated, parts), n * inner * (4 + 4 + 2 + 2),
+        row(f"{tag}/state space: skip, gate, norm in parts", lambda: ops.ssd_gate_norm(so, xs, skip, sfused, 0, 0, nw, 1e-6, sgated, parts),
+            n * inner * (4 + (2 if one else 4) + 2 + 2),
             like=f"{tag}/head norm and SiLU gate")
         # ---- experts
         x, wr, rb = rnd(n, W, dtype=bf), rnd(E, W, scale=0.05), rnd(E)

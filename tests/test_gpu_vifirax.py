@@ -6,7 +6,7 @@ another in 32-bit; long prompts and long decoding; batches of unequal requests; 
 that reads another's keys; decoding from captured graphs; greedy generation through the scheduler; the trace runner; a model without any
 attention.  Mechanisms alone: the turn with a factor, row norms and biases with and without keys of the mixer's own, a one in the softmax's
 denominator, one gate per head, a bias on a branch, low-rank maps and the decays made of them, the state space and the delta rule with decays per
-key channel across portions, segments and slots (a write far back read much later), the router's softmax over the chosen logits, experts of
+key channel across portions, chunks, segments and slots (a write far back read much later), the router's softmax over the chosen logits, experts of
 SiLU units (few rows and many).
 """
 import json
@@ -594,7 +594,7 @@ def check_portions(part, names, tensors, want, hs, dtype):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("sizes", [(4, 24, 16, 2, 4, 3), (3, 10, 7, 1, 2, 2), (2, 64, 128, 1, 4, 1), (6, 8, 256, 3, 3, 6), (2, 80, 24, 2, 1, 5), (1, 16, 16, 1, 7, 1)])
+@pytest.mark.parametrize("sizes", [(4, 24, 16, 2, 4, 3), (3, 10, 7, 1, 2, 2), (2, 64, 128, 1, 4, 1), (6, 8, 256, 3, 3, 6), (2, 80, 24, 2, 1, 5), (1, 16, 16, 1, 7, 1), (4, 40, 48, 2, 4, 2)])
 def test_the_state_space_across_portions_segments_and_slots(sizes, dtype):
     """heads, values, state rows, groups, taps, norm groups of widely different sizes against the plain statement on whole sequences; an early
     token's large value still read three hundred tokens later through a head that forgets next to nothing."""
@@ -623,6 +623,50 @@ def test_the_state_space_across_portions_segments_and_slots(sizes, dtype):
     quiet[3] = 0.0
     assert (plain.mamba2(m, wd, "", quiet, 1e-5)[-1] - want[0][-1]).abs().max() > 0.02 * float(want[0].abs().max())
     check_portions(part, None, None, want, hs, dtype)
+
+
+@pytest.mark.parametrize("H,G,N,V", [(2, 1, 16, 8), (4, 2, 128, 64), (3, 3, 48, 40), (2, 2, 112, 24), (6, 2, 64, 72), (1, 1, 80, 32)])
+def test_the_state_space_in_chunks(H, G, N, V):
+    """The chunked kernel alone on given rows: requests whose lengths lie around a chunk's border, in one batch, in two steps that carry the state;
+    for pairs of places at both sides of the borders the row B of one and the row C of the other are made to agree, so that one write decides one
+    read; heads that forget within a token and heads that forget next to nothing."""
+    from wllm_b200.kernels import ops
+    g = torch.Generator().manual_seed(H * 100 + N)
+    lengths = (1, 2, 63, 64, 65, 129, 200, 128)
+    slots = list(range(len(lengths)))[::-1]
+    C = H * V + 2 * G * N
+    state = torch.full((len(lengths) + 1, H, N, V), float("nan"), device=DEV)
+    state[:len(lengths)] = 0.0
+    rate = torch.logspace(-6, 0.5, H, dtype=torch.float64) if H > 1 else torch.tensor([1e-3], dtype=torch.float64)
+    parts = {i: [] for i in range(len(lengths))}
+    got = {i: [] for i in range(len(lengths))}
+    for step in range(2):
+        lens = list(lengths if step == 0 else lengths[::-1])
+        n = sum(lens)
+        xbc = torch.randn(n, C, generator=g) * 0.3
+        starts = [sum(lens[:i]) for i in range(len(lens))]
+        b, c = H * V, H * V + G * N
+        for t0, L in zip(starts, lens):
+            for s, t in ((0, L - 1), (62, 63), (63, 64), (0, 64), (64, 127), (63, 128), (1, 199)):
+                if s <= t < L:
+                    v = torch.randn(G * N, generator=g)
+                    xbc[t0 + s, b:b + G * N], xbc[t0 + t, c:c + G * N] = v, v
+        xbc = xbc.to(torch.bfloat16)
+        dt = torch.rand(n, H, generator=g).double() + 0.05
+        pairs = torch.stack([-rate * dt, dt], dim=-1).float().contiguous()
+        out = torch.full((n, H * V), float("nan"), device=DEV)
+        ops.ssd_chunks(xbc.to(DEV), pairs.to(DEV), state, out, i32(starts), i32(lens), i32(slots), H, H // G, N, V)
+        for i, (t0, L) in enumerate(zip(starts, lens)):
+            parts[i].append((xbc[t0:t0 + L].double(), dt[t0:t0 + L]))
+            got[i].append(out[t0:t0 + L].double().cpu())
+    for i in parts:
+        x = torch.cat([p[0] for p in parts[i]])
+        n = x.shape[0]
+        want = plain.ssd(x[:, :H * V].reshape(n, H, V), x[:, H * V:H * V + G * N].reshape(n, G, N), x[:, H * V + G * N:].reshape(n, G, N),
+                         torch.cat([p[1] for p in parts[i]]), -rate, torch.zeros(H, dtype=torch.float64)).reshape(n, H * V)
+        scale = want.abs().view(n, H, V).amax(dim=(0, 2)).repeat_interleave(V).clamp(min=1e-3)
+        assert ((torch.cat(got[i]) - want).abs() / scale).max() < 2e-4, (i, lengths[i])
+    assert torch.isnan(state[-1]).all()
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])

@@ -1279,14 +1279,14 @@ def ssd_prepare(fused, parts: int, x_off: int, dt_off: int, taps: int, conv: tor
     """What enters a state space (csrc/state_space.cu) from the fused projection [n, W] (or float32 partial sums [parts, n, W]): the
     columns from `x_off` through their causal convolution (conv [C, taps], the last tap the token's own; conv_bias [C] or None; the inputs in
     front of a portion come from `conv_state` [slots, taps - 1, C]) and SiLU into out [n, C]; the columns dt_off .. + heads become
-    pairs [n, heads, 2] = (a - 1, dt), dt = softplus(. + dt_bias), a = exp(-exp(a_log) dt).  `shift` (every request of the step brings at
-    most one token): conv_state is brought up to date too."""
+    pairs [n, heads, 2] = (a - 1, dt), dt = softplus(. + dt_bias), a = exp(-exp(a_log) dt); out in bfloat16 (for ssd_chunks): the pairs are
+    (log a, dt).  `shift` (every request of the step brings at most one token): conv_state is brought up to date too."""
     _need_cuda(fused, conv, conv_bias, a_log, dt_bias, conv_state, out, pairs)
     ptr, dt, row_stride, nparts, part_stride, n = _fused_args(fused, parts)
     C, H = conv.shape[0], a_log.shape[0]
     assert conv.shape == (C, taps) and a_log.shape == dt_bias.shape == (H,) and conv.dtype == a_log.dtype == dt_bias.dtype
     assert conv_bias is None or (conv_bias.shape == (C,) and conv_bias.dtype == conv.dtype and conv_bias.is_contiguous())
-    assert out.shape == (n, C) and pairs.shape == (n, H, 2) and out.dtype == pairs.dtype == torch.float32
+    assert out.shape == (n, C) and pairs.shape == (n, H, 2) and pairs.dtype == torch.float32
     assert all(t.is_contiguous() for t in (conv, a_log, dt_bias, out, pairs))
     assert x_off + C <= fused.shape[-1] and dt_off + H <= fused.shape[-1]
     assert taps == 1 or (conv_state.dtype == torch.float32 and conv_state.is_contiguous() and conv_state.shape[1:] == (taps - 1, C))
@@ -1294,8 +1294,34 @@ def ssd_prepare(fused, parts: int, x_off: int, dt_off: int, taps: int, conv: tor
     _check(lib.wllm_ssd_prepare(ptr, dt, row_stride, nparts, part_stride, x_off, dt_off, n, C, H, taps, _ptr(conv), _ptr(conv_bias),
                                 _ptr(a_log), _ptr(dt_bias), _dt(conv), _ptr(_int32(ctx.token_req, "token_req")),
                                 _ptr(_int32(ctx.req_q_start, "req_q_start")), _ptr(_int32(ctx.req_q_len, "req_q_len")),
-                                _ptr(_int32(ctx.req_slot, "req_slot")), _ptr(conv_state if taps > 1 else None), _ptr(out), _ptr(pairs),
+                                _ptr(_int32(ctx.req_slot, "req_slot")), _ptr(conv_state if taps > 1 else None), _ptr(out), _dt(out), _ptr(pairs),
                                 1 if shift and taps > 1 else 0, _stream()), "ssd_prepare")
+
+
+SSD_CHUNKS_FROM = 64       # a step whose longest portion has this many tokens runs the state space in chunks (bfloat16)
+
+
+def ssd_chunks_ok(heads: int, state_dim: int, vdim: int) -> bool:
+    """Sizes the chunked state space takes: state rows in steps of 16 up to 128, values in steps of 8."""
+    return state_dim % 16 == 0 and state_dim <= 128 and vdim % 8 == 0
+
+
+def ssd_chunks(xbc: torch.Tensor, pairs: torch.Tensor, state: torch.Tensor, out: torch.Tensor, req_q_start, req_q_len, req_slot, heads: int, share: int,
+               state_dim: int, vdim: int) -> torch.Tensor:
+    """The state space over every request's tokens of the step in chunks on the tensor cores (csrc/state_space.cu): xbc [n, x | B | C]
+    bfloat16 and pairs [n, heads, 2] = (log a, dt) as ssd_prepare leaves them; S <- a S + dt B x^T from and to `state` [slots, heads,
+    state_dim, vdim], out [n, heads * vdim] = S^T C, float32."""
+    _need_cuda(xbc, pairs, state, out, req_q_start, req_q_len, req_slot)
+    n, inner, rows = xbc.shape[0], heads * vdim, heads // share * state_dim
+    assert xbc.dtype == torch.bfloat16 and xbc.is_contiguous() and xbc.shape[1] == inner + 2 * rows and heads % share == 0
+    assert pairs.dtype == torch.float32 and pairs.is_contiguous() and pairs.shape == (n, heads, 2)
+    assert state.dtype == out.dtype == torch.float32 and state.is_contiguous() and out.is_contiguous()
+    assert state.shape[1:] == (heads, state_dim, vdim) and out.shape == (n, inner)
+    lib = load_family("state_space")
+    _check(lib.wllm_ssd_chunks(_ptr(xbc), xbc.shape[1], inner, inner + rows, _ptr(pairs), _ptr(state), _ptr(out),
+                               _ptr(_int32(req_q_start, "req_q_start")), _ptr(_int32(req_q_len, "req_q_len")), _ptr(_int32(req_slot, "req_slot")),
+                               req_q_len.shape[0], heads, share, state_dim, vdim, _stream()), f"ssd_chunks(heads={heads}, state={state_dim}x{vdim})")
+    return out
 
 
 def ssd_conv_update(fused, parts: int, x_off: int, taps: int, ctx, conv_state: torch.Tensor) -> None:
@@ -1311,16 +1337,16 @@ def ssd_conv_update(fused, parts: int, x_off: int, taps: int, ctx, conv_state: t
 
 def ssd_gate_norm(o: torch.Tensor, x: torch.Tensor, skip: torch.Tensor, fused, parts: int, z_off: int, weight: torch.Tensor, eps: float,
                   out: torch.Tensor, groups: int) -> torch.Tensor:
-    """out [n, inner] = y / sqrt(mean over a part of y^2 + eps) * weight, the row being `groups` equal parts, y = (o + skip_h x) silu(z): o, x
-    [n, inner] float32 (x may be columns of wider rows), skip [heads], z the columns of `fused` from z_off; 32-bit inside, rounded once."""
+    """out [n, inner] = y / sqrt(mean over a part of y^2 + eps) * weight, the row being `groups` equal parts, y = (o + skip_h x) silu(z): o
+    [n, inner] float32, x of either type (it may be columns of wider rows), skip [heads], z the columns of `fused` from z_off; 32-bit inside, rounded once."""
     _need_cuda(o, x, skip, fused, weight, out)
     ptr, dt, row_stride, nparts, part_stride, n = _fused_args(fused, parts)
     inner, H = o.shape[1], skip.shape[0]
-    assert o.dtype == x.dtype == torch.float32 and o.is_contiguous() and x.shape == o.shape == out.shape == (n, inner) and x.stride(1) == 1
+    assert o.dtype == torch.float32 and o.is_contiguous() and x.shape == o.shape == out.shape == (n, inner) and x.stride(1) == 1
     assert skip.dtype == weight.dtype and weight.shape == (inner,) and weight.is_contiguous() and skip.is_contiguous() and inner % H == 0
     assert out.is_contiguous() and z_off + inner <= fused.shape[-1]
     lib = load_family("state_space")
-    _check(lib.wllm_ssd_gate_norm(_ptr(o), _ptr(x), ctypes.c_longlong(max(x.stride(0), inner)), _ptr(skip), ptr, dt, row_stride, nparts,
+    _check(lib.wllm_ssd_gate_norm(_ptr(o), _ptr(x), _dt(x), ctypes.c_longlong(max(x.stride(0), inner)), _ptr(skip), ptr, dt, row_stride, nparts,
                                   part_stride, z_off, _ptr(weight), _dt(weight), c_float(eps), _ptr(out), _dt(out), n, inner, inner // H,
                                   groups, _stream()), "ssd_gate_norm")
     return out

@@ -13,8 +13,9 @@ then o_proj.
 spec options: num_heads, groups, state_dim, value_dim, conv_taps, norm_groups, eps, in_proj, conv, conv_bias (None: no bias), decay_log,
 step_bias, skip, norm_weight, o_proj (checkpoint names).
 
-Convolution, steps, decays and state are 32-bit (csrc/state_space.cu); the recurrence is the decayed-state scan of
-csrc/linear_attention.cu with q = C, k = B, v = x, whose long portions run in segments side by side.
+Steps, decays and state are 32-bit (csrc/state_space.cu).  The recurrence is the decayed-state scan of csrc/linear_attention.cu with q = C,
+k = B, v = x, whose long portions run in segments side by side, and, under bfloat16 in steps with portions of `SSD_CHUNKS_FROM` tokens and
+more, a form in chunks on the tensor cores, which takes x, B and C in bfloat16.
 """
 from __future__ import annotations
 
@@ -41,6 +42,7 @@ class StateSpace:
         self.channels = self.inner + 2 * self.groups * self.state_dim
         self.width = self.inner + self.channels + self.heads
         self.hidden_size, self.model_dtype = hidden_size, model_dtype
+        self.chunks = model_dtype == torch.bfloat16 and ops.ssd_chunks_ok(self.heads, self.state_dim, self.vdim)
         self.names = {k: spec.options[k] for k in ("in_proj", "conv", "decay_log", "step_bias", "skip", "norm_weight", "o_proj")}
         self.bias_name = spec.options.get("conv_bias")
         self.tag = ""
@@ -84,7 +86,8 @@ class StateSpace:
         """The mixer on the columns from col0 of a fused product [n, W] (or partial sums [parts, n, W])."""
         n, H, N, V, f32 = fused.shape[-2], self.heads, self.state_dim, self.vdim, torch.float32
         inner, rows = self.inner, self.groups * self.state_dim
-        xbc = ctx.buffer(self.tag + "ssd_xbc", (n, self.channels), f32)
+        chunked = self.chunks and ctx.max_q_len >= ops.SSD_CHUNKS_FROM
+        xbc = ctx.buffer(self.tag + "ssd_xbc", (n, self.channels), self.model_dtype if chunked else f32)
         pairs = ctx.buffer(self.tag + "ssd_pairs", (n, H, 2), f32)
         conv_state = ctx.state(cache.state_names["conv"]) if self.taps > 1 else None
         single = ctx.num_multi == 0              # no request brings more than one token
@@ -94,14 +97,18 @@ class StateSpace:
             ops.ssd_conv_update(fused, parts, col0 + inner, self.taps, ctx, conv_state)
         x, b, c = xbc[:, :inner], xbc[:, inner:inner + rows], xbc[:, inner + rows:]
         o = ctx.buffer(self.tag + "ssd_o", (n, inner), f32)
-        seg_len, max_seg = ops.linattn_segment_plan(ctx.max_q_len, ctx.num_multi, H, V)
-        seg_state = seg_decay = None
-        if max_seg > 1:
-            R = ctx.n_requests
-            seg_state = ctx.buffer(self.tag + "ssd_seg_state", (R * max_seg * H * N * V,), f32)
-            seg_decay = ctx.buffer(self.tag + "ssd_seg_decay", (R * max_seg * H * N,), f32)
-        ops.linattn_scan(c, b, x, None, None, ctx.state(cache.state_names["state"]), o, ctx.req_q_start, ctx.req_q_len, ctx.req_slot,
-                         H, N, V, seg_len, max_seg, seg_state, seg_decay, pairs=pairs, share=H // self.groups)
+        state, share = ctx.state(cache.state_names["state"]), H // self.groups
+        if chunked:
+            ops.ssd_chunks(xbc, pairs, state, o, ctx.req_q_start, ctx.req_q_len, ctx.req_slot, H, share, N, V)
+        else:
+            seg_len, max_seg = ops.linattn_segment_plan(ctx.max_q_len, ctx.num_multi, H, V)
+            seg_state = seg_decay = None
+            if max_seg > 1:
+                R = ctx.n_requests
+                seg_state = ctx.buffer(self.tag + "ssd_seg_state", (R * max_seg * H * N * V,), f32)
+                seg_decay = ctx.buffer(self.tag + "ssd_seg_decay", (R * max_seg * H * N,), f32)
+            ops.linattn_scan(c, b, x, None, None, state, o, ctx.req_q_start, ctx.req_q_len, ctx.req_slot, H, N, V, seg_len, max_seg, seg_state,
+                             seg_decay, pairs=pairs, share=share)
         gated = ctx.buffer(self.tag + "ssd_gated", (n, inner), self.model_dtype)
         ops.ssd_gate_norm(o, x, self.skip, fused, parts, col0, self.gain, self.eps, gated, self.norm_groups)
         return as_branch(ops.project(gated, self.wo, lambda name, shape, dt: ctx.buffer(self.tag + "ssd_out_" + name, shape, dt)))
