@@ -1462,7 +1462,7 @@ def vifirax_config(size: dict) -> dict:
     E, top, eff = size["experts"]
     dense, moe = {"kind": "dense", "ff": size["ff"]}, {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}}
     att = {"heads": nq, "kv_heads": nkv, "dim": hd, "vdim": hd, "scale": hd ** -0.5,
-           "rot": {"dims": dims, "base": 1e6, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+           "rot": {"dims": dims, "base": 5e5, "scaling": {"factor": 8.0, "original": 4096, "fast": 24.0, "slow": 2.0}}}
     return {"architecture": "Vifirax", "vocab": size["vocab"], "width": size["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5, "layers": [
         {"type": "mamba2", "mixer": {"heads": sh, "vdim": sv, "state": sn, "groups": sg, "conv": taps, "norm_groups": parts}, "mlp": moe},
         {"type": "channel_delta", "mixer": {"heads": dh, "kv_heads": dg, "dim": dd, "vdim": dv, "conv": dtaps, "decay_rank": rank, "gate_rank": rank}, "mlp": dense},

@@ -87,7 +87,7 @@ def test_cache_groups_and_state_follow_from_the_mixers():
 
 
 @pytest.mark.parametrize("rot", [
-    {"dims": 16, "base": 10000.0, "scaling": {"factor": 4.0, "original": 512, "fast": 32.0, "slow": 1.0}},
+    {"dims": 20, "base": 10000.0, "scaling": {"factor": 6.0, "original": 512, "fast": 32.0, "slow": 1.0}},
     {"dims": 64, "base": 500000.0, "scaling": {"factor": 16.0, "original": 8192, "fast": 20.0, "slow": 2.0}},
     {"dims": 12, "base": 500.0, "scaling": {"factor": 3.0, "original": 64, "fast": 8.0, "slow": 1.0}},
     {"dims": 6, "base": 50.0, "scaling": {"factor": 5.0, "original": 20, "fast": 3.0, "slow": 2.9}},       # the band between is narrow
